@@ -74,6 +74,41 @@ typedef struct {
     int32_t vocab_size_per_layer_input;  /* rows of embed_tokens_per_layer.weight                        */
 } oxg4_config;
 
+/* Models whose layers are listed one by one, each with its own mixer, sizes and (optional) feed-forward, between
+ * norms before and after every sublayer: x += norm_b(f(norm(x))). No counterpart in the reference. Everything but
+ * model creation goes through the same entry points as a Gemma 4 model. */
+typedef enum {
+    OXG4_MIXER_GQA = 0,               /* the attention of the Gemma 4 models; not valid in a layer list */
+    OXG4_MIXER_LATENT_ATTENTION = 1,  /* low-rank queries, one cached latent and one rotated key part per token */
+    OXG4_MIXER_LIGHTNING = 2,         /* linear attention with a fixed decay per head                          */
+    OXG4_MIXER_WKV = 3                /* RWKV-style time mixing: token shift, decay per token and channel      */
+} oxg4_mixer;
+
+typedef struct {
+    int32_t mixer;                    /* oxg4_mixer                                                            */
+    int32_t heads;
+    int32_t dim;                      /* key size per head (latent attention: the unrotated part)             */
+    int32_t vdim;                     /* value size per head (wkv: equal to dim)                              */
+    int32_t q_rank;                   /* latent attention: query latent                                        */
+    int32_t kv_rank;                  /*                   cached latent                                       */
+    int32_t rot_dim;                  /*                   rotated part of queries and keys                    */
+    int32_t rot_dims;                 /*                   how many of its dimensions turn                     */
+    float rot_base;
+    float scale;                      /*                   factor on the scores                                */
+    const float* decay;               /* lightning: [heads]                                                    */
+    int32_t ff;                       /* SiLU-gated feed-forward of this width after the mixer; 0 = none       */
+    int32_t weights_of;               /* -1, or the layer whose tensors this layer uses (own cache and state)  */
+} oxg4_layer_spec;
+
+typedef struct {
+    int32_t vocab_size;
+    int32_t width;
+    int32_t num_layers;
+    float norm_eps;
+    int32_t weight_dtype;             /* as in oxg4_config                                                     */
+    const oxg4_layer_spec* layers;    /* [num_layers]                                                          */
+} oxg4_layered_config;
+
 typedef struct {
     int32_t batch;
     int32_t layer_count;              /* Gemma4CudaCacheTable::layer_count                          */
@@ -91,6 +126,10 @@ const char* oxg4_last_error(void);
 
 /* CudaContext::new(n) + stream creation (mod.rs:221-232). `device` is the ordinal of Device::Cuda(n). */
 int32_t oxg4_model_create(const oxg4_config* config, int32_t device, oxg4_model** out);
+
+/* A model of listed layers. Tensor names for oxg4_model_upload: "embed", "head", "final.norm" and "l<i>." + norm1, norm1b,
+ * norm2, norm2b, mix.*, mlp.* (synthetic.layered_weight_names lists them with their shapes). */
+int32_t oxg4_model_create_layered(const oxg4_layered_config* config, int32_t device, oxg4_model** out);
 
 /* Upload of one checkpoint tensor (mod.rs:236-279). `name` is the checkpoint name with or without
  * the "model.language_model." prefix. The copy has completed when the call returns, so it may be
@@ -173,6 +212,9 @@ int32_t oxg4_cache_position(const oxg4_cache* cache, int32_t b);
  * (reset_generation_state, mod.rs:178-180, plus a fresh table). */
 int32_t oxg4_cache_reset(oxg4_cache* cache);
 
+/* The same for one sequence of the table: its pages, state slot and row can serve another request. */
+int32_t oxg4_cache_reset_sequence(oxg4_cache* cache, int32_t b);
+
 /* ---- steps ------------------------------------------------------------------------------------------ */
 
 /* prefill_prompt (gemma4_cuda/decode.rs:431-459). `tokens` holds the prompts back to back,
@@ -180,6 +222,12 @@ int32_t oxg4_cache_reset(oxg4_cache* cache);
  * of each prompt's final token. The cache must be empty. */
 int32_t oxg4_prefill(oxg4_model* model, oxg4_cache* cache, const uint32_t* tokens,
                      const int32_t* lens, float* last_logits);
+
+/* Portions (no counterpart in the reference): lens[b] >= 0 further tokens of every sequence, which continues where its
+ * cache and state stand; `tokens` holds them back to back. want (may be NULL) has one byte per token; the logits of the
+ * tokens marked non-zero are written to `logits`, [number marked, vocab], in token order. */
+int32_t oxg4_extend(oxg4_model* model, oxg4_cache* cache, const uint32_t* tokens, const int32_t* lens,
+                    const uint8_t* want, float* logits);
 
 /* prefill_token (decode.rs:464-472): one token per sequence, no LM head.
  * A token id of 0xFFFFFFFF leaves that sequence untouched in this step. */

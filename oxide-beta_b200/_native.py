@@ -30,6 +30,21 @@ class Config(C.Structure):
         ("vocab_size_per_layer_input", C.c_int32)]
 
 
+class LayerSpec(C.Structure):
+    _fields_ = [("mixer", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("q_rank", C.c_int32),
+                ("kv_rank", C.c_int32), ("rot_dim", C.c_int32), ("rot_dims", C.c_int32), ("rot_base", C.c_float),
+                ("scale", C.c_float), ("decay", C.POINTER(C.c_float)), ("ff", C.c_int32), ("weights_of", C.c_int32)]
+
+
+class LayeredConfig(C.Structure):
+    _fields_ = [("vocab_size", C.c_int32), ("width", C.c_int32), ("num_layers", C.c_int32), ("norm_eps", C.c_float),
+                ("weight_dtype", C.c_int32), ("layers", C.POINTER(LayerSpec))]
+
+
+# oxg4_mixer
+MIXERS = {"latent_attention": 1, "lightning": 2, "wkv": 3}
+
+
 class CacheInfo(C.Structure):
     _fields_ = [("batch", C.c_int32), ("layer_count", C.c_int32), ("physical_cache_count", C.c_int32),
                 ("shared_layer_count", C.c_int32), ("page_tokens", C.c_int32), ("kv_dtype", C.c_int32),
@@ -50,6 +65,7 @@ TOKEN_CALLBACK = C.CFUNCTYPE(C.c_int32, C.c_uint32, C.c_void_p)
 SYMBOLS = {
     "oxg4_last_error": (C.c_char_p, []),
     "oxg4_model_create": (C.c_int32, [C.POINTER(Config), C.c_int32, C.POINTER(C.c_void_p)]),
+    "oxg4_model_create_layered": (C.c_int32, [C.POINTER(LayeredConfig), C.c_int32, C.POINTER(C.c_void_p)]),
     "oxg4_model_upload": (C.c_int32, [C.c_void_p, C.c_char_p, C.c_int32, C.POINTER(C.c_int64), C.c_int32,
                                       C.c_void_p, C.c_size_t]),
     "oxg4_model_finalize": (C.c_int32, [C.c_void_p]),
@@ -85,6 +101,8 @@ SYMBOLS = {
     "oxg4_cache_info_get": (C.c_int32, [C.c_void_p, C.POINTER(CacheInfo)]),
     "oxg4_cache_position": (C.c_int32, [C.c_void_p, C.c_int32]),
     "oxg4_cache_reset": (C.c_int32, [C.c_void_p]),
+    "oxg4_cache_reset_sequence": (C.c_int32, [C.c_void_p, C.c_int32]),
+    "oxg4_extend": (C.c_int32, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p]),
     "oxg4_prefill": (C.c_int32, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p]),
     "oxg4_prefill_token": (C.c_int32, [C.c_void_p, C.c_void_p, C.c_void_p]),
     "oxg4_decode_logits": (C.c_int32, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p]),

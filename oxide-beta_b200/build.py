@@ -4,6 +4,7 @@
 shared object sits next to this file so that it travels with the source tree; it is never
 installed into site-packages.
 """
+import fcntl
 import os
 import subprocess
 import sys
@@ -16,7 +17,7 @@ SOURCES = ["oxg4.cu"]
 
 def _newest_source() -> float:
     # every file under csrc/ is compiled into the one translation unit: any edit triggers a rebuild
-    files = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cu", ".cuh", ".h"))]
+    files = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cu", ".cuh", ".h", ".inl"))]
     files.append(os.path.join(os.path.dirname(HERE), "include", "oxg4.h"))
     return max(os.path.getmtime(f) for f in files if os.path.exists(f))
 
@@ -29,8 +30,14 @@ def build_library(force: bool = False, verbose: bool = False) -> str:
            "-shared", "-Xcompiler", "-fPIC", "--threads", "4", "-cudart", "static"]
     if verbose:
         cmd += ["-Xptxas", "-v"]
-    cmd += [os.path.join(CSRC, s) for s in SOURCES] + ["-o", OUT]
-    subprocess.check_call(cmd)
+    # one build at a time, and a half-written library never carries the final name
+    with open(OUT + ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if not force and os.path.exists(OUT) and os.path.getmtime(OUT) >= _newest_source():
+            return OUT
+        part = OUT + ".part"
+        subprocess.check_call(cmd + [os.path.join(CSRC, s) for s in SOURCES] + ["-o", part], stdout=sys.stderr)
+        os.replace(part, OUT)
     return OUT
 
 

@@ -60,11 +60,13 @@ struct RowsNormArgs {
     const float* w_post;
     float scalar;
     const float* w_norm;
-    const uint16_t* embed;   // [V, H] BF16 embedding table, or null
+    const void* embed;       // [V, H] embedding table (BF16 or f32, the type of x), or null
     const uint32_t* tokens;  // [B]
     float embed_scale;
     float eps;
-    uint16_t* x;             // [B, H] BF16 activations for the next projection
+    void* x;                 // [B, H] activations for the next projection, BF16 or f32, or null
+    float* x_f32;            // [B, H] the same unrounded, or null (token shift)
+    int norm_n;              // values of a row that count for the means (rows may end in zero padding); 0: H
     PeerExchange px;         // px.tp > 1: `raw` is the local gather buffer; wait for every rank's push first
 };
 
@@ -88,14 +90,22 @@ DEVINL float4 sum_splits4(const float* base, size_t split_stride, int splits) {
     return t;
 }
 
+DEVINL void store_x4(uint16_t* p, float4 v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(f32_to_bf16_bits(v.x) | (f32_to_bf16_bits(v.y) << 16),
+                                              f32_to_bf16_bits(v.z) | (f32_to_bf16_bits(v.w) << 16));
+}
+DEVINL void store_x4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+
 // One CTA per row; hidden size a multiple of 4. The row is read once: the pending projection output (its
 // K-split partials added in split order) and the residual stream stay in registers between the two reductions.
+template <typename XT>
 __global__ void __launch_bounds__(kRowsThreads) rows_norm_kernel(const RowsNormArgs a) {
     __shared__ float red[32];
     pdl_wait();
     pdl_launch();
     const int b = blockIdx.x, tid = threadIdx.x, H = a.H, H4 = a.H >> 2;
     const size_t ro = (size_t)b * H;
+    const float norm_n = (float)(a.norm_n ? a.norm_n : H);
     float4 hv[kRowsMaxJ];
     if (a.embed != nullptr) {
         uint32_t tok = a.tokens[b];
@@ -105,9 +115,14 @@ __global__ void __launch_bounds__(kRowsThreads) rows_norm_kernel(const RowsNormA
             const int i4 = tid + j * kRowsThreads;
             hv[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             if (i4 < H4) {
-                const uint2 e = *reinterpret_cast<const uint2*>(a.embed + (size_t)tok * H + 4 * i4);
-                hv[j] = make_float4(bf16lo(e.x) * a.embed_scale, bf16hi(e.x) * a.embed_scale, bf16lo(e.y) * a.embed_scale,
-                                    bf16hi(e.y) * a.embed_scale);
+                if constexpr (sizeof(XT) == 2) {
+                    const uint2 e = *reinterpret_cast<const uint2*>((const uint16_t*)a.embed + (size_t)tok * H + 4 * i4);
+                    hv[j] = make_float4(bf16lo(e.x) * a.embed_scale, bf16hi(e.x) * a.embed_scale, bf16lo(e.y) * a.embed_scale,
+                                        bf16hi(e.y) * a.embed_scale);
+                } else {
+                    const float4 e = *reinterpret_cast<const float4*>((const float*)a.embed + (size_t)tok * H + 4 * i4);
+                    hv[j] = make_float4(e.x * a.embed_scale, e.y * a.embed_scale, e.z * a.embed_scale, e.w * a.embed_scale);
+                }
             }
         }
     } else if (a.raw == nullptr) {
@@ -142,7 +157,7 @@ __global__ void __launch_bounds__(kRowsThreads) rows_norm_kernel(const RowsNormA
             ss[0] += t[j].w * t[j].w;
         }
         block_sum<1>(ss, red);
-        const float r = 1.0f / sqrtf(ss[0] / (float)H + a.eps);
+        const float r = 1.0f / sqrtf(ss[0] / norm_n + a.eps);
 #pragma unroll
         for (int j = 0; j < kRowsMaxJ; ++j) {
             const int i4 = tid + j * kRowsThreads;
@@ -168,16 +183,15 @@ __global__ void __launch_bounds__(kRowsThreads) rows_norm_kernel(const RowsNormA
         }
     }
     block_sum<1>(ss2, red);
-    const float r2 = 1.0f / sqrtf(ss2[0] / (float)H + a.eps);
+    const float r2 = 1.0f / sqrtf(ss2[0] / norm_n + a.eps);
 #pragma unroll
     for (int j = 0; j < kRowsMaxJ; ++j) {
         const int i4 = tid + j * kRowsThreads;
         if (i4 < H4) {
             const float4 w = *reinterpret_cast<const float4*>(a.w_norm + 4 * i4);
-            uint2 o;
-            o.x = f32_to_bf16_bits(hv[j].x * r2 * w.x) | (f32_to_bf16_bits(hv[j].y * r2 * w.y) << 16);
-            o.y = f32_to_bf16_bits(hv[j].z * r2 * w.z) | (f32_to_bf16_bits(hv[j].w * r2 * w.w) << 16);
-            *reinterpret_cast<uint2*>(a.x + ro + 4 * i4) = o;
+            const float4 n = make_float4(hv[j].x * r2 * w.x, hv[j].y * r2 * w.y, hv[j].z * r2 * w.z, hv[j].w * r2 * w.w);
+            if (a.x_f32) *reinterpret_cast<float4*>(a.x_f32 + ro + 4 * i4) = n;
+            if (a.x) store_x4((XT*)a.x + ro + 4 * i4, n);
         }
     }
 }
@@ -352,9 +366,9 @@ __global__ void pool_fill_kernel(uint4* __restrict__ pool, size_t n16, uint32_t 
     }
 }
 
-// x[b, i] = bf16(gelu_tanh(sum_s gu[s, b, i]) * sum_s gu[s, b, I + i]); grid (ceil(I / 256), B)
+// x[b, i] = bf16(act(sum_s gu[s, b, i]) * sum_s gu[s, b, I + i]), act = tanh-GELU or SiLU; grid (ceil(I / 1024), B)
 __global__ void __launch_bounds__(kRowsThreads)
-geglu_rows_kernel(int B, int I, const float* gu, int splits, uint16_t* x) {
+geglu_rows_kernel(int B, int I, const float* gu, int splits, uint16_t* x, int act) {
     pdl_wait();
     pdl_launch();
     const int b = blockIdx.y, i = (blockIdx.x * kRowsThreads + threadIdx.x) * 4;          // I is a multiple of 4
@@ -363,10 +377,8 @@ geglu_rows_kernel(int B, int I, const float* gu, int splits, uint16_t* x) {
     const float* row = gu + (size_t)b * (2 * (size_t)I);
     const float4 g = sum_splits4(row + i, split_stride, splits);
     const float4 u = sum_splits4(row + I + i, split_stride, splits);
-    uint2 o;
-    o.x = f32_to_bf16_bits(gelu_mul(g.x, u.x)) | (f32_to_bf16_bits(gelu_mul(g.y, u.y)) << 16);
-    o.y = f32_to_bf16_bits(gelu_mul(g.z, u.z)) | (f32_to_bf16_bits(gelu_mul(g.w, u.w)) << 16);
-    *reinterpret_cast<uint2*>(x + (size_t)b * I + i) = o;
+    store_x4(x + (size_t)b * I + i, make_float4(glu_mul(act, g.x, u.x), glu_mul(act, g.y, u.y), glu_mul(act, g.z, u.z),
+                                               glu_mul(act, g.w, u.w)));
 }
 
 }  // namespace oxg4

@@ -8,10 +8,13 @@
 //                        (or h = embedding row * sqrt(H) for the first layer), store h once, then
 //                        x = bf16(rmsnorm(h, w_norm))
 //             PRO_PLAIN: x = bf16(in)
+//             PRO_SHIFT: PRO_NORM, then one input per segment of output rows: n + (previous token's n - n) * mu_s,
+//                        n = rmsnorm(h, w_norm) in f32 (token shift of a time-mixing layer; one row)
+//             PRO_GNORM: x = bf16(in / rms(its group) * w * act(gate)), each factor optional (one row)
 //   body      out[n] = sum_k x[k] * W[n,k], f32 accumulate, 16-byte coalesced streaming loads,
 //             warp-shuffle reductions
 //   epilogue  EPI_STORE : out[b, n]
-//             EPI_GATEUP: out[b, i] = gelu_tanh(gate_i . x) * (up_i . x)
+//             EPI_GATEUP: out[b, i] = act(gate_i . x) * (up_i . x), act = tanh-GELU or SiLU
 //             EPI_LOGITS: optional logits store + running arg-max with repetition penalty
 //
 // Work split (EPI_STORE / EPI_GATEUP). Every CTA owns a contiguous block of output rows (for
@@ -27,7 +30,7 @@
 
 namespace oxg4 {
 
-enum { PRO_PLAIN = 0, PRO_NORM = 1 };
+enum { PRO_PLAIN = 0, PRO_NORM = 1, PRO_SHIFT = 2, PRO_GNORM = 3 };
 enum { EPI_STORE = 0, EPI_GATEUP = 1, EPI_LOGITS = 2 };
 
 constexpr int kGemvThreads = 512;
@@ -45,8 +48,20 @@ struct GemvArgs {
     int slots;               // most pieces a row is cut into inside one CTA
     int B;                   // activation rows in the step
     int bpp;                 // activation rows per pass (tensor-core kernel: grid.y = ceil(B / bpp))
-    // PRO_PLAIN
-    const float* in;         // [B, K]
+    // PRO_PLAIN, PRO_GNORM
+    const float* in;         // [B, K]; with input segments [nseg, B, K]
+    // input segments: output rows [s * seg_rows, (s + 1) * seg_rows) multiply input s (nseg = 0: one input)
+    int nseg, seg_rows;
+    // PRO_SHIFT
+    const float* mu;         // [nseg, K]
+    const float* shift_state;  // [K] normed input of the previous token (ignored at position 0)
+    const int32_t* pos;      // [1]
+    float* x_f32;            // [K] receives this token's normed input (block 0)
+    // PRO_GNORM
+    int gn_n, gn_group;      // values and group size (0: no norm); x is zero from gn_n to K
+    const float* gn_w;       // or null
+    const float* gn_gate;    // or null
+    int act;                 // PRO_GNORM: gate activation; EPI_GATEUP: activation of the gate projection
     // PRO_NORM (K == hidden size)
     const float* h_in;       // [B, K] residual stream before the pending update (unused with embed)
     float* h_out;            // [B, K] residual stream after it (written by block 0)
@@ -58,6 +73,7 @@ struct GemvArgs {
     const uint32_t* tokens;  // [B]
     float embed_scale;
     float eps;
+    int norm_n;              // values of a row that count for the PRO_NORM means (rows may end in zero padding); 0: K
     // weights of later kernels to pull into L2 while this kernel runs (each CTA takes a slice)
     const void* pf_ptr[2];
     unsigned long long pf_bytes[2];
@@ -134,8 +150,10 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
     constexpr int STEP = 32 * EPL;                     // elements per chunk
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int K = a.K;
-    XT* xs = reinterpret_cast<XT*>(smem_raw);                                        // [NB][K]
-    float* red = reinterpret_cast<float*>(smem_raw + (size_t)NB * K * sizeof(XT));   // [NB*32]
+    constexpr bool SEGS = (PRO == PRO_SHIFT || PRO == PRO_PLAIN) && EPI == EPI_STORE;  // may have several inputs
+    const int nseg = SEGS ? max(1, a.nseg) : 1;
+    XT* xs = reinterpret_cast<XT*>(smem_raw);                                        // [nseg][NB][K]
+    float* red = reinterpret_cast<float*>(smem_raw + (size_t)nseg * NB * K * sizeof(XT));   // [NB*32]
     float* pieces = red + NB * 32;                     // [rows_cta][slots][NB] / Cand scratch
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int b0 = blockIdx.y * NB;
@@ -210,7 +228,7 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
     }
     // norm weights are model constants: fetch them before waiting on the previous kernel
     float wpost[kSimtMaxJ], wnorm[kSimtMaxJ];
-    if constexpr (PRO == PRO_NORM) {
+    if constexpr (PRO == PRO_NORM || PRO == PRO_SHIFT) {
 #pragma unroll
         for (int j = 0; j < kSimtMaxJ; ++j) {
             const int i = tid + j * kSimtThreads;
@@ -224,11 +242,38 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
 
     // ---- prologue: build x[nb][K] in shared memory ----
     if constexpr (PRO == PRO_PLAIN) {
-        for (int b = 0; b < nb; ++b)
-            for (int i = tid; i < K; i += kSimtThreads)
-                T::store_x(xs + (size_t)b * K + i, a.in[(size_t)(b0 + b) * K + i]);
+        for (int sg = 0; sg < nseg; ++sg)
+            for (int b = 0; b < nb; ++b)
+                for (int i = tid; i < K; i += kSimtThreads)
+                    T::store_x(xs + ((size_t)sg * NB + b) * K + i, a.in[((size_t)sg * a.B + b0 + b) * K + i]);
+    } else if constexpr (PRO == PRO_GNORM) {
+        auto put = [&](int i, float v) {
+            if (a.gn_w) v *= a.gn_w[i];
+            if (a.gn_gate) v *= a.act == ACT_SILU ? silu(a.gn_gate[i]) : sigmoid(a.gn_gate[i]);
+            T::store_x(xs + i, v);
+        };
+        if (a.gn_group == 0 || a.gn_group == a.gn_n) {
+            float r = 1.0f;
+            if (a.gn_group) {
+                float ss[1] = {0.0f};
+                for (int i = tid; i < a.gn_n; i += kSimtThreads) ss[0] += a.in[i] * a.in[i];
+                block_sum<1>(ss, red);
+                r = 1.0f / sqrtf(ss[0] / (float)a.gn_n + a.eps);
+            }
+            for (int i = tid; i < a.gn_n; i += kSimtThreads) put(i, a.in[i] * r);
+        } else {
+            for (int g = warp; g < a.gn_n / a.gn_group; g += kSimtWarps) {
+                const float* src = a.in + (size_t)g * a.gn_group;
+                float s = 0.0f;
+                for (int i = lane; i < a.gn_group; i += 32) s += src[i] * src[i];
+                s = 1.0f / sqrtf(warp_sum(s) / (float)a.gn_group + a.eps);
+                for (int i = lane; i < a.gn_group; i += 32) put(g * a.gn_group + i, src[i] * s);
+            }
+        }
+        for (int i = a.gn_n + tid; i < K; i += kSimtThreads) T::store_x(xs + i, 0.0f);
     } else {
         const bool writer = (blockIdx.x == 0);
+        const float norm_n = (float)(a.norm_n ? a.norm_n : K);
         for (int b = 0; b < nb; ++b) {
             float hv[kSimtMaxJ];
             float ss[1];
@@ -259,7 +304,7 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
                     ss[0] += t[j] * t[j];
                 }
                 block_sum<1>(ss, red);
-                const float r = 1.0f / sqrtf(ss[0] / (float)K + a.eps);
+                const float r = 1.0f / sqrtf(ss[0] / norm_n + a.eps);
 #pragma unroll
                 for (int j = 0; j < kSimtMaxJ; ++j) hv[j] = (hv[j] + t[j] * r * wpost[j]) * a.scalar;
             }
@@ -273,17 +318,31 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
                 }
             }
             block_sum<1>(ss, red);
-            const float r2 = 1.0f / sqrtf(ss[0] / (float)K + a.eps);
+            const float r2 = 1.0f / sqrtf(ss[0] / norm_n + a.eps);
+            if constexpr (PRO == PRO_SHIFT) {
+                const bool first = a.pos[0] == 0;
 #pragma unroll
-            for (int j = 0; j < kSimtMaxJ; ++j) {
-                const int i = tid + j * kSimtThreads;
-                if (i < K) T::store_x(xs + (size_t)b * K + i, hv[j] * r2 * wnorm[j]);
+                for (int j = 0; j < kSimtMaxJ; ++j) {
+                    const int i = tid + j * kSimtThreads;
+                    if (i >= K) continue;
+                    const float c = hv[j] * r2 * wnorm[j], p = first ? 0.0f : a.shift_state[i];
+                    if (writer) a.x_f32[i] = c;
+                    for (int sg = 0; sg < nseg; ++sg)
+                        T::store_x(xs + (size_t)sg * K + i, c + (p - c) * a.mu[(size_t)sg * K + i]);
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < kSimtMaxJ; ++j) {
+                    const int i = tid + j * kSimtThreads;
+                    if (i < K) T::store_x(xs + (size_t)b * K + i, hv[j] * r2 * wnorm[j]);
+                }
             }
         }
     }
     // rows of a partial batch chunk that do not exist read zeros
-    for (int b = nb; b < NB; ++b)
-        for (int i = tid; i < K; i += kSimtThreads) xs[(size_t)b * K + i] = (XT)0;
+    for (int sg = 0; sg < nseg; ++sg)
+        for (int b = nb; b < NB; ++b)
+            for (int i = tid; i < K; i += kSimtThreads) xs[((size_t)sg * NB + b) * K + i] = (XT)0;
     __syncthreads();
     pdl_launch();
     stamp(a.ts, 2);
@@ -302,6 +361,10 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
             const int nfull = has_tail ? ncs - 1 : ncs;
             const WT* p = row_ptr(row_first + rl) + (size_t)cc * STEP + lane * EPL;
             int k = cc * STEP + lane * EPL;
+            const XT* xr = xs;                         // the input of this row's segment
+            if constexpr (SEGS) {
+                if (nseg > 1) xr = xs + (size_t)((row_first + rl) / a.seg_rows) * NB * K;
+            }
             float acc[NB];
 #pragma unroll
             for (int b = 0; b < NB; ++b) acc[b] = 0.0f;
@@ -311,7 +374,7 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
 #pragma unroll
                 for (int q = 0; q < 8; ++q) w[q] = ldg_stream16(p + q * STEP);
 #pragma unroll
-                for (int q = 0; q < 8; ++q) fma16<WT, NB>(acc, w[q], xs, K, k + q * STEP);
+                for (int q = 0; q < 8; ++q) fma16<WT, NB>(acc, w[q], xr, K, k + q * STEP);
                 p += 8 * STEP;
                 k += 8 * STEP;
             }
@@ -320,15 +383,15 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
 #pragma unroll
                 for (int q = 0; q < 4; ++q) w[q] = ldg_stream16(p + q * STEP);
 #pragma unroll
-                for (int q = 0; q < 4; ++q) fma16<WT, NB>(acc, w[q], xs, K, k + q * STEP);
+                for (int q = 0; q < 4; ++q) fma16<WT, NB>(acc, w[q], xr, K, k + q * STEP);
                 p += 4 * STEP;
                 k += 4 * STEP;
                 j += 4;
             }
             if (j + 2 <= nfull) {
                 uint4 w0 = ldg_stream16(p), w1 = ldg_stream16(p + STEP);
-                fma16<WT, NB>(acc, w0, xs, K, k);
-                fma16<WT, NB>(acc, w1, xs, K, k + STEP);
+                fma16<WT, NB>(acc, w0, xr, K, k);
+                fma16<WT, NB>(acc, w1, xr, K, k + STEP);
                 p += 2 * STEP;
                 k += 2 * STEP;
                 j += 2;
@@ -336,7 +399,7 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
             for (; j < ncs; ++j) {
                 if (k < K) {
                     uint4 w0 = ldg_stream16(p);
-                    fma16<WT, NB>(acc, w0, xs, K, k);
+                    fma16<WT, NB>(acc, w0, xr, K, k);
                 }
                 p += STEP;
                 k += STEP;
@@ -369,7 +432,7 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
             for (int idx = tid; idx < pairs * nb; idx += kSimtThreads) {
                 const int pl = idx % pairs, b = idx / pairs;
                 const float g = row_total(2 * pl, b), u = row_total(2 * pl + 1, b);
-                a.out[(size_t)(b0 + b) * (a.N / 2) + row_first / 2 + pl] = gelu_mul(g, u);
+                a.out[(size_t)(b0 + b) * (a.N / 2) + row_first / 2 + pl] = glu_mul(a.act, g, u);
             }
         }
     } else {

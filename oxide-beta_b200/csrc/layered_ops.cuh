@@ -1,0 +1,621 @@
+// Kernels of models whose layers are listed one by one (csrc/layered.inl): recurrent mixers with a matrix state per
+// head (lightning attention, RWKV-style time mixing), token shift, grouped output norms with a gate, and multi-head
+// latent attention over a paged cache of latents. They sit around the projections of gemv.cuh (one row, or f32
+// weights) and tc_gemm.cuh (BF16 weights, many rows); the sandwich norms and the residual stream are those of
+// rows_norm_kernel / the PRO_NORM prologue.
+//
+// Everything here computes in f32. Activations are rounded to BF16 only where they become the operand of a
+// BF16 projection. "Split input": the consumer of a tcgen05 projection adds its K-split partials itself, in split
+// order, so every reader takes (pointer, number of splits, distance between splits).
+#pragma once
+#include "common.cuh"
+#include "gemv.cuh"
+
+namespace oxg4 {
+
+struct SplitIn {             // [splits][rows][ld] f32, columns start at `col`
+    const float* p;
+    int splits;
+    size_t stride;           // elements between two splits
+    int ld;
+    DEVINL float at(int row, int col) const {
+        const float* q = p + (size_t)row * ld + col;
+        float t = q[0];
+        for (int s = 1; s < splits; ++s) t += q[(size_t)s * stride];
+        return t;
+    }
+};
+
+// The rows of a pass as runs of consecutive tokens of one sequence (a decode step: one run of one token per
+// sequence) and their positions.
+struct RunRows {
+    const int32_t* row0;     // [runs] first row
+    const int32_t* n;        // [runs] rows
+    const int32_t* pos;      // [R]
+    const int32_t* seq;      // [R] or null: row r is sequence r
+    const uint32_t* tok;     // [R]; kInactiveToken rows are left out
+    DEVINL int seq_of(int row) const { return seq ? seq[row] : row; }
+};
+
+template <typename XT> DEVINL void store_act(XT* p, float v);
+template <> DEVINL void store_act<float>(float* p, float v) { *p = v; }
+template <> DEVINL void store_act<uint16_t>(uint16_t* p, float v) { *p = (uint16_t)f32_to_bf16_bits(v); }
+
+// ---- token shift --------------------------------------------------------------------------------------------
+// mix[s][r] = h_r + (h_(r-1) - h_r) * mu_s for S mixes; h_(r-1) is the previous row of the run, the sequence's shift
+// state for the first row of a run, zero at position 0. grid (R), rows of H values (a multiple of 4).
+template <typename XT>
+__global__ void __launch_bounds__(256)
+shift_mix_kernel(int R, int H, int S, const float* h, const float* state, const float* mu, RunRows rows, XT* mix) {
+    pdl_wait();
+    pdl_launch();
+    const int r = blockIdx.x, s_ = rows.seq_of(r);
+    const bool first = rows.seq == nullptr || r == 0 || rows.seq[r - 1] != s_;
+    const float* prev = first ? state + (size_t)s_ * H : h + (size_t)(r - 1) * H;
+    const bool zero = first && rows.pos[r] == 0;
+    for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
+        const float4 c = *reinterpret_cast<const float4*>(h + (size_t)r * H + i);
+        float4 p = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (!zero) p = *reinterpret_cast<const float4*>(prev + i);
+        for (int s = 0; s < S; ++s) {
+            const float4 m = *reinterpret_cast<const float4*>(mu + (size_t)s * H + i);
+            const float a = c.x + (p.x - c.x) * m.x, b = c.y + (p.y - c.y) * m.y, d = c.z + (p.z - c.z) * m.z,
+                        e = c.w + (p.w - c.w) * m.w;
+            XT* o = mix + ((size_t)s * R + r) * H + i;
+            if constexpr (sizeof(XT) == 2) {
+                *reinterpret_cast<uint2*>(o) = make_uint2(f32_to_bf16_bits(a) | (f32_to_bf16_bits(b) << 16),
+                                                          f32_to_bf16_bits(d) | (f32_to_bf16_bits(e) << 16));
+            } else {
+                *reinterpret_cast<float4*>(o) = make_float4(a, b, d, e);
+            }
+        }
+    }
+}
+
+// ---- per-channel decay of the time mixing -------------------------------------------------------------------
+// w[n] = exp(-exp(W2[n, :] . tanh(low) + w0[n]))
+template <typename WT>
+DEVINL float channel_decay(const WT* w2_row, const float* tanh_low, int rank, float w0) {
+    float t = w0;
+    for (int j = 0; j < rank; ++j) t = fmaf(WTraits<WT>::elem(w2_row, j), tanh_low[j], t);
+    return expf(-expf(t));
+}
+
+constexpr int kDecayRows = 8;
+// out[r, n] for R rows and N channels; grid (ceil(N / 256), ceil(R / 8)), dynamic shared memory 8 * rank floats
+template <typename WT>
+__global__ void __launch_bounds__(256)
+wkv_decay_kernel(int R, int N, int rank, SplitIn low, int col, const WT* w2, const float* w0, float* out) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* th = reinterpret_cast<float*>(smem_raw);
+    pdl_wait();
+    pdl_launch();
+    const int r0 = blockIdx.y * kDecayRows, nr = min(kDecayRows, R - r0);
+    for (int i = threadIdx.x; i < nr * rank; i += blockDim.x) th[i] = tanhf(low.at(r0 + i / rank, col + i % rank));
+    __syncthreads();
+    const int n = blockIdx.x * 256 + threadIdx.x;
+    if (n >= N) return;
+    float t[kDecayRows];
+#pragma unroll
+    for (int q = 0; q < kDecayRows; ++q) t[q] = w0[n];
+    for (int j = 0; j < rank; ++j) {
+        const float w = WTraits<WT>::elem(w2, (size_t)n * rank + j);
+#pragma unroll
+        for (int q = 0; q < kDecayRows; ++q)
+            if (q < nr) t[q] = fmaf(w, th[q * rank + j], t[q]);
+    }
+#pragma unroll
+    for (int q = 0; q < kDecayRows; ++q)
+        if (q < nr) out[(size_t)(r0 + q) * N + n] = expf(-expf(t[q]));
+}
+
+// ---- recurrence ---------------------------------------------------------------------------------------------
+// Per head a state S [dim, vdim] in f32, walked token by token:
+//   REC_LIGHTNING  q, k, v = silu(.);  S = decay_h S + k v^T;  o = S^T q
+//   REC_WKV        o = (S + diag(u) k v^T)^T r;  S = diag(w) S + k v^T, w per token and key channel
+// The bonus term is v * sum_k r_k u_k k_k, one scalar per token and head.
+// Grid (heads, slices of vdim, runs). A thread owns KPT consecutive key channels of one value column; the KS threads
+// that share a column are neighbouring lanes. Tokens are staged in shared memory in tiles, activations applied on
+// the way; the dot products of 8 tokens are reduced across the KS lanes together.
+// State in memory: [sequence][head][vdim][dim]. At position 0 the state starts at zero whatever the memory holds.
+enum { REC_LIGHTNING = 0, REC_WKV = 1 };
+constexpr int kRecThreads = 256;
+constexpr int kRecTile = 16;             // tokens staged at a time
+
+struct RecurArgs {
+    SplitIn in;                          // fused input projection
+    int c_q, c_k, c_v;                   // first columns of q (r), k and v, head by head
+    int heads, dim, vdim;
+    const float* decay;                  // LIGHTNING: [heads]
+    const float* u;                      // WKV: [heads, dim]
+    const float* w;                      // WKV: [R, heads * dim] decays, or null: computed here (runs of one token)
+    int c_low, rank;                     //   from the low-rank columns
+    const void* w2;                      //   [heads * dim, rank]
+    const float* w0;                     //   [heads * dim]
+    float* state;
+    RunRows rows;
+    float* out;                          // [R, ld_out]
+    int ld_out;
+    // token-shift state: the normed input of the run's last row, copied by one CTA per run
+    const float* shift_src;              // [R, shift_n] or null
+    float* shift_dst;                    // [sequences, shift_n]
+    int shift_n;
+};
+
+template <int KIND, typename WT, int KS, int KPT>
+__global__ void __launch_bounds__(kRecThreads) recur_kernel(const RecurArgs a) {
+    constexpr int DP = KS * KPT;         // key channels, padded
+    constexpr int VS = kRecThreads / KS; // value columns of this CTA
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* sq = reinterpret_cast<float*>(smem_raw);          // [tile][DP]
+    float* sk = sq + kRecTile * DP;
+    float* sw = sk + kRecTile * DP;                          // WKV only
+    float* sv = sw + (KIND == REC_WKV ? kRecTile * DP : 0);  // [tile][VS]
+    float* sb = sv + kRecTile * VS;                          // [tile] bonus (WKV)
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int hd = blockIdx.x, v0 = blockIdx.y * VS, run = blockIdx.z;
+    const int ks = tid % KS, vc = tid / KS, v = v0 + vc;
+    pdl_wait();
+    pdl_launch();
+    const int row0 = a.rows.row0[run], n = a.rows.n[run];
+    if (a.rows.tok[row0] == kInactiveToken) return;
+    const int seq = a.rows.seq_of(row0);
+    const bool fresh = a.rows.pos[row0] == 0;
+    if (a.shift_src != nullptr && hd == 0 && blockIdx.y == 0)
+        for (int i = tid; i < a.shift_n; i += kRecThreads)
+            a.shift_dst[(size_t)seq * a.shift_n + i] = a.shift_src[(size_t)(row0 + n - 1) * a.shift_n + i];
+    float* st = a.state + (((size_t)seq * a.heads + hd) * a.vdim + v) * a.dim;
+    const bool have_v = v < a.vdim;
+    float S[KPT];
+#pragma unroll
+    for (int i = 0; i < KPT; ++i) {
+        const int k = ks * KPT + i;
+        S[i] = (!fresh && have_v && k < a.dim) ? st[k] : 0.0f;
+    }
+    const float dh = KIND == REC_LIGHTNING ? a.decay[hd] : 0.0f;
+    const int hk = hd * a.dim, hv = hd * a.vdim;
+    for (int t0 = 0; t0 < n; t0 += kRecTile) {
+        const int nt = min(kRecTile, n - t0);
+        __syncthreads();
+        for (int i = tid; i < kRecTile * DP; i += kRecThreads) {
+            const int t = i / DP, k = i % DP;
+            float q = 0.0f, kk = 0.0f, w = 0.0f;
+            if (t < nt && k < a.dim) {
+                const int r = row0 + t0 + t;
+                q = a.in.at(r, a.c_q + hk + k);
+                kk = a.in.at(r, a.c_k + hk + k);
+                if constexpr (KIND == REC_LIGHTNING) {
+                    q = silu(q);
+                    kk = silu(kk);
+                } else if (a.w != nullptr) {
+                    w = a.w[(size_t)r * a.heads * a.dim + hk + k];
+                }
+            }
+            sq[i] = q;
+            sk[i] = kk;
+            if constexpr (KIND == REC_WKV) sw[i] = w;
+        }
+        for (int i = tid; i < kRecTile * VS; i += kRecThreads) {
+            const int t = i / VS, c = v0 + i % VS;
+            float x = 0.0f;
+            if (t < nt && c < a.vdim) {
+                x = a.in.at(row0 + t0 + t, a.c_v + hv + c);
+                if constexpr (KIND == REC_LIGHTNING) x = silu(x);
+            }
+            sv[i] = x;
+        }
+        if constexpr (KIND == REC_WKV) {
+            if (a.w == nullptr) {                            // one-token run: decay of this head's channels
+                float* th = sb + kRecTile;                   // [rank]
+                for (int j = tid; j < a.rank; j += kRecThreads) th[j] = tanhf(a.in.at(row0, a.c_low + j));
+                __syncthreads();
+                for (int k = tid; k < a.dim; k += kRecThreads)
+                    sw[k] = channel_decay((const WT*)a.w2 + (size_t)(hk + k) * a.rank, th, a.rank, a.w0[hk + k]);
+            }
+            __syncthreads();
+            for (int t = warp; t < nt; t += kRecThreads / 32) {
+                float b = 0.0f;
+                for (int k = lane; k < a.dim; k += 32) b += sq[t * DP + k] * a.u[hk + k] * sk[t * DP + k];
+                b = warp_sum(b);
+                if (lane == 0) sb[t] = b;
+            }
+        }
+        __syncthreads();
+        for (int tb = 0; tb < nt; tb += 8) {
+            float acc[8];
+#pragma unroll
+            for (int t = 0; t < 8; ++t) {
+                acc[t] = 0.0f;
+                if (tb + t >= nt) continue;
+                const float* q = sq + (tb + t) * DP + ks * KPT;
+                const float* k = sk + (tb + t) * DP + ks * KPT;
+                const float* w = sw + (tb + t) * DP + ks * KPT;
+                const float x = sv[(tb + t) * VS + vc];
+                float s = 0.0f;
+#pragma unroll
+                for (int i = 0; i < KPT; i += 4) {
+                    const float4 q4 = *reinterpret_cast<const float4*>(q + i), k4 = *reinterpret_cast<const float4*>(k + i);
+                    if constexpr (KIND == REC_LIGHTNING) {
+                        S[i] = fmaf(dh, S[i], k4.x * x); s = fmaf(q4.x, S[i], s);
+                        S[i + 1] = fmaf(dh, S[i + 1], k4.y * x); s = fmaf(q4.y, S[i + 1], s);
+                        S[i + 2] = fmaf(dh, S[i + 2], k4.z * x); s = fmaf(q4.z, S[i + 2], s);
+                        S[i + 3] = fmaf(dh, S[i + 3], k4.w * x); s = fmaf(q4.w, S[i + 3], s);
+                    } else {
+                        const float4 w4 = *reinterpret_cast<const float4*>(w + i);
+                        s = fmaf(q4.x, S[i], s); S[i] = fmaf(w4.x, S[i], k4.x * x);
+                        s = fmaf(q4.y, S[i + 1], s); S[i + 1] = fmaf(w4.y, S[i + 1], k4.y * x);
+                        s = fmaf(q4.z, S[i + 2], s); S[i + 2] = fmaf(w4.z, S[i + 2], k4.z * x);
+                        s = fmaf(q4.w, S[i + 3], s); S[i + 3] = fmaf(w4.w, S[i + 3], k4.w * x);
+                    }
+                }
+                acc[t] = s;
+            }
+#pragma unroll
+            for (int t = 0; t < 8; ++t) {
+#pragma unroll
+                for (int o = KS / 2; o > 0; o >>= 1) acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], o);
+            }
+            // lane ks of a column stores tokens ks, ks + KS, ...
+            if (have_v) {
+#pragma unroll
+                for (int t = 0; t < 8; ++t)
+                    if ((t % KS) == ks && tb + t < nt) {
+                        float o = acc[t];
+                        if constexpr (KIND == REC_WKV) o = fmaf(sb[tb + t], sv[(tb + t) * VS + vc], o);
+                        a.out[(size_t)(row0 + t0 + tb + t) * a.ld_out + hv + v] = o;
+                    }
+            }
+        }
+    }
+    if (have_v) {
+#pragma unroll
+        for (int i = 0; i < KPT; ++i) {
+            const int k = ks * KPT + i;
+            if (k < a.dim) st[k] = S[i];
+        }
+    }
+}
+
+// ---- output norm and gate of a mixer ------------------------------------------------------------------------
+// x[r, j] = o[r, j] / rms(group of j) * w[j] * act(gate[r, j]); group = 0: no norm, w = null: no weight. The values lie
+// in heads of `hs` columns that start `hs_ld` apart in `o`. One CTA per row, `n` values, padded with zeros to `ld_x`.
+struct GroupNormArgs {
+    SplitIn o;
+    int hs, hs_ld;
+    int n, group;
+    const float* w;
+    SplitIn gate;
+    int c_gate, act;                     // act: ACT_NONE without a gate
+    float eps;
+};
+
+template <typename XT>
+__global__ void __launch_bounds__(256) group_norm_rows_kernel(const GroupNormArgs a, XT* x, int ld_x) {
+    __shared__ float red[32];
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* v = reinterpret_cast<float*>(smem_raw);           // [n]
+    pdl_wait();
+    pdl_launch();
+    const int r = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    float ss[1] = {0.0f};
+    for (int j = tid; j < a.n; j += blockDim.x) {
+        const float t = a.o.at(r, (j / a.hs) * a.hs_ld + j % a.hs);
+        v[j] = t;
+        ss[0] += t * t;
+    }
+    float whole = 1.0f;
+    if (a.group == a.n) {
+        block_sum<1>(ss, red);
+        whole = 1.0f / sqrtf(ss[0] / (float)a.n + a.eps);
+    } else if (a.group > 0) {
+        __syncthreads();
+        for (int g = warp; g < a.n / a.group; g += 8) {
+            float s = 0.0f;
+            for (int j = lane; j < a.group; j += 32) s += v[g * a.group + j] * v[g * a.group + j];
+            s = 1.0f / sqrtf(warp_sum(s) / (float)a.group + a.eps);
+            for (int j = lane; j < a.group; j += 32) v[g * a.group + j] *= s;
+        }
+    }
+    __syncthreads();
+    for (int j = tid; j < ld_x; j += blockDim.x) {
+        float t = 0.0f;
+        if (j < a.n) {
+            t = v[j] * whole;
+            if (a.w) t *= a.w[j];
+            if (a.act == ACT_SIGMOID) t *= sigmoid(a.gate.at(r, a.c_gate + j));
+            else if (a.act == ACT_SILU) t *= silu(a.gate.at(r, a.c_gate + j));
+        }
+        store_act(x + (size_t)r * ld_x + j, t);
+    }
+}
+
+// ---- latent attention ---------------------------------------------------------------------------------------
+// The cache row of a token is [latent (rank) | rotated key part (rot)], padded with zeros to `ld` elements; slot =
+// position, pages of `page_tokens` rows. Scores and values are taken in latent space: the query is carried through
+// W_uk ("absorbed") and the attention output through W_uv, so a cached token costs ld elements whatever the heads.
+struct LatentCache {
+    void* pool;                          // [pages][page_tokens][ld]
+    const int32_t* page_table;           // [sequences, pages_per_seq]
+    int pages_per_seq, page_tokens, ld;
+    DEVINL size_t row(int seq, int pos) const {
+        const int page = page_table[(size_t)seq * pages_per_seq + pos / page_tokens];
+        return ((size_t)page * page_tokens + pos % page_tokens) * ld;
+    }
+};
+
+struct LatentArgs {
+    SplitIn in;                          // fused input projection
+    int c_dq, c_dkv;
+    int heads, dim, rot, rot_dims, vdim, rank, q_rank;
+    const float *dq_norm, *dkv_norm, *inv_freq;
+    float eps, scale;
+    RunRows rows;
+    LatentCache cache;
+};
+
+// rotation of the pair (u, v) = (x[2i], x[2i+1]) at `pos`
+DEVINL void rotate_pair(float& u, float& v, int pos, float inv_freq) {
+    float s, c;
+    sincosf((float)pos * inv_freq, &s, &c);
+    const float x = u * c - v * s;
+    v = v * c + u * s;
+    u = x;
+}
+
+// norms the latent of row r, rotates the shared key part and stores both in the cache; whole CTA
+template <typename KT>
+DEVINL void latent_append(const LatentArgs& a, int r, float* red) {
+    const int tid = threadIdx.x, nth = blockDim.x;
+    float ss[1] = {0.0f};
+    for (int j = tid; j < a.rank; j += nth) {
+        const float t = a.in.at(r, a.c_dkv + j);
+        ss[0] += t * t;
+    }
+    block_sum<1>(ss, red);
+    const float s = 1.0f / sqrtf(ss[0] / (float)a.rank + a.eps);
+    const int pos = a.rows.pos[r];
+    KT* dst = (KT*)a.cache.pool + a.cache.row(a.rows.seq_of(r), pos);
+    for (int j = tid; j < a.rank; j += nth) store_act(dst + j, a.in.at(r, a.c_dkv + j) * s * a.dkv_norm[j]);
+    for (int i = tid; i < (a.rot + 1) / 2; i += nth) {
+        float u = a.in.at(r, a.c_dkv + a.rank + 2 * i);
+        float v = 2 * i + 1 < a.rot ? a.in.at(r, a.c_dkv + a.rank + 2 * i + 1) : 0.0f;
+        if (2 * i + 1 < a.rot_dims) rotate_pair(u, v, pos, a.inv_freq[i]);
+        store_act(dst + a.rank + 2 * i, u);
+        if (2 * i + 1 < a.rot) store_act(dst + a.rank + 2 * i + 1, v);
+    }
+    for (int j = a.rank + a.rot + tid; j < a.cache.ld; j += nth) store_act(dst + j, 0.0f);
+}
+
+// many rows: x_q = normed query latent (input of W_uq, padded with zeros to ld_x), and the cache append. grid (R)
+template <typename XT, typename KT>
+__global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a, XT* x_q, int ld_x) {
+    __shared__ float red[32];
+    pdl_wait();
+    pdl_launch();
+    const int r = blockIdx.x, tid = threadIdx.x;
+    float ss[1] = {0.0f};
+    for (int j = tid; j < a.q_rank; j += blockDim.x) {
+        const float t = a.in.at(r, a.c_dq + j);
+        ss[0] += t * t;
+    }
+    block_sum<1>(ss, red);
+    const float s = 1.0f / sqrtf(ss[0] / (float)a.q_rank + a.eps);
+    for (int j = tid; j < ld_x; j += blockDim.x)
+        store_act(x_q + (size_t)r * ld_x + j, j < a.q_rank ? a.in.at(r, a.c_dq + j) * s * a.dq_norm[j] : 0.0f);
+    if (a.rows.tok[r] != kInactiveToken) latent_append<KT>(a, r, red);
+}
+
+// Queries in latent space, few rows: q_abs[r, h, :] = q_unrotated . W_uk[h], followed by the rotated part; f32
+// [R, heads, rank + rot]. grid (heads + 1, R, slices of 256 latent columns); the CTAs of x == heads append the token to
+// the cache when `append` is set. dynamic shared memory: dim + rot floats
+template <typename WT, typename KT>
+__global__ void __launch_bounds__(256)
+latent_query_kernel(const LatentArgs a, SplitIn q, const WT* w_uk, float* q_abs, int append) {
+    __shared__ float red[32];
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* sq = reinterpret_cast<float*>(smem_raw);
+    pdl_wait();
+    pdl_launch();
+    const int hd = blockIdx.x, r = blockIdx.y, tid = threadIdx.x;
+    if (a.rows.tok[r] == kInactiveToken) return;
+    if (hd == a.heads) {
+        if (append && blockIdx.z == 0) latent_append<KT>(a, r, red);
+        return;
+    }
+    const int dq = a.dim + a.rot;
+    for (int j = tid; j < dq; j += 256) sq[j] = q.at(r, hd * dq + j);
+    __syncthreads();
+    float* dst = q_abs + ((size_t)r * a.heads + hd) * (a.rank + a.rot);
+    const int n = blockIdx.z * 256 + tid;
+    if (n < a.rank) {
+        float t0 = 0.0f, t1 = 0.0f, t2 = 0.0f, t3 = 0.0f;
+        const size_t base = (size_t)hd * a.dim * a.rank + n;
+        int d = 0;
+        for (; d + 4 <= a.dim; d += 4) {
+            t0 = fmaf(sq[d], WTraits<WT>::elem(w_uk, base + (size_t)d * a.rank), t0);
+            t1 = fmaf(sq[d + 1], WTraits<WT>::elem(w_uk, base + (size_t)(d + 1) * a.rank), t1);
+            t2 = fmaf(sq[d + 2], WTraits<WT>::elem(w_uk, base + (size_t)(d + 2) * a.rank), t2);
+            t3 = fmaf(sq[d + 3], WTraits<WT>::elem(w_uk, base + (size_t)(d + 3) * a.rank), t3);
+        }
+        for (; d < a.dim; ++d) t0 = fmaf(sq[d], WTraits<WT>::elem(w_uk, base + (size_t)d * a.rank), t0);
+        dst[n] = (t0 + t1) + (t2 + t3);
+    }
+    if (blockIdx.z == 0) {
+        const int pos = a.rows.pos[r];
+        for (int i = tid; i < (a.rot + 1) / 2; i += 256) {
+            float u = sq[a.dim + 2 * i], v = 2 * i + 1 < a.rot ? sq[a.dim + 2 * i + 1] : 0.0f;
+            if (2 * i + 1 < a.rot_dims) rotate_pair(u, v, pos, a.inv_freq[i]);
+            dst[a.rank + 2 * i] = u;
+            if (2 * i + 1 < a.rot) dst[a.rank + 2 * i + 1] = v;
+        }
+    }
+}
+
+// many rows: the unrotated query parts as BF16 operands of the per-head products with W_uk^T, [heads][R][ld_u], and the
+// rotated parts in f32, [R, heads, rot]. grid (R)
+__global__ void __launch_bounds__(256)
+latent_split_query_kernel(const LatentArgs a, int R, SplitIn q, uint16_t* x_u, int ld_u, float* q_rot) {
+    pdl_wait();
+    pdl_launch();
+    const int r = blockIdx.x, dq = a.dim + a.rot, pos = a.rows.pos[r];
+    for (int j = threadIdx.x; j < a.heads * ld_u; j += blockDim.x) {
+        const int hd = j / ld_u, d = j % ld_u;
+        store_act(x_u + ((size_t)hd * R + r) * ld_u + d, d < a.dim ? q.at(r, hd * dq + d) : 0.0f);
+    }
+    const int half = (a.rot + 1) / 2;
+    for (int j = threadIdx.x; j < a.heads * half; j += blockDim.x) {
+        const int hd = j / half, i = j % half, c = hd * dq + a.dim + 2 * i;
+        float u = q.at(r, c), v = 2 * i + 1 < a.rot ? q.at(r, c + 1) : 0.0f;
+        if (2 * i + 1 < a.rot_dims) rotate_pair(u, v, pos, a.inv_freq[i]);
+        float* dst = q_rot + ((size_t)r * a.heads + hd) * a.rot + 2 * i;
+        dst[0] = u;
+        if (2 * i + 1 < a.rot) dst[1] = v;
+    }
+}
+
+// Split-KV partials of the latent attention: `o` un-normalised [splits][R * heads][rank], `ml` (running maximum,
+// denominator) [splits][R * heads][2]; a split without a visible key has denominator 0 and leaves `o` unwritten.
+struct LatentPart {
+    float* o;
+    float* ml;
+    int splits;
+    size_t rows;                         // R * heads
+};
+
+// Attention of one (row, head, split) per CTA on the CUDA cores: f32 caches, and BF16 weights with an f32 cache.
+// grid (heads, R, splits), 256 threads, dynamic shared memory (8 + 1) * (rank + rot) + 16 floats. rank <= 32 * RPL.
+template <typename KT, int RPL>
+__global__ void __launch_bounds__(256) latent_attn_kernel(const LatentArgs a, const float* q_abs, LatentPart part) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    const int DK = a.rank + a.rot;
+    float* sq = reinterpret_cast<float*>(smem_raw);          // [DK]
+    float* so = sq + DK;                                     // [8][rank]
+    float* sm = so + 8 * a.rank;                             // [8][2]
+    pdl_wait();
+    pdl_launch();
+    const int hd = blockIdx.x, r = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const size_t pr = (size_t)blockIdx.z * part.rows + (size_t)r * a.heads + hd;
+    if (a.rows.tok[r] == kInactiveToken) return;
+    const int visible = a.rows.pos[r] + 1, seq = a.rows.seq_of(r);
+    const int per = (visible + part.splits - 1) / part.splits;
+    const int p0 = blockIdx.z * per, p1 = min(visible, p0 + per);
+    if (p0 >= p1) {
+        if (tid == 0) { part.ml[2 * pr] = -INFINITY; part.ml[2 * pr + 1] = 0.0f; }
+        return;
+    }
+    const float* q = q_abs + ((size_t)r * a.heads + hd) * DK;
+    for (int j = tid; j < DK; j += 256) sq[j] = q[j];
+    __syncthreads();
+    float m = -INFINITY, l = 0.0f, acc[RPL];
+#pragma unroll
+    for (int i = 0; i < RPL; ++i) acc[i] = 0.0f;
+    for (int p = p0 + warp; p < p1; p += 8) {
+        const KT* row = (const KT*)a.cache.pool + a.cache.row(seq, p);
+        float c[RPL], s = 0.0f;
+#pragma unroll
+        for (int i = 0; i < RPL; ++i) {
+            const int j = lane + 32 * i;
+            c[i] = j < a.rank ? WTraits<KT>::elem(row, j) : 0.0f;
+            if (j < a.rank) s = fmaf(sq[j], c[i], s);
+        }
+        for (int j = a.rank + lane; j < DK; j += 32) s = fmaf(sq[j], WTraits<KT>::elem(row, j), s);
+        s = warp_sum(s) * a.scale;
+        const float m2 = fmaxf(m, s), f = expf(m - m2), e = expf(s - m2);
+        l = l * f + e;
+#pragma unroll
+        for (int i = 0; i < RPL; ++i) acc[i] = fmaf(e, c[i], acc[i] * f);
+        m = m2;
+    }
+#pragma unroll
+    for (int i = 0; i < RPL; ++i)
+        if (lane + 32 * i < a.rank) so[warp * a.rank + lane + 32 * i] = acc[i];
+    if (lane == 0) { sm[2 * warp] = m; sm[2 * warp + 1] = l; }
+    __syncthreads();
+    float M = -INFINITY, L = 0.0f;
+    for (int w = 0; w < 8; ++w) M = fmaxf(M, sm[2 * w]);
+    for (int w = 0; w < 8; ++w) L += sm[2 * w + 1] > 0.0f ? sm[2 * w + 1] * expf(sm[2 * w] - M) : 0.0f;
+    for (int j = tid; j < a.rank; j += 256) {
+        float t = 0.0f;
+        for (int w = 0; w < 8; ++w)
+            if (sm[2 * w + 1] > 0.0f) t += so[w * a.rank + j] * expf(sm[2 * w] - M);
+        part.o[pr * a.rank + j] = t;
+    }
+    if (tid == 0) { part.ml[2 * pr] = M; part.ml[2 * pr + 1] = L; }
+}
+
+// attention output of (row, head) in latent space: column j, partials added in split order; `sc` [splits] holds the
+// factors exp(m_s - M) / L of latent_part_factors
+DEVINL void latent_part_factors(const LatentPart& part, size_t rh, float* sc) {
+    if (threadIdx.x < 32) {
+        float M = -INFINITY;
+        for (int s = threadIdx.x; s < part.splits; s += 32) {
+            const float* ml = part.ml + 2 * ((size_t)s * part.rows + rh);
+            if (__ldcg(ml + 1) > 0.0f) M = fmaxf(M, __ldcg(ml));
+        }
+        M = warp_max(M);
+        float L = 0.0f;
+        for (int s = threadIdx.x; s < part.splits; s += 32) {
+            const float* ml = part.ml + 2 * ((size_t)s * part.rows + rh);
+            const float l = __ldcg(ml + 1), f = l > 0.0f ? expf(__ldcg(ml) - M) : 0.0f;
+            sc[s] = f;
+            L += l * f;
+        }
+        L = warp_sum(L);
+        __syncwarp();
+        for (int s = threadIdx.x; s < part.splits; s += 32) sc[s] = L > 0.0f ? sc[s] / L : 0.0f;
+    }
+    __syncthreads();
+}
+DEVINL float latent_part_value(const LatentPart& part, size_t rh, int rank, int j, const float* sc) {
+    float t = 0.0f;
+    for (int s = 0; s < part.splits; ++s)
+        if (sc[s] > 0.0f) t = fmaf(__ldcg(part.o + ((size_t)s * part.rows + rh) * rank + j), sc[s], t);
+    return t;
+}
+
+// many rows: merged output as BF16 operands of the per-head products with W_uv, [heads][R][ld]. grid (heads, R)
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(int R, int heads, int rank, LatentPart part, uint16_t* x, int ld) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* sc = reinterpret_cast<float*>(smem_raw);
+    pdl_wait();
+    pdl_launch();
+    const int hd = blockIdx.x, r = blockIdx.y;
+    const size_t rh = (size_t)r * heads + hd;
+    latent_part_factors(part, rh, sc);
+    for (int j = threadIdx.x; j < ld; j += 128)
+        store_act(x + ((size_t)hd * R + r) * ld + j, j < rank ? latent_part_value(part, rh, rank, j, sc) : 0.0f);
+}
+
+// few rows: merge, W_uv and the output gate: out[r, h * vdim + v] = (W_uv[h, v, :] . o) * sigmoid(gate). W_uv rows are
+// `ldw` elements apart. grid (heads, R, slices of 32 value columns), 256 threads, shared memory splits + rank floats
+template <typename WT>
+__global__ void __launch_bounds__(256)
+latent_out_kernel(int heads, int rank, int vdim, LatentPart part, const WT* w_uv, int ldw, SplitIn gate, int c_gate,
+                  const uint32_t* tok, float* out, int ld_out) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* so = reinterpret_cast<float*>(smem_raw);
+    float* sc = so + rank;
+    pdl_wait();
+    pdl_launch();
+    const int hd = blockIdx.x, r = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    if (tok[r] == kInactiveToken) return;
+    const size_t rh = (size_t)r * heads + hd;
+    latent_part_factors(part, rh, sc);
+    for (int j = threadIdx.x; j < rank; j += 256) so[j] = latent_part_value(part, rh, rank, j, sc);
+    __syncthreads();
+    for (int i = warp; i < 32; i += 8) {
+        const int v = blockIdx.z * 32 + i;
+        if (v >= vdim) break;
+        const size_t base = ((size_t)hd * vdim + v) * ldw;
+        float t = 0.0f;
+        for (int j = lane; j < rank; j += 32) t = fmaf(WTraits<WT>::elem(w_uv, base + j), so[j], t);
+        t = warp_sum(t);
+        if (lane == 0) {
+            const int c = hd * vdim + v;
+            out[(size_t)r * ld_out + c] = t * sigmoid(gate.at(r, c_gate + c));
+        }
+    }
+}
+
+}  // namespace oxg4

@@ -26,6 +26,7 @@
 #include "sampling.cuh"
 #include "batch_ops.cuh"
 #include "tc_gemm.cuh"
+#include "layered_ops.cuh"
 #include "tp.h"
 
 using namespace oxg4;
@@ -75,6 +76,34 @@ struct GemvPlan {             // how a projection is cut into CTA row blocks and
     int N = 0, K = 0, cpr = 0, grid = 0, slots = 1, rows_max = 0;
 };
 
+// A projection of a layered model: W [N, K] row-major, rows and columns zero-padded. With nseg > 1 the rows form
+// segments of seg_rows (a multiple of the tcgen05 tile) and every segment multiplies its own input.
+struct Proj {
+    const void* w = nullptr;
+    const void* w1 = nullptr; // gate/up: the up projection (N counts the gate rows only)
+    int N = 0, K = 0, nseg = 1, seg_rows = 0;
+    GemvPlan gp;
+};
+
+enum MixerKind { MIX_GQA = OXG4_MIXER_GQA, MIX_LATENT = OXG4_MIXER_LATENT_ATTENTION, MIX_LIGHTNING = OXG4_MIXER_LIGHTNING,
+                 MIX_WKV = OXG4_MIXER_WKV };
+
+// What a layer of a layered model (csrc/layered.inl) needs beyond the common part of LayerPlan.
+struct MixPlan {
+    int kind = MIX_GQA;
+    int heads = 0, dim = 0, vdim = 0, ow = 0, owp = 0;        // ow = heads * vdim, owp: padded
+    int q_rank = 0, q_rankp = 0, rank = 0, rot = 0, rot_dims = 0, ld = 0;    // latent attention; ld: cache row
+    int low_rank = 0, ff = 0, ffp = 0;
+    int c_q = 0, c_k = 0, c_v = 0, c_g = 0, c_low = 0, c_dq = 0, c_dkv = 0;  // columns of the fused input projection
+    int vpad = 0;             // latent attention: rows per head of the padded W_uv
+    float scale = 1;
+    Proj in, uq, uk, uv, o, gateup, down;
+    const void *w_uk = nullptr, *w_uv = nullptr, *w2 = nullptr;             // checkpoint layout
+    const float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
+    const float *out_norm = nullptr, *mu = nullptr, *w0 = nullptr, *u = nullptr, *decay = nullptr, *dq_norm = nullptr,
+                *dkv_norm = nullptr, *inv_freq = nullptr;
+};
+
 struct LayerPlan {            // Gemma4DecodeLayerPlan (gemma4_cuda/mod.rs:65-93)
     bool sliding = false;
     // head geometry of this layer (local to the tensor-parallel rank): sliding layers use head_dim and
@@ -94,6 +123,7 @@ struct LayerPlan {            // Gemma4DecodeLayerPlan (gemma4_cuda/mod.rs:65-93
     const float *input_ln = nullptr, *post_attn_ln = nullptr, *pre_ff_ln = nullptr,
                 *post_ff_ln = nullptr, *q_norm = nullptr, *k_norm = nullptr;
     float* inv_freq = nullptr;
+    MixPlan mix;              // layered models only
 };
 
 struct ProfileSlot {
@@ -122,8 +152,15 @@ struct oxg4_model {
     int stage_next = 0;
     std::vector<LayerPlan> layers;
     const void* embed = nullptr;
+    const void* head = nullptr;   // output projection: the embedding table, or a matrix of its own (layered models)
     const float* final_norm = nullptr;
+    bool layered = false;         // layers listed one by one (csrc/layered.inl)
+    std::vector<oxg4_layer_spec> specs;
+    std::vector<std::vector<float>> spec_decay;
+    std::vector<void*> owned;     // device allocations of a layered model besides `tensors`
+    int64_t owned_bytes = 0;
     // local (per tensor-parallel rank) sizes
+    int Hn = 0;               // values of a residual row that count for its means; H is Hn rounded up to 8 in a layered model
     int H = 0, Nq = 0, I = 0, V = 0, Vloc = 0, v0 = 0;
     int Dmax = 0, qkv_n_max = 0, qw_max = 0, kvw_max = 0;   // largest head_dim / fused rows / Nq*D / Nkv*D over the layers
     int P = 0;                // hidden_size_per_layer_input (0: no per-layer embeddings)
@@ -249,7 +286,7 @@ extern "C" int32_t oxg4_model_create(const oxg4_config* c, int32_t device, oxg4_
     m->cfg.rope_factor = m->rope_factor.data();
     m->cfg.tp_size = tp;
     m->device = device;
-    m->H = c->hidden_size;
+    m->H = m->Hn = c->hidden_size;
     m->Nq = c->num_attention_heads / tp;
     m->P = c->hidden_size_per_layer_input;
     m->I = c->intermediate_size / tp;
@@ -287,6 +324,7 @@ extern "C" void oxg4_model_destroy(oxg4_model* m) {
     while (!m->caches.empty()) oxg4_cache_destroy(m->caches.back());   // a table points into its model: it goes first
     for (auto& kv : m->tensors) cudaFree(kv.second.d);
     for (auto& l : m->layers) cudaFree(l.inv_freq);
+    for (void* p : m->owned) cudaFree(p);
     for (int i = 0; i < 2; ++i) {
         if (m->stage[i]) cudaFreeHost(m->stage[i]);
         if (m->stage_ev[i]) cudaEventDestroy(m->stage_ev[i]);
@@ -344,7 +382,7 @@ extern "C" int32_t oxg4_model_upload(oxg4_model* m, const char* name, int32_t dt
         // tensor parallelism: keep only this rank's rows / columns (csrc/tp.h)
         const int ln_ = layer_of_name(n);
         const bool has_layer = ln_ >= 0 && ln_ < m->cfg.num_hidden_layers;
-        const ShardSpec sh = shard_of(n, shape[0], shape[1], m->tp_rank, m->tp, m->cfg.num_attention_heads,
+        const ShardSpec sh = m->layered ? ShardSpec{0, shape[0], 0, shape[1]} : shard_of(n, shape[0], shape[1], m->tp_rank, m->tp, m->cfg.num_attention_heads,
                                       has_layer ? layer_kv_heads(m->cfg, m->cfg.layer_is_sliding, ln_) : m->cfg.num_key_value_heads,
                                       has_layer ? layer_head_dim(m->cfg, m->cfg.layer_is_sliding, ln_) : m->cfg.head_dim,
                                       m->cfg.intermediate_size);
@@ -421,6 +459,10 @@ static int32_t set_gemv_attrs() {
     SETA(PRO_PLAIN, EPI_STORE);
     SETA(PRO_NORM, EPI_GATEUP);
     SETA(PRO_NORM, EPI_LOGITS);
+    if constexpr (NB == 1) {
+        SETA(PRO_SHIFT, EPI_STORE);
+        SETA(PRO_GNORM, EPI_STORE);
+    }
 #undef SETA
     return OXG4_OK;
 }
@@ -459,6 +501,18 @@ static int32_t set_attn_attrs() {
     return OXG4_OK;
 }
 
+static int32_t finalize_layered(oxg4_model* m);
+static int32_t set_projection_attrs(oxg4_model* m) {
+    if (m->es == 2) {
+        TRY((set_gemv_attrs<uint16_t, 1>()));
+        TRY((set_mma_attrs<8>()));
+        TRY((set_mma_attrs<16>()));
+    } else {
+        TRY((set_gemv_attrs<float, 1>())); TRY((set_gemv_attrs<float, 2>())); TRY((set_gemv_attrs<float, 4>()));
+    }
+    return allow_big_smem(topk_stage2_kernel);
+}
+
 extern "C" int32_t oxg4_model_finalize(oxg4_model* m) {
     if (!m) return fail(OXG4_INVALID_ARGUMENT, "null model");
     if (m->finalized) return OXG4_OK;
@@ -468,11 +522,18 @@ extern "C" int32_t oxg4_model_finalize(oxg4_model* m) {
         if (m->stage[i]) { cudaFreeHost(m->stage[i]); m->stage[i] = nullptr; }
         if (m->stage_ev[i]) { cudaEventDestroy(m->stage_ev[i]); m->stage_ev[i] = nullptr; }
     }
+    if (m->layered) {
+        TRY(finalize_layered(m));
+        TRY(set_projection_attrs(m));
+        CK(cudaDeviceSynchronize());
+        m->finalized = true;
+        return OXG4_OK;
+    }
     const oxg4_config& c = m->cfg;
     const int L = c.num_hidden_layers, H = m->H;
     const Tensor* t = nullptr;
     TRY(need(m, "embed_tokens.weight", {c.vocab_size, H}, &t));
-    m->embed = t->d;
+    m->embed = m->head = t->d;
     TRY(need(m, "norm.weight", {H}, &t));
     m->final_norm = (const float*)t->d;
     if (m->P > 0) {
@@ -580,16 +641,9 @@ extern "C" int32_t oxg4_model_finalize(oxg4_model* m) {
     m->p_down = make_plan(H, m->I, m->es, m->num_sms, 1);
     m->p_lm = make_plan(m->Vloc, H, m->es, m->num_sms, 1);
     m->p_lm_simt_grid = std::min(m->num_sms, std::max(1, (m->Vloc + 2 * kSimtWarps - 1) / (2 * kSimtWarps)));
-    if (m->es == 2) {
-        TRY((set_gemv_attrs<uint16_t, 1>()));
-        TRY((set_mma_attrs<8>()));
-        TRY((set_mma_attrs<16>()));
-    } else {
-        TRY((set_gemv_attrs<float, 1>())); TRY((set_gemv_attrs<float, 2>())); TRY((set_gemv_attrs<float, 4>()));
-    }
+    TRY(set_projection_attrs(m));
     TRY((set_attn_attrs<uint16_t, 64>())); TRY((set_attn_attrs<uint16_t, 128>())); TRY((set_attn_attrs<uint16_t, 256>()));
     TRY((set_attn_attrs<float, 64>())); TRY((set_attn_attrs<float, 128>())); TRY((set_attn_attrs<float, 256>()));
-    TRY(allow_big_smem(topk_stage2_kernel));
     CK(cudaDeviceSynchronize());
     m->finalized = true;
     return OXG4_OK;
@@ -597,7 +651,7 @@ extern "C" int32_t oxg4_model_finalize(oxg4_model* m) {
 
 extern "C" int64_t oxg4_weight_count(const oxg4_model* m) { return m ? (int64_t)m->tensors.size() : 0; }
 extern "C" int64_t oxg4_weight_bytes(const oxg4_model* m) {
-    int64_t b = 0;
+    int64_t b = m ? m->owned_bytes : 0;
     if (m) for (auto& kv : m->tensors) b += (int64_t)kv.second.bytes;
     return b;
 }
@@ -705,6 +759,14 @@ struct oxg4_cache {
     float *ple_emb = nullptr, *ple_ctx = nullptr, *ple_packed = nullptr, *ple_h = nullptr, *ple_gate = nullptr, *ple_act = nullptr,
           *ple_raw = nullptr;
 
+    // layered models: runs of a chunk (one per sequence in it), recurrent states and token-shift states per layer, scratch
+    int32_t *pf_run_row0 = nullptr, *pf_run_n = nullptr;
+    std::vector<float*> state, shift;
+    void *mix_x = nullptr, *mix_y = nullptr, *x_q = nullptr, *x_u = nullptr, *x_l = nullptr;
+    float *xf = nullptr, *in_buf = nullptr, *q_buf = nullptr, *uk_buf = nullptr, *uv_buf = nullptr, *wdec = nullptr, *lat_q = nullptr,
+          *lat_o = nullptr, *lat_ml = nullptr;
+    int lat_splits = 1;
+
     int32_t *dec_grp_row0 = nullptr, *dec_grp_n = nullptr;      // decode: one group per sequence
     float *last_h = nullptr, *last_raw = nullptr;               // [B, H] residual stream / pending update of every sequence's last prompt token
     uint16_t* last_x = nullptr;                                 // [B, H] tcgen05 path: its normed BF16 activations
@@ -756,6 +818,8 @@ static int32_t attn_mma_setup();
 static int tc_pick_splits(int tiles, int kblocks, int grid, int B, int n_total, int K, double max_extra = 0.3);
 static int32_t encode_bf16_2d(CUtensorMap* map, const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows);
 
+static int32_t layered_cache_build(oxg4_cache* c, int pages_full);
+
 static int32_t cache_build(oxg4_cache* c) {
     oxg4_model* m = c->m;
     const int B = c->B, L = m->cfg.num_hidden_layers, H = m->H, PT = c->PT;
@@ -792,7 +856,7 @@ static int32_t cache_build(oxg4_cache* c) {
     CK(cudaMemcpy(c->pt_slide, pts.data(), pts.size() * 4, cudaMemcpyHostToDevice));
     CK(cudaMemcpy(c->cap_full, capf.data(), B * 4, cudaMemcpyHostToDevice));
     CK(cudaMemcpy(c->cap_slide, caps.data(), B * 4, cudaMemcpyHostToDevice));
-    c->mma_attn = c->kv_dtype == OXG4_BF16 && PT % kAmTile == 0 && getenv("OXG4_DISABLE_MMA_ATTN") == nullptr;
+    c->mma_attn = !m->layered && c->kv_dtype == OXG4_BF16 && PT % kAmTile == 0 && getenv("OXG4_DISABLE_MMA_ATTN") == nullptr;
     c->kpool.assign(L, nullptr);
     c->vpool.assign(L, nullptr);
     c->pool_bytes.assign(L, 0);
@@ -802,7 +866,7 @@ static int32_t cache_build(oxg4_cache* c) {
     c->min_split = 16;
     c->attn_cluster = true;
     int smax = 1, part_floats = 1, ticket_n = 1;
-    for (int l = 0; l < L; ++l) {
+    for (int l = 0; l < L && !m->layered; ++l) {
         const LayerPlan& p = m->layers[l];
         if (p.shared) {
             // a KV-shared layer reads the pools of its source layer (cache.rs:70-84)
@@ -885,7 +949,9 @@ static int32_t cache_build(oxg4_cache* c) {
     TRY(dalloc(c, &c->last_raw, (size_t)B * H));
     TRY(dalloc(c, &c->last_x, (size_t)B * H));
     CK(cudaMallocHost(&c->h_pf_tok, sizeof(uint32_t) * kPrefillRows));
-    CK(cudaMallocHost(&c->h_pf_meta, sizeof(int32_t) * (2 * kPrefillRows + 4 * kAmMaxGroups)));
+    TRY(dalloc(c, &c->pf_run_row0, kPrefillRows));
+    TRY(dalloc(c, &c->pf_run_n, kPrefillRows));
+    CK(cudaMallocHost(&c->h_pf_meta, sizeof(int32_t) * (4 * kPrefillRows + 4 * kAmMaxGroups)));
     {
         std::vector<int32_t> r0(B), ones(B, 1);
         for (int b = 0; b < B; ++b) r0[b] = b;
@@ -906,8 +972,8 @@ static int32_t cache_build(oxg4_cache* c) {
     }
     // models with per-layer embeddings run through the small-batch kernels only (the extra projections per layer
     // are tiny and have no tcgen05 variant)
-    c->tc_ok = m->es == 2 && m->P == 0 && getenv("OXG4_DISABLE_TCGEN05") == nullptr;
-    c->use_tc = c->tc_ok && B >= 8 && B <= kPrefillRows;       // up to 256 sequences: row blocks of 128 / 256 (UMMA N)
+    c->tc_ok = m->es == 2 && m->P == 0 && (m->layered || getenv("OXG4_DISABLE_TCGEN05") == nullptr);
+    c->use_tc = c->tc_ok && B >= (m->layered ? 2 : 8) && B <= kPrefillRows;       // up to 256 sequences: row blocks of 128 / 256 (UMMA N)
     c->ls_qkv.assign(L, 1);
     c->ls_o.assign(L, 1);
     c->lps_qkv.assign(L, 1);
@@ -922,7 +988,9 @@ static int32_t cache_build(oxg4_cache* c) {
         TRY(dalloc(c, &c->ple_act, (size_t)R * m->P));
         TRY(dalloc(c, &c->ple_raw, (size_t)R * H));
     }
-    if (c->tc_ok) {
+    if (m->layered) TRY(layered_cache_build(c, pages_full));
+    if (c->tc_ok && m->layered) TRY(tc_gemm_setup());
+    if (c->tc_ok && !m->layered) {
         TRY(tc_gemm_setup());
         const int sms = m->num_sms;
         auto tiles = [](int n) { return (n + kTcTileM - 1) / kTcTileM; };
@@ -1005,6 +1073,7 @@ extern "C" int32_t oxg4_cache_create(oxg4_model* m, int32_t batch, const int32_t
     for (int b = 0; b < batch; ++b)
         if (max_seq[b] <= 0) return fail(OXG4_INVALID_SHAPE, "zero max_sequence");     // cache.rs:36-38
     if (page_tokens <= 0) return fail(OXG4_INVALID_SHAPE, "page_tokens must be positive");
+    if (m->layered && batch > kPrefillRows) return fail(OXG4_UNSUPPORTED, "a layered model takes at most %d sequences per table", kPrefillRows);
     if (kv_dtype != OXG4_F32 && kv_dtype != OXG4_BF16) return fail(OXG4_INVALID_ARGUMENT, "kv_dtype must be OXG4_F32 or OXG4_BF16");
     TRY(bind_device(m));
     oxg4_cache* c = new oxg4_cache();
@@ -1104,6 +1173,18 @@ extern "C" int32_t oxg4_cache_reset(oxg4_cache* c) {
     return OXG4_OK;
 }
 
+extern "C" int32_t oxg4_cache_reset_sequence(oxg4_cache* c, int32_t b) {
+    if (!c) return fail(OXG4_INVALID_ARGUMENT, "null cache");
+    if (b < 0 || b >= c->B) return fail(OXG4_INVALID_ARGUMENT, "sequence out of range");
+    TRY(bind_device(c->m));
+    cudaStream_t st = c->m->stream;
+    CK(cudaMemsetAsync(c->pos + b, 0, sizeof(int32_t), st));
+    CK(cudaMemsetAsync(c->seen + (size_t)b * c->m->V, 0, (size_t)c->m->V, st));
+    CK(cudaStreamSynchronize(st));
+    c->pos_host[b] = 0;
+    return OXG4_OK;
+}
+
 // ------------------------------------------------------------------------------------------------
 // tcgen05 projection: tensor maps, split choice, launch
 // ------------------------------------------------------------------------------------------------
@@ -1152,15 +1233,18 @@ static int tc_pick_splits(int tiles, int kblocks, int grid, int B, int n_total, 
 }
 
 // out[S, B, n_mats * N] = per-split partials of x[B, K] . W_m[N, K]^T on device pointers (BF16 in, f32 out).
+// seg_tiles > 0: the rows of W form segments of that many 128-row tiles, segment s multiplies rows s * B .. of x.
 static int32_t tc_gemm_launch(const void* w_dev, const void* w1_dev, const void* x_dev, int N, int K, int B, int S,
-                              float* out_dev, int ld, int col0, int* err_dev, int num_sms, cudaStream_t st, bool pdl) {
+                              float* out_dev, int ld, int col0, int* err_dev, int num_sms, cudaStream_t st, bool pdl,
+                              int seg_tiles = 0) {
     if (B < 1 || B > kPrefillRows || K % 8 != 0)
         return fail(OXG4_INVALID_SHAPE, "tcgen05 projection: 1..%d rows and K %% 8 == 0 required", kPrefillRows);
     const int bn = B <= 16 ? 16 : (B <= 32 ? 32 : (B <= 64 ? 64 : (B <= 128 ? 128 : 256)));
     CUtensorMap mw, mw1, mx;
     TRY(encode_bf16_2d(&mw, w_dev, (uint64_t)N, (uint64_t)K, kTcTileM));
     TRY(encode_bf16_2d(&mw1, w1_dev ? w1_dev : w_dev, (uint64_t)N, (uint64_t)K, kTcTileM));
-    TRY(encode_bf16_2d(&mx, x_dev, (uint64_t)B, (uint64_t)K, (uint32_t)bn));
+    const int n_segs = seg_tiles > 0 ? ((N + kTcTileM - 1) / kTcTileM + seg_tiles - 1) / seg_tiles : 1;
+    TRY(encode_bf16_2d(&mx, x_dev, (uint64_t)B * n_segs, (uint64_t)K, (uint32_t)bn));
     const int kblocks = (K + kTcTileK - 1) / kTcTileK;
     TcGemmArgs a{};
     a.N = N; a.K = K; a.B = B;
@@ -1168,6 +1252,7 @@ static int32_t tc_gemm_launch(const void* w_dev, const void* w1_dev, const void*
     a.S = S;
     a.TB = (B + bn - 1) / bn;
     a.kb_per_split = (kblocks + S - 1) / S;
+    a.seg_tiles = seg_tiles;
     a.out = out_dev;
     a.ld = ld;
     a.col0 = col0;
@@ -1273,12 +1358,12 @@ struct Launcher {
 
     // tcgen05 batched projection (csrc/tc_gemm.cuh): partials [S, B, ld] of x . W^T
     void tc(const char* kind, oxg4_cache* c, int rows, const void* w0, const void* w1, const uint16_t* x, int N, int K,
-            int S, float* out, int ld, int col0) {
+            int S, float* out, int ld, int col0, int seg_tiles = 0) {
         if (status != OXG4_OK) return;
         cudaEvent_t e0, e1;
         prof_begin(e0, e1);
         status = tc_gemm_launch(w0, w1, x, N, K, rows, S, out, ld, col0, c->tc_err, m->num_sms, m->stream,
-                                m->use_pdl && !m->profiling);
+                                m->use_pdl && !m->profiling, seg_tiles);
         if (status != OXG4_OK) return;
         prof_end(kind, e0, e1);
         ++kernels;
@@ -1328,7 +1413,11 @@ static void (*pick_gemv(int nb, int pro, int epi))(const GemvArgs) {
     if (pro == PRO_PLAIN && epi == EPI_STORE) return gemv_kernel<WT, NB, PRO_PLAIN, EPI_STORE>;     \
     if (pro == PRO_NORM && epi == EPI_GATEUP) return gemv_kernel<WT, NB, PRO_NORM, EPI_GATEUP>;     \
     if (pro == PRO_NORM && epi == EPI_LOGITS) return gemv_kernel<WT, NB, PRO_NORM, EPI_LOGITS>;
-    if (nb == 1) { PICK(1) }
+    if (nb == 1) {
+        PICK(1)
+        if (pro == PRO_SHIFT && epi == EPI_STORE) return gemv_kernel<WT, 1, PRO_SHIFT, EPI_STORE>;
+        if (pro == PRO_GNORM && epi == EPI_STORE) return gemv_kernel<WT, 1, PRO_GNORM, EPI_STORE>;
+    }
     if constexpr (sizeof(WT) == 4) {      // BF16 weights with more than one row use the tensor-core kernel
         if (nb == 2) { PICK(2) }
         if (nb == 4) { PICK(4) }
@@ -1360,7 +1449,8 @@ static void launch_gemv(Launcher& ln, const char* kind, oxg4_cache* c, int rows,
     a.pf_cap_kb = m->pf_cap_kb;
     if (epi == EPI_GATEUP && m->pf_cap_gu_kb >= 0) a.pf_cap_kb = m->pf_cap_gu_kb;
     if (!strcmp(kind, "down") && m->pf_cap_down_kb >= 0) a.pf_cap_kb = m->pf_cap_down_kb;
-    if (pro == PRO_NORM && p.K > std::min(kGemvMaxJ * kGemvThreads, kSimtMaxJ * kSimtThreads)) {
+    a.norm_n = p.K == m->H ? m->Hn : p.K;
+    if ((pro == PRO_NORM || pro == PRO_SHIFT) && p.K > std::min(kGemvMaxJ * kGemvThreads, kSimtMaxJ * kSimtThreads)) {
         ln.status = fail(OXG4_UNSUPPORTED, "hidden size above %d is not supported",
                          std::min(kGemvMaxJ * kGemvThreads, kSimtMaxJ * kSimtThreads));
         return;
@@ -1382,12 +1472,14 @@ static void launch_gemv(Launcher& ln, const char* kind, oxg4_cache* c, int rows,
         return;
     }
     // one activation row with BF16 weights, or f32 weights: SIMT kernel
-    const int nb = B >= 3 ? 4 : B;
+    int nb = B >= 3 ? 4 : B;
+    auto simt_need = [&](int n) {
+        return (size_t)std::max(1, a.nseg) * n * p.K * m->es + (size_t)n * 32 * 4 +
+               std::max((size_t)p.rows_max * p.slots * n * 4, (size_t)n * kSimtWarps * sizeof(Cand));
+    };
+    while (nb > 1 && simt_need(nb) > limit) nb /= 2;
     a.bpp = nb;
-    size_t smem = (size_t)nb * p.K * m->es + (size_t)nb * 32 * 4;
-    size_t extra = (size_t)p.rows_max * p.slots * nb * 4;
-    extra = std::max(extra, (size_t)nb * kSimtWarps * sizeof(Cand));
-    smem += extra;
+    const size_t smem = simt_need(nb);
     if (smem > limit) {
         ln.status = fail(OXG4_UNSUPPORTED, "projection %s needs %zu bytes of shared memory", kind, smem);
         return;
@@ -1450,6 +1542,22 @@ struct RowSet {
     const int32_t* grp_row0[2] = {nullptr, nullptr};
     const int32_t* grp_n[2] = {nullptr, nullptr};
     int NG[2] = {0, 0};
+    // runs of consecutive rows of one sequence (layered models)
+    const int32_t* run_row0 = nullptr;
+    const int32_t* run_n = nullptr;
+    std::vector<int> run_len;            // host copy of run_n
+};
+
+// The residual update a pass over the layers leaves to the kernel that follows: h + rmsnorm(sum of raw, w_post),
+// times scalar, goes to h_out.
+struct Pending {
+    const float* h = nullptr;
+    float* h_out = nullptr;
+    const float* raw = nullptr;          // [splits, R, H]
+    int splits = 1;
+    const float* w_post = nullptr;
+    float scalar = 1.0f;
+    PeerExchange px{};
 };
 
 // Launches every kernel of one step on the model's stream (eagerly or under stream capture).
@@ -1615,11 +1723,13 @@ static void ple_layer(oxg4_cache* c, Launcher& ln, const RowSet& rs, int l) {
     }
 }
 
-// All layers for the rows of `rs`. On return the last layer's residual update is still pending:
-// tcgen05 path: c->hA (+ the partials of the down projection), small-batch path: c->hA + c->down_raw.
-static void run_layers(oxg4_cache* c, Launcher& ln, const RowSet& rs, bool use_tc, bool peer, bool last_layer_prefetch,
-                       const TraceCtx* tr) {
+// All layers for the rows of `rs`. The last layer's residual update is returned still pending.
+static Pending run_layered(oxg4_cache* c, Launcher& ln, const RowSet& rs, bool use_tc, const TraceCtx* tr);
+
+static Pending run_layers(oxg4_cache* c, Launcher& ln, const RowSet& rs, bool use_tc, bool peer, bool last_layer_prefetch,
+                          const TraceCtx* tr) {
     oxg4_model* m = c->m;
+    if (m->layered) return run_layered(c, ln, rs, use_tc, tr);
     const int R = rs.R, L = m->cfg.num_hidden_layers, H = m->H;
     const int s_gu = rs.chunk ? c->ps_gu : c->s_gu, s_down = rs.chunk ? c->ps_down : c->s_down;
     if (m->P > 0) ple_prepare(c, ln, rs);
@@ -1653,13 +1763,13 @@ static void run_layers(oxg4_cache* c, Launcher& ln, const RowSet& rs, bool use_t
                 n.w_post = m->layers[l - 1].post_ff_ln;
                 n.scalar = m->layers[l - 1].layer_scalar;
             }
-            ln.go("norm", rows_norm_kernel, dim3(R), dim3(kRowsThreads), 0, n);
+            ln.go("norm", rows_norm_kernel<uint16_t>, dim3(R), dim3(kRowsThreads), 0, n);
             copy_trace_tc();
             if (tr && tr->inject_dev) {
                 RowsNormArgs f = n;                      // layer-wise teacher forcing: forced input, nothing pending
                 f.embed = nullptr; f.raw = nullptr; f.w_post = nullptr; f.scalar = 1.0f;
                 f.h_in = tr->inject_dev + (size_t)l * R * H;
-                ln.go("norm", rows_norm_kernel, dim3(R), dim3(kRowsThreads), 0, f);
+                ln.go("norm", rows_norm_kernel<uint16_t>, dim3(R), dim3(kRowsThreads), 0, f);
             }
             ln.tc("qkv", c, R, p.wqkv, nullptr, c->x_h, nqkv, H, s_qkv, c->qkv_part, nqkv, 0);
             launch_attention(ln, c, rs, l, c->qkv_part, s_qkv, c->x_a, true);
@@ -1691,10 +1801,10 @@ static void run_layers(oxg4_cache* c, Launcher& ln, const RowSet& rs, bool use_t
             n2.w_norm = p.pre_ff_ln;
             n2.eps = m->cfg.rms_norm_eps;
             n2.x = c->x_h;
-            ln.go("norm", rows_norm_kernel, dim3(R), dim3(kRowsThreads), 0, n2);
+            ln.go("norm", rows_norm_kernel<uint16_t>, dim3(R), dim3(kRowsThreads), 0, n2);
             ln.tc("gateup", c, R, p.wgate, p.wup, c->x_h, m->I, H, s_gu, c->gu_part, 2 * m->I, 0);
             ln.go("geglu", geglu_rows_kernel, dim3((m->I / 4 + kRowsThreads - 1) / kRowsThreads, R), dim3(kRowsThreads), 0, R,
-                  m->I, (const float*)c->gu_part, s_gu, c->x_i);
+                  m->I, (const float*)c->gu_part, s_gu, c->x_i, (int)ACT_GELU_TANH);
             const bool direct_d = m->tp > 1 && !peer && s_down == 1;
             ln.tc("down", c, R, p.wdown, nullptr, c->x_i, H, m->I, s_down, direct_d ? c->down_raw : c->down_part, H, 0);
             if (m->tp > 1) {
@@ -1795,36 +1905,48 @@ static void run_layers(oxg4_cache* c, Launcher& ln, const RowSet& rs, bool use_t
         }
         if (m->P > 0) ple_layer(c, ln, rs, l);
     }
+    Pending pd;
+    pd.h = m->P > 0 ? c->ple_h : c->hA;      // with per-layer embeddings the pending update is that branch
+    pd.h_out = c->hB;
+    pd.w_post = m->P > 0 ? m->layers[L - 1].ple_norm : m->layers[L - 1].post_ff_ln;
+    pd.scalar = m->layers[L - 1].layer_scalar;
+    pd.raw = m->P > 0 ? c->ple_raw : c->down_raw;
+    if (use_tc) {
+        pd.raw = m->tp > 1 ? (peer ? c->px[1].gathered : c->down_raw) : c->down_part;
+        pd.splits = m->tp > 1 ? (peer ? m->tp : 1) : s_down;
+        if (m->tp > 1 && peer) pd.px = c->px[1];
+    }
+    return pd;
 }
 
-// tcgen05 path: the last layer's pending update + final norm for `rows` rows: h -> c->hB, x -> c->x_h
-static void closing_norm_tc(oxg4_cache* c, Launcher& ln, int rows, bool chunk, bool peer) {
+// tcgen05 path: the last layer's pending update + final norm for `rows` rows: h -> pd.h_out, x -> c->x_h
+static void closing_norm_tc(oxg4_cache* c, Launcher& ln, int rows, const Pending& pd) {
     oxg4_model* m = c->m;
-    const int L = m->cfg.num_hidden_layers;
     RowsNormArgs n{};
     n.B = rows; n.H = m->H;
-    n.h_in = c->hA; n.h_out = c->hB;
-    n.raw = m->tp > 1 ? (peer ? c->px[1].gathered : c->down_raw) : c->down_part;
-    n.raw_splits = m->tp > 1 ? (peer ? m->tp : 1) : (chunk ? c->ps_down : c->s_down);
-    if (m->tp > 1 && peer) n.px = c->px[1];
-    n.w_post = m->layers[L - 1].post_ff_ln;
-    n.scalar = m->layers[L - 1].layer_scalar;
+    n.norm_n = m->Hn;
+    n.h_in = pd.h; n.h_out = pd.h_out;
+    n.raw = pd.raw;
+    n.raw_splits = pd.splits;
+    n.px = pd.px;
+    n.w_post = pd.w_post;
+    n.scalar = pd.scalar;
     n.w_norm = m->final_norm;
     n.eps = m->cfg.rms_norm_eps;
     n.x = c->x_h;
-    ln.go("norm", rows_norm_kernel, dim3(rows), dim3(kRowsThreads), 0, n);
+    ln.go("norm", rows_norm_kernel<uint16_t>, dim3(rows), dim3(kRowsThreads), 0, n);
 }
 
 // Tied LM head over B rows + arg-max / top-k (decode.rs:495-508, kernel_module.rs:1988-2075).
 // tcgen05 path: x [B, H] BF16 normed activations. Small-batch path: the pending update (h_in + raw) is closed by
 // the kernel's prologue.
 static void lm_head(oxg4_cache* c, Launcher& ln, int kind, int top_k, float penalty, bool use_tc, const uint16_t* x,
-                    const float* h_in, const float* raw, const TraceCtx* tr) {
+                    const Pending& pd, const TraceCtx* tr) {
     oxg4_model* m = c->m;
     const int B = c->B, L = m->cfg.num_hidden_layers, H = m->H;
     auto trace_final = [&]() {
         if (tr && ln.status == OXG4_OK &&
-            cudaMemcpyAsync(tr->trace_dev + (size_t)L * B * H, c->hB, sizeof(float) * B * H, cudaMemcpyDeviceToDevice,
+            cudaMemcpyAsync(tr->trace_dev + (size_t)L * B * H, pd.h_out, sizeof(float) * B * H, cudaMemcpyDeviceToDevice,
                             m->stream) != cudaSuccess)
             ln.status = fail(OXG4_CUDA, "Gemma 4 CUDA error: trace copy failed");
     };
@@ -1836,7 +1958,7 @@ static void lm_head(oxg4_cache* c, Launcher& ln, int kind, int top_k, float pena
         if (m->tp > 1 && kind == STEP_TOPK) {
             // every rank ranks its own vocabulary slice; N * k (score, id) pairs per sequence cross the links
             // instead of the [B, V] logits
-            ln.tc("lmhead", c, B, (const char*)m->embed + (size_t)m->v0 * H * m->es, nullptr, x, m->Vloc, H, 1,
+            ln.tc("lmhead", c, B, (const char*)m->head + (size_t)m->v0 * H * m->es, nullptr, x, m->Vloc, H, 1,
                   c->logits, m->V, m->v0);
             const int chunks = (m->Vloc + kTopkChunk - 1) / kTopkChunk;
             ln.go("topk1", topk_stage1_kernel, dim3(chunks, B), dim3(kTopkThreads), 0, (const float*)c->logits, m->V,
@@ -1852,7 +1974,7 @@ static void lm_head(oxg4_cache* c, Launcher& ln, int kind, int top_k, float pena
         // full logits wanted on the host: every rank fills its vocabulary columns, the sum assembles the rows
         if (m->tp > 1 && cudaMemsetAsync(c->logits, 0, sizeof(float) * (size_t)B * m->V, m->stream) != cudaSuccess)
             ln.status = fail(OXG4_CUDA, "Gemma 4 CUDA error: cudaMemsetAsync failed");
-        ln.tc("lmhead", c, B, (const char*)m->embed + (size_t)m->v0 * H * m->es, nullptr, x, m->Vloc, H, 1, c->logits,
+        ln.tc("lmhead", c, B, (const char*)m->head + (size_t)m->v0 * H * m->es, nullptr, x, m->Vloc, H, 1, c->logits,
               m->V, m->v0);
         ln.allreduce(c->logits, (size_t)B * m->V);
         // top-k over the full logits (k = 1 is the arg-max the greedy loop feeds back)
@@ -1865,12 +1987,12 @@ static void lm_head(oxg4_cache* c, Launcher& ln, int kind, int top_k, float pena
     }
     // post-FF norm + residual + layer_scalar of the last layer, final norm, tied LM head with fused arg-max
     GemvArgs a{};
-    a.W0 = (const char*)m->embed + (size_t)m->v0 * H * m->es;
-    a.h_in = h_in;
-    a.h_out = c->hB;
-    a.raw = raw;
-    a.w_post = m->P > 0 ? m->layers[L - 1].ple_norm : m->layers[L - 1].post_ff_ln;
-    a.scalar = m->layers[L - 1].layer_scalar;
+    a.W0 = (const char*)m->head + (size_t)m->v0 * H * m->es;
+    a.h_in = pd.h;
+    a.h_out = pd.h_out;
+    a.raw = pd.raw;
+    a.w_post = pd.w_post;
+    a.scalar = pd.scalar;
     a.w_norm = m->final_norm;
     const bool want_logits = (kind == STEP_LOGITS) || top_k > 1;
     a.out = want_logits ? c->logits : nullptr;
@@ -1926,11 +2048,13 @@ static int32_t run_step(oxg4_cache* c, int kind, int top_k, float penalty, int* 
         rs.grp_n[k] = c->dec_grp_n;
         rs.NG[k] = B;
     }
-    run_layers(c, ln, rs, c->use_tc, peer, kind != STEP_PREFILL, tr);
+    rs.run_row0 = c->dec_grp_row0;
+    rs.run_n = c->dec_grp_n;
+    rs.run_len.assign(B, 1);
+    const Pending pd = run_layers(c, ln, rs, c->use_tc, peer, kind != STEP_PREFILL, tr);
     if (kind != STEP_PREFILL) {
-        if (c->use_tc) closing_norm_tc(c, ln, B, false, peer);
-        const bool ple = m->P > 0;       // the last layer's pending update is then its per-layer-embedding branch
-        lm_head(c, ln, kind, top_k, penalty, c->use_tc, c->x_h, ple ? c->ple_h : c->hA, ple ? c->ple_raw : c->down_raw, tr);
+        if (c->use_tc) closing_norm_tc(c, ln, B, pd);
+        lm_head(c, ln, kind, top_k, penalty, c->use_tc, c->x_h, pd, tr);
     }
     if (kind == STEP_TOPK && top_k > 1)      // a no-op unless the step's control words ask for a sampled token
         ln.go("sample", sample_candidates_kernel, dim3(1), dim3(64), 0, B, top_k, m->cfg.final_logit_softcapping,
@@ -2234,6 +2358,7 @@ extern "C" int32_t oxg4_decode_trace(oxg4_model* m, oxg4_cache* c, const uint32_
     if (!m || !c || !tokens || !trace || c->m != m) return fail(OXG4_INVALID_ARGUMENT, "null or mismatched handle");
     TRY(bind_device(m));
     TRY(check_tokens(c, tokens, true));
+    if (m->layered && inject) return fail(OXG4_UNSUPPORTED, "layer inputs cannot be forced in a layered model");
     const int L = m->cfg.num_hidden_layers;
     const size_t per = (size_t)c->B * m->H;
     float *d_inject = nullptr, *d_trace = nullptr;
@@ -2251,7 +2376,8 @@ extern "C" int32_t oxg4_decode_trace(oxg4_model* m, oxg4_cache* c, const uint32_
     if (s == OXG4_OK && cudaStreamSynchronize(m->stream) != cudaSuccess) s = fail(OXG4_CUDA, "Gemma 4 CUDA error: trace step failed");
     if (s == OXG4_OK) {
         m->launches += n;
-        cudaMemcpy(trace, d_trace, sizeof(float) * per * (L + 1), cudaMemcpyDeviceToHost);
+        cudaMemcpy2D(trace, sizeof(float) * m->Hn, d_trace, sizeof(float) * m->H, sizeof(float) * m->Hn, (size_t)c->B * (L + 1),
+                     cudaMemcpyDeviceToHost);
         if (logits) {
             cudaMemcpy(logits, c->logits, sizeof(float) * (size_t)c->B * m->V, cudaMemcpyDeviceToHost);
             softcap(logits, (size_t)c->B * m->V, m->cfg.final_logit_softcapping);
@@ -2280,6 +2406,7 @@ static int32_t smoke_check(oxg4_model* m, uint32_t token, int32_t layer, bool ne
     if (!m) return fail(OXG4_INVALID_ARGUMENT, "null argument");
     if (!m->finalized) return fail(OXG4_INVALID_ARGUMENT, "model is not finalized");
     if (m->tp > 1) return fail(OXG4_UNSUPPORTED, "the diagnostic entry points run on a single-GPU model");
+    if (m->layered) return fail(OXG4_UNSUPPORTED, "the diagnostic entry points run on Gemma 4 models");
     if (token >= (uint32_t)m->V) return fail(OXG4_INVALID_ARGUMENT, "token id exceeds CUDA embedding table");   // attention.rs:13-17
     if (need_layer && (layer < 0 || layer >= m->cfg.num_hidden_layers)) return fail(OXG4_INVALID_ARGUMENT, "layer out of range");
     if (own_kv && m->layers[layer].shared) return fail(OXG4_UNSUPPORTED, "layer %d shares the K/V of layer %d", layer, m->layers[layer].source);
@@ -2480,14 +2607,160 @@ extern "C" int32_t oxg4_profile_count(const oxg4_model* m, const char* kind) {
     return it == m->profile.end() ? 0 : it->second.count;
 }
 
-// prefill_prompt (decode.rs:386-459): the prompts of all sequences go through the layers in chunks of up to
-// kPrefillRows tokens, each chunk one pass with matrix-shaped projections (tcgen05 for BF16 weights) and causal /
-// sliding paged attention over the chunk; a chunk may hold the tail of one sequence and the head of the next.
-// Unlike the reference there is no 4096-token limit and no requirement that the prompt fits the sliding ring.
+// Feeds lens[b] (possibly zero) further tokens of every sequence, which continues at its current position. The tokens of
+// all sequences go through the layers in chunks of up to kPrefillRows, each chunk one pass with matrix-shaped projections
+// (tcgen05 for BF16 weights) and causal / sliding paged attention over the chunk; a chunk may hold the tail of one
+// sequence and the head of the next. `want` (null: none) marks the tokens whose logits are wanted; they are written to
+// `logits` in token order.
+static int32_t ingest(oxg4_model* m, oxg4_cache* c, const uint32_t* tokens, const int32_t* lens, const uint8_t* want,
+                      float* logits) {
+    const int B = c->B, H = m->H;
+    std::vector<int64_t> off(B + 1, 0);
+    for (int b = 0; b < B; ++b) {
+        if (lens[b] < 0) return fail(OXG4_INVALID_ARGUMENT, "negative token count");
+        if (lens[b] > c->max_seq[b] - c->pos_host[b]) return fail(OXG4_INVALID_SHAPE, "prompt does not fit the cache table");
+        off[b + 1] = off[b] + lens[b];
+    }
+    for (int64_t i = 0; i < off[B]; ++i) {
+        if (tokens[i] >= (uint32_t)m->V) return fail(OXG4_INVALID_ARGUMENT, "token id exceeds CUDA decode vocabulary");
+        if (m->P > 0 && tokens[i] >= (uint32_t)m->cfg.vocab_size_per_layer_input)
+            return fail(OXG4_INVALID_SHAPE, "invalid batched PLE input");                       // ple.rs:113-119
+    }
+    TRY(bind_device(m));
+    const bool use_tc = c->tc_ok;
+    // tokens per attention group, per layer kind (0 sliding, 1 global): 8 / (query heads per KV head)
+    int tg[2] = {1, 1};
+    for (auto& lp : m->layers) tg[lp.sliding ? 0 : 1] = std::max(1, kAmRows / lp.G);
+    int32_t* h_pos = c->h_pf_meta;
+    int32_t* h_seq = h_pos + kPrefillRows;
+    int32_t* h_g0[2] = {h_seq + kPrefillRows, h_seq + kPrefillRows + 2 * kAmMaxGroups};
+    int32_t* h_gn[2] = {h_g0[0] + kAmMaxGroups, h_g0[1] + kAmMaxGroups};
+    int32_t* h_run0 = h_seq + kPrefillRows + 4 * kAmMaxGroups;
+    int32_t* h_runn = h_run0 + kPrefillRows;
+    // wanted rows wait in last_x / last_h + last_raw until B of them (or all) are there: one LM head pass over B rows
+    int held = 0;
+    int64_t delivered = 0;
+    Pending last;
+    last.h = c->last_h;
+    last.raw = c->last_raw;
+    auto flush = [&]() -> int32_t {
+        if (held == 0) return OXG4_OK;
+        Launcher ln{m};
+        lm_head(c, ln, STEP_LOGITS, 1, 1.0f, use_tc, c->last_x, last, nullptr);
+        TRY(ln.status);
+        m->launches += ln.kernels;
+        CK(cudaMemcpyAsync(logits + (size_t)delivered * m->V, c->logits, sizeof(float) * (size_t)held * m->V, cudaMemcpyDeviceToHost,
+                           m->stream));
+        CK(cudaStreamSynchronize(m->stream));
+        softcap(logits + (size_t)delivered * m->V, (size_t)held * m->V, m->cfg.final_logit_softcapping);
+        delivered += held;
+        held = 0;
+        return OXG4_OK;
+    };
+    int b = 0, p = 0;                                          // next token to place: sequence b, position p
+    while (b < B) {
+        int R = 0, NG[2] = {0, 0};
+        std::vector<int> wanted;                               // rows whose logits are asked for
+        RowSet rs;
+        while (b < B && R < kPrefillRows) {
+            if (lens[b] == 0) { ++b; continue; }
+            const int take = std::min(kPrefillRows - R, lens[b] - p);
+            for (int i = 0; i < take; ++i) {
+                c->h_pf_tok[R + i] = tokens[off[b] + p + i];
+                h_pos[R + i] = c->pos_host[b] + p + i;
+                if (want && want[off[b] + p + i]) wanted.push_back(R + i);
+                h_seq[R + i] = b;
+            }
+            for (int k = 0; k < 2; ++k)
+                for (int i = 0; i < take; i += tg[k]) {
+                    h_g0[k][NG[k]] = R + i;
+                    h_gn[k][NG[k]] = std::min(tg[k], take - i);
+                    ++NG[k];
+                }
+            h_run0[rs.run_len.size()] = R;
+            h_runn[rs.run_len.size()] = take;
+            rs.run_len.push_back(take);
+            R += take;
+            p += take;
+            if (p == lens[b]) { ++b; p = 0; }
+        }
+        if (R == 0) break;
+        cudaStream_t st = m->stream;
+        CK(cudaMemcpyAsync(c->pf_tok, c->h_pf_tok, sizeof(uint32_t) * R, cudaMemcpyHostToDevice, st));
+        CK(cudaMemcpyAsync(c->pf_pos, h_pos, sizeof(int32_t) * R, cudaMemcpyHostToDevice, st));
+        CK(cudaMemcpyAsync(c->pf_seq, h_seq, sizeof(int32_t) * R, cudaMemcpyHostToDevice, st));
+        for (int k = 0; k < 2; ++k) {
+            CK(cudaMemcpyAsync(c->pf_grp_row0[k], h_g0[k], sizeof(int32_t) * NG[k], cudaMemcpyHostToDevice, st));
+            CK(cudaMemcpyAsync(c->pf_grp_n[k], h_gn[k], sizeof(int32_t) * NG[k], cudaMemcpyHostToDevice, st));
+        }
+        CK(cudaMemcpyAsync(c->pf_run_row0, h_run0, sizeof(int32_t) * rs.run_len.size(), cudaMemcpyHostToDevice, st));
+        CK(cudaMemcpyAsync(c->pf_run_n, h_runn, sizeof(int32_t) * rs.run_len.size(), cudaMemcpyHostToDevice, st));
+        const bool prof = getenv("GEMMA4_PROFILE") != nullptr && getenv("OXG4_PROFILE_PREFILL") != nullptr;
+        m->profiling = prof;           // events around every launch of the chunk (a measurement aid, like the reference's GEMMA4_PROFILE)
+        Launcher ln{m};
+        rs.R = R;
+        rs.run_row0 = c->pf_run_row0;
+        rs.run_n = c->pf_run_n;
+        rs.tok = c->pf_tok;
+        rs.pos = c->pf_pos;
+        rs.seq = c->pf_seq;
+        rs.chunk = true;
+        for (int k = 0; k < 2; ++k) {
+            rs.grp_row0[k] = c->pf_grp_row0[k];
+            rs.grp_n[k] = c->pf_grp_n[k];
+            rs.NG[k] = NG[k];
+        }
+        const Pending pd = run_layers(c, ln, rs, use_tc, false, false, nullptr);
+        // keep what the LM head will need of every wanted row
+        if (use_tc && !wanted.empty() && ln.status == OXG4_OK) closing_norm_tc(c, ln, R, pd);
+        last.w_post = pd.w_post;
+        last.scalar = pd.scalar;
+        last.h_out = pd.h_out;         // scratch for the LM head's prologue; never the rows still to be copied
+        for (size_t i = 0; i < wanted.size() && ln.status == OXG4_OK; ++i) {
+            const size_t src = (size_t)wanted[i] * H, dst = (size_t)held * H;
+            if (use_tc) {
+                CK(cudaMemcpyAsync(c->last_x + dst, c->x_h + src, sizeof(uint16_t) * H, cudaMemcpyDeviceToDevice, st));
+            } else {
+                CK(cudaMemcpyAsync(c->last_h + dst, pd.h + src, sizeof(float) * H, cudaMemcpyDeviceToDevice, st));
+                CK(cudaMemcpyAsync(c->last_raw + dst, pd.raw + src, sizeof(float) * H, cudaMemcpyDeviceToDevice, st));
+            }
+            if (++held == B) TRY(flush());
+        }
+        m->profiling = false;
+        TRY(ln.status);
+        m->launches += ln.kernels;
+        CK(cudaStreamSynchronize(st));                         // the pinned staging is reused by the next chunk
+        if (prof) {
+            std::map<std::string, double> sum;
+            for (auto& pe : m->prof_events) {
+                float ms = 0;
+                cudaEventElapsedTime(&ms, pe.second.first, pe.second.second);
+                sum[pe.first] += ms;
+                cudaEventDestroy(pe.second.first);
+                cudaEventDestroy(pe.second.second);
+            }
+            m->prof_events.clear();
+            fprintf(stderr, "Gemma4 prefill chunk (%d rows):", R);
+            for (auto& kv : sum) fprintf(stderr, " %s %.3f ms", kv.first.c_str(), kv.second);
+            fprintf(stderr, "\n");
+        }
+        TRY(check_tc(c));
+    }
+    TRY(flush());
+    TRY(check_tc(c));
+    // device step state: every sequence continues behind its new tokens
+    for (int i = 0; i < B; ++i) c->pos_host[i] += lens[i];
+    CK(cudaMemcpyAsync(c->pos, c->pos_host.data(), sizeof(int32_t) * B, cudaMemcpyHostToDevice, m->stream));
+    CK(cudaStreamSynchronize(m->stream));
+    return OXG4_OK;
+}
+
+// prefill_prompt (decode.rs:386-459), whole prompts into an empty cache table, last-token logits. Unlike the reference
+// there is no 4096-token limit and no requirement that the prompt fits the sliding ring.
 extern "C" int32_t oxg4_prefill(oxg4_model* m, oxg4_cache* c, const uint32_t* tokens, const int32_t* lens,
                                 float* last_logits) {
     if (!m || !c || !tokens || !lens || c->m != m) return fail(OXG4_INVALID_ARGUMENT, "null or mismatched handle");
-    const int B = c->B, H = m->H;
+    const int B = c->B;
     std::vector<int64_t> off(B + 1, 0);
     for (int b = 0; b < B; ++b) {
         if (lens[b] <= 0) return fail(OXG4_INVALID_ARGUMENT, "batched prefill requires at least one token per sequence");
@@ -2514,112 +2787,17 @@ extern "C" int32_t oxg4_prefill(oxg4_model* m, oxg4_cache* c, const uint32_t* to
         if (last_logits) return oxg4_decode_logits(m, c, step_tokens.data(), last_logits);
         return oxg4_prefill_token(m, c, step_tokens.data());
     }
-    const bool use_tc = c->tc_ok;
-    // tokens per attention group, per layer kind (0 sliding, 1 global): 8 / (query heads per KV head)
-    int tg[2] = {1, 1};
-    for (auto& lp : m->layers) tg[lp.sliding ? 0 : 1] = std::max(1, kAmRows / lp.G);
-    int32_t* h_pos = c->h_pf_meta;
-    int32_t* h_seq = h_pos + kPrefillRows;
-    int32_t* h_g0[2] = {h_seq + kPrefillRows, h_seq + kPrefillRows + 2 * kAmMaxGroups};
-    int32_t* h_gn[2] = {h_g0[0] + kAmMaxGroups, h_g0[1] + kAmMaxGroups};
-    int b = 0, p = 0;                                          // next token to place: sequence b, position p
-    while (b < B) {
-        int R = 0, NG[2] = {0, 0};
-        std::vector<std::pair<int, int>> finishing;            // (sequence, row) of every last prompt token in this chunk
-        while (b < B && R < kPrefillRows) {
-            const int take = std::min(kPrefillRows - R, lens[b] - p);
-            for (int i = 0; i < take; ++i) {
-                c->h_pf_tok[R + i] = tokens[off[b] + p + i];
-                h_pos[R + i] = p + i;
-                h_seq[R + i] = b;
-            }
-            for (int k = 0; k < 2; ++k)
-                for (int i = 0; i < take; i += tg[k]) {
-                    h_g0[k][NG[k]] = R + i;
-                    h_gn[k][NG[k]] = std::min(tg[k], take - i);
-                    ++NG[k];
-                }
-            R += take;
-            p += take;
-            if (p == lens[b]) { finishing.push_back({b, R - 1}); ++b; p = 0; }
-        }
-        cudaStream_t st = m->stream;
-        CK(cudaMemcpyAsync(c->pf_tok, c->h_pf_tok, sizeof(uint32_t) * R, cudaMemcpyHostToDevice, st));
-        CK(cudaMemcpyAsync(c->pf_pos, h_pos, sizeof(int32_t) * R, cudaMemcpyHostToDevice, st));
-        CK(cudaMemcpyAsync(c->pf_seq, h_seq, sizeof(int32_t) * R, cudaMemcpyHostToDevice, st));
-        for (int k = 0; k < 2; ++k) {
-            CK(cudaMemcpyAsync(c->pf_grp_row0[k], h_g0[k], sizeof(int32_t) * NG[k], cudaMemcpyHostToDevice, st));
-            CK(cudaMemcpyAsync(c->pf_grp_n[k], h_gn[k], sizeof(int32_t) * NG[k], cudaMemcpyHostToDevice, st));
-        }
-        const bool prof = getenv("GEMMA4_PROFILE") != nullptr && getenv("OXG4_PROFILE_PREFILL") != nullptr;
-        m->profiling = prof;           // events around every launch of the chunk (a measurement aid, like the reference's GEMMA4_PROFILE)
-        Launcher ln{m};
-        RowSet rs;
-        rs.R = R;
-        rs.tok = c->pf_tok;
-        rs.pos = c->pf_pos;
-        rs.seq = c->pf_seq;
-        rs.chunk = true;
-        for (int k = 0; k < 2; ++k) {
-            rs.grp_row0[k] = c->pf_grp_row0[k];
-            rs.grp_n[k] = c->pf_grp_n[k];
-            rs.NG[k] = NG[k];
-        }
-        run_layers(c, ln, rs, use_tc, false, false, nullptr);
-        if (last_logits && !finishing.empty() && ln.status == OXG4_OK) {
-            // keep what the LM head will need of every sequence that ends in this chunk
-            if (use_tc) closing_norm_tc(c, ln, R, true, false);
-            for (auto& f : finishing) {
-                if (use_tc) {
-                    CK(cudaMemcpyAsync(c->last_x + (size_t)f.first * H, c->x_h + (size_t)f.second * H, sizeof(uint16_t) * H,
-                                       cudaMemcpyDeviceToDevice, st));
-                } else {
-                    // the last layer's pending update: the MLP block's output, or with per-layer embeddings that branch
-                    const float* h_src = m->P > 0 ? c->ple_h : c->hA;
-                    const float* raw_src = m->P > 0 ? c->ple_raw : c->down_raw;
-                    CK(cudaMemcpyAsync(c->last_h + (size_t)f.first * H, h_src + (size_t)f.second * H, sizeof(float) * H,
-                                       cudaMemcpyDeviceToDevice, st));
-                    CK(cudaMemcpyAsync(c->last_raw + (size_t)f.first * H, raw_src + (size_t)f.second * H,
-                                       sizeof(float) * H, cudaMemcpyDeviceToDevice, st));
-                }
-            }
-        }
-        m->profiling = false;
-        TRY(ln.status);
-        m->launches += ln.kernels;
-        CK(cudaStreamSynchronize(st));                         // the pinned staging is reused by the next chunk
-        if (prof) {
-            std::map<std::string, double> sum;
-            for (auto& pe : m->prof_events) {
-                float ms = 0;
-                cudaEventElapsedTime(&ms, pe.second.first, pe.second.second);
-                sum[pe.first] += ms;
-                cudaEventDestroy(pe.second.first);
-                cudaEventDestroy(pe.second.second);
-            }
-            m->prof_events.clear();
-            fprintf(stderr, "Gemma4 prefill chunk (%d rows):", R);
-            for (auto& kv : sum) fprintf(stderr, " %s %.3f ms", kv.first.c_str(), kv.second);
-            fprintf(stderr, "\n");
-        }
-        TRY(check_tc(c));
-    }
-    // device step state: every sequence continues at position lens[b]
-    std::vector<int32_t> np(lens, lens + B);
-    CK(cudaMemcpyAsync(c->pos, np.data(), sizeof(int32_t) * B, cudaMemcpyHostToDevice, m->stream));
-    CK(cudaStreamSynchronize(m->stream));      // np leaves scope; later steps read c->pos in stream order
-    for (int i = 0; i < B; ++i) c->pos_host[i] = lens[i];
-    if (last_logits) {
-        Launcher ln{m};
-        lm_head(c, ln, STEP_LOGITS, 1, 1.0f, use_tc, c->last_x, c->last_h, c->last_raw, nullptr);
-        TRY(ln.status);
-        m->launches += ln.kernels;
-        CK(cudaMemcpyAsync(last_logits, c->logits, sizeof(float) * (size_t)B * m->V, cudaMemcpyDeviceToHost, m->stream));
-        CK(cudaStreamSynchronize(m->stream));
-        TRY(check_tc(c));
-        softcap(last_logits, (size_t)B * m->V, m->cfg.final_logit_softcapping);
-    }
-    return OXG4_OK;
+    if (!last_logits) return ingest(m, c, tokens, lens, nullptr, nullptr);
+    std::vector<uint8_t> want((size_t)off[B], 0);
+    for (int b = 0; b < B; ++b) want[off[b + 1] - 1] = 1;
+    return ingest(m, c, tokens, lens, want.data(), last_logits);
+}
+
+// Portions of prompts: see ingest.
+extern "C" int32_t oxg4_extend(oxg4_model* m, oxg4_cache* c, const uint32_t* tokens, const int32_t* lens, const uint8_t* want,
+                               float* logits) {
+    if (!m || !c || !tokens || !lens || c->m != m || (want && !logits)) return fail(OXG4_INVALID_ARGUMENT, "null or mismatched handle");
+    return ingest(m, c, tokens, lens, want, logits);
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -2794,6 +2972,12 @@ extern "C" int32_t oxg4_debug_fill_cache(oxg4_model* m, oxg4_cache* c, const int
     for (int l = 0; l < L; ++l) {
         const size_t n16 = c->pool_bytes[l] / 16;
         if (n16 == 0) continue;
+        if (m->layered) {
+            // one pool of latents; recurrent states keep their (zero or earlier) contents
+            if (c->kv_dtype == OXG4_BF16) pool_fill_kernel<uint16_t><<<(int)std::min<size_t>((n16 + 255) / 256, (size_t)m->num_sms * 16), 256, 0, m->stream>>>((uint4*)c->kpool[l], n16, 2u * l + 1u);
+            else pool_fill_kernel<float><<<(int)std::min<size_t>((n16 + 255) / 256, (size_t)m->num_sms * 16), 256, 0, m->stream>>>((uint4*)c->kpool[l], n16, 2u * l + 1u);
+            continue;
+        }
         const int grid = (int)std::min<size_t>((n16 + 255) / 256, (size_t)m->num_sms * 16);
         if (c->kv_dtype == OXG4_BF16) {
             pool_fill_kernel<uint16_t><<<grid, 256, 0, m->stream>>>((uint4*)c->kpool[l], n16, 2u * l + 1u);
@@ -2936,4 +3120,5 @@ extern "C" int32_t oxg4_debug_tc_gemm(const uint16_t* w_host, const uint16_t* x_
     return s;
 }
 
+#include "layered.inl"
 #include "tp_group.inl"

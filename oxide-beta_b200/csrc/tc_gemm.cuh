@@ -41,6 +41,9 @@ struct TcGemmArgs {
     int TB;                  // row blocks: ceil(B / BN). Units of one weight tile are adjacent, so that tile
                              // crosses HBM once and the other row blocks find it in L2 (prompt chunks: B up to 256)
     int kb_per_split;        // 64-column blocks per split
+    int seg_tiles;           // > 0: the weight rows form segments of this many tiles and segment s multiplies its own
+                             // activations, rows s * B .. of the activation matrix (several mixes of one input; one
+                             // product per head). One weight matrix only
     float* out;              // [S, B, ld]; matrix m occupies columns col0 + m * N ..
     int ld, col0;            // row stride of `out` (>= n_mats * N) and first column written
     int* err;                // device flag, set non-zero if a bounded wait ran out
@@ -164,7 +167,7 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             const bool second = tg >= tiles_per_mat;
             wmap = second ? &map_w1 : &map_w;
             trow = (second ? tg - tiles_per_mat : tg) * kTcTileM;
-            xrow = (t % a.TB) * BN;
+            xrow = (t % a.TB) * BN + (a.seg_tiles > 0 ? tg / a.seg_tiles * a.B : 0);
         };
         auto advance = [&]() {
             if (++jr == nk) jr = 0;

@@ -198,6 +198,10 @@ class Gemma4CudaCacheTable:
     def reset(self):
         N.check(N.lib().oxg4_cache_reset(self._h))
 
+    def reset_sequence(self, b: int):
+        """Frees what sequence b holds: its pages and state slot can serve another request."""
+        N.check(N.lib().oxg4_cache_reset_sequence(self._h, b))
+
     def fill_synthetic(self, lens: Sequence[int]):
         """Measurement aid: marks lens[b] positions per sequence as cached and fills the K/V pools with a fixed
         pseudo-random pattern (timing only; the contents are not the K/V of any prompt)."""
@@ -308,6 +312,23 @@ class Gemma4CudaState:
             return None
         return out[0] if table.batch == 1 else out
 
+    def extend(self, tokens, table: Gemma4CudaCacheTable, lens=None, want=None):
+        """Feeds lens[b] further tokens of every sequence (back to back in `tokens`), which continue where their cache
+        and state stand. `want`: places in `tokens` whose logits are returned, [len(want), vocab], ascending."""
+        t = _as_u32(tokens).reshape(-1)
+        ln = np.ascontiguousarray([t.size] if lens is None else lens, dtype=np.int32)
+        if ln.size != table.batch or int(ln.sum()) != t.size:
+            raise Oxg4Error(2, "lens must name the tokens of every sequence of the table")
+        places = [] if want is None else list(want)
+        mark = np.zeros(max(t.size, 1), dtype=np.uint8)
+        mark[places] = 1
+        if places != sorted(set(places)):
+            raise Oxg4Error(2, "wanted places must be ascending")
+        out = np.empty((len(places), self.config.vocab_size), dtype=np.float32)
+        N.check(N.lib().oxg4_extend(self._h, table._h, _ptr(t), _ptr(ln), _ptr(mark) if places else None,
+                                    _ptr(out) if places else None))
+        return out
+
     def prefill_token(self, token, table: Gemma4CudaCacheTable):
         t = _as_u32(np.atleast_1d(token))
         N.check(N.lib().oxg4_prefill_token(self._h, table._h, _ptr(t)))
@@ -388,7 +409,8 @@ class Gemma4CudaState:
                                             repetition_penalty, _ptr(s), _ptr(out), C.byref(ms)))
         return out, s, ms.value
 
-    PROFILE_KINDS = ["qkv", "qkv_post", "attn", "attn_merge", "o", "gateup", "down", "lmhead", "norm", "geglu", "sum",
+    PROFILE_KINDS = ["qkv", "shift", "decay", "recur", "outnorm", "latent", "uq", "latsplit", "latq", "latmerge", "latuv", "latout",
+                     "qkv_post", "attn", "attn_merge", "o", "gateup", "down", "lmhead", "norm", "geglu", "sum",
                      "topk1", "topk2", "tp_pick", "allreduce", "allgather", "step_begin", "step_end"]
 
     def profile_step(self, tokens, table: Gemma4CudaCacheTable, totals: bool = False) -> dict:

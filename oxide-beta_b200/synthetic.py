@@ -219,21 +219,103 @@ def write_checkpoint(directory: str, cfg: dict, weights, dtype: str):
             f.write(b)
 
 
-def read_checkpoint(directory: str):
-    """Returns (text_config, {canonical name: memory-mapped array}). BF16 comes back as uint16."""
-    with open(os.path.join(directory, "config.json")) as f:
-        cfg = json.load(f)
-    cfg = cfg.get("text_config", cfg)
-    path = os.path.join(directory, "model.safetensors")
+def write_tensors(path: str, weights):
+    """One safetensors file: uint16 arrays are BF16 bit patterns, the rest is stored as F32."""
+    header, blobs, off = {}, [], 0
+    for name, a in weights:
+        a = np.ascontiguousarray(a)
+        header[name] = {"dtype": "BF16" if a.dtype == np.uint16 else "F32", "shape": list(a.shape),
+                        "data_offsets": [off, off + a.nbytes]}
+        blobs.append(a.tobytes())
+        off += a.nbytes
+    hj = json.dumps(header, separators=(",", ":")).encode()
+    hj += b" " * ((8 - len(hj) % 8) % 8)
+    with open(path, "wb") as f:
+        f.write(struct.pack("<Q", len(hj)))
+        f.write(hj)
+        for b in blobs:
+            f.write(b)
+
+
+def read_tensors(path: str):
+    """{name: memory-mapped array} of a safetensors file. BF16 comes back as uint16."""
     with open(path, "rb") as f:
         (hl,) = struct.unpack("<Q", f.read(8))
         header = json.loads(f.read(hl))
     mm = np.memmap(path, dtype=np.uint8, mode="r", offset=8 + hl)
     out = {}
     for name, meta in header.items():
-        if name == "__metadata__" or not name.startswith(PREFIX):
-            continue   # gemma4_cuda/mod.rs:236-243: only the language-model tensors are taken
+        if name == "__metadata__" or meta["dtype"] not in _ST_DTYPE:
+            continue
         np_dtype, _ = _ST_DTYPE[meta["dtype"]]
         a, b = meta["data_offsets"]
-        out[name[len(PREFIX):]] = mm[a:b].view(np_dtype).reshape(meta["shape"])
-    return cfg, out
+        # a copy where the file does not keep the element type's alignment
+        raw = mm[a:b] if (8 + hl + a) % np.dtype(np_dtype).itemsize == 0 else np.array(mm[a:b])
+        out[name] = raw.view(np_dtype).reshape(meta["shape"])
+    return out
+
+
+def read_config(directory: str) -> dict:
+    with open(os.path.join(directory, "config.json")) as f:
+        return json.load(f)
+
+
+def read_checkpoint(directory: str):
+    """Returns (text_config, {canonical name: memory-mapped array}). BF16 comes back as uint16."""
+    cfg = read_config(directory)
+    tensors = read_tensors(os.path.join(directory, "model.safetensors"))
+    # gemma4_cuda/mod.rs:236-243: only the language-model tensors are taken
+    return cfg.get("text_config", cfg), {n[len(PREFIX):]: a for n, a in tensors.items() if n.startswith(PREFIX)}
+
+
+# ---- models of listed layers (pabovik.py) ------------------------------------------------------
+
+def layered_weight_names(cfg: dict, low_rank: int = 16):
+    """(name, shape, kind) of every tensor. kind: 'matrix' | 'norm' | 'mu' | 'w0' | 'u'."""
+    H, out = cfg["width"], [("embed", (cfg["vocab"], cfg["width"]), "matrix")]
+    for i, layer in enumerate(cfg["layers"]):
+        if layer.get("weights_of") is not None:
+            continue
+        p, c = f"l{i}.", layer["mixer"]
+        heads, dim = c["heads"], c["dim"]
+        hd, ow = heads * dim, heads * c.get("vdim", dim)
+        out += [(p + "norm1", (H,), "norm"), (p + "norm1b", (H,), "norm")]
+        if layer["type"] == "wkv":
+            out += [(p + "mix.mu." + s, (H,), "mu") for s in "rkvgw"]
+            out += [(p + "mix." + s, (hd, H), "matrix") for s in "rkvg"]
+            out += [(p + "mix.w1", (low_rank, H), "matrix"), (p + "mix.w2", (hd, low_rank), "matrix"), (p + "mix.w0", (hd,), "w0"),
+                    (p + "mix.u", (heads, dim), "u"), (p + "mix.norm", (hd,), "norm")]
+        elif layer["type"] == "lightning":
+            out += [(p + "mix.q", (hd, H), "matrix"), (p + "mix.k", (hd, H), "matrix"), (p + "mix.v", (ow, H), "matrix"),
+                    (p + "mix.g", (ow, H), "matrix"), (p + "mix.norm", (ow,), "norm")]
+        else:
+            rank, rot = c["kv_rank"], c["rot_dim"]
+            out += [(p + "mix.dq", (c["q_rank"], H), "matrix"), (p + "mix.dq.norm", (c["q_rank"],), "norm"),
+                    (p + "mix.uq", (heads * (dim + rot), c["q_rank"]), "matrix"), (p + "mix.dkv", (rank + rot, H), "matrix"),
+                    (p + "mix.dkv.norm", (rank,), "norm"), (p + "mix.uk", (hd, rank), "matrix"),
+                    (p + "mix.uv", (ow, rank), "matrix"), (p + "mix.g", (ow, H), "matrix")]
+        out.append((p + "mix.o", (H, ow), "matrix"))
+        if layer.get("mlp"):
+            ff = layer["mlp"]["ff"]
+            out += [(p + "norm2", (H,), "norm"), (p + "norm2b", (H,), "norm"), (p + "mlp.gate", (ff, H), "matrix"),
+                    (p + "mlp.up", (ff, H), "matrix"), (p + "mlp.down", (H, ff), "matrix")]
+    return out + [("final.norm", (H,), "norm"), ("head", (cfg["vocab"], H), "matrix")]
+
+
+def layered_weights(cfg: dict, seed: int = 0, low_rank: int = 16, gain: float = 1.0):
+    """Yields (name, BF16 bit pattern array): matrices N(0, gain^2 / columns), norm weights around 1, shift mixes in
+    [0, 1], decay offsets that spread the decays between fast and slow channels."""
+    rng = np.random.default_rng(seed)
+    for name, shape, kind in layered_weight_names(cfg, low_rank):
+        a = rng.standard_normal(shape, dtype=np.float32)
+        if kind == "matrix":
+            a *= np.float32(gain if name == "embed" else gain / np.sqrt(shape[1]))
+        elif kind == "norm":
+            a = 1.0 + 0.2 * a
+        elif kind == "mu":
+            a = rng.random(shape, dtype=np.float32)
+        elif kind == "w0":
+            a = rng.uniform(-6.0, 0.5, shape).astype(np.float32)
+        else:
+            a *= np.float32(0.5)
+        yield name, f32_to_bf16_bits(a.astype(np.float32)).reshape(shape)
