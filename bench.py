@@ -281,7 +281,14 @@ def main():
                          "ingesting the prompts (decode timing at long contexts without the prefill time)")
     ap.add_argument("--layers", type=int, default=None, help="profiling aid: keep only the first LAYERS layers")
     ap.add_argument("--vocab", type=int, default=None, help="profiling aid: shrink the vocabulary")
+    ap.add_argument("--design", default=None, choices=["pabovik"],
+                    help="instead of the workload: prefill and decode throughput and per-kernel times of this design at a few "
+                         "sizes, beside a Gemma 4 model of equal width, depth and feed-forward (bench_layered.py)")
     args = ap.parse_args()
+    if args.design:
+        import bench_layered
+        bench_layered.main(args.design)
+        return
     warmup = max(args.warmup, 3)
 
     rank = int(os.environ.get("RANK", "0"))

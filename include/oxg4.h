@@ -272,6 +272,8 @@ int64_t oxg4_kernel_launches(const oxg4_model* model);
  * around every kernel and every tensor-parallel collective. Measurement aid in the role of the
  * reference's GEMMA4_PROFILE hook (crates/oxide-torch-models/examples/gemma4_load.rs:277-284). */
 int32_t oxg4_profile_step(oxg4_model* model, oxg4_cache* cache, const uint32_t* tokens);
+/* The same for portions of prompts (arguments as in oxg4_extend): the kinds then cover every chunk of the call. */
+int32_t oxg4_profile_extend(oxg4_model* model, oxg4_cache* cache, const uint32_t* tokens, const int32_t* lens);
 float oxg4_profile_ms(const oxg4_model* model, const char* kind);
 int32_t oxg4_profile_count(const oxg4_model* model, const char* kind);
 

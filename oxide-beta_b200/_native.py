@@ -114,6 +114,7 @@ SYMBOLS = {
                                        C.POINTER(C.c_float)]),
     "oxg4_kernel_launches": (C.c_int64, [C.c_void_p]),
     "oxg4_profile_step": (C.c_int32, [C.c_void_p, C.c_void_p, C.c_void_p]),
+    "oxg4_profile_extend": (C.c_int32, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p]),
     "oxg4_profile_ms": (C.c_float, [C.c_void_p, C.c_char_p]),
     "oxg4_profile_count": (C.c_int32, [C.c_void_p, C.c_char_p]),
     "oxg4_debug_wait_timeout": (C.c_int32, [C.c_void_p, C.c_void_p, C.c_int32, C.c_uint32]),

@@ -310,6 +310,9 @@ static int layered_splits(const oxg4_model* m, const Proj& p, int R, bool chunk)
     return tc_pick_splits(tiles, (p.K + kTcTileK - 1) / kTcTileK, m->num_sms, chunk ? kPrefillRows : R, n, p.K, chunk ? 1.0 : 0.3);
 }
 
+static int32_t latent_mma_setup(const MixPlan& x);
+constexpr int kLatentChunkSplits = 4;     // most splits of the visible positions in a prompt chunk
+
 static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
     oxg4_model* m = c->m;
     const int B = c->B, L = m->cfg.num_hidden_layers, H = m->H, R = c->rows_cap;
@@ -323,7 +326,7 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
         return n * std::max((size_t)layered_splits(m, p, B, false) * B, (size_t)layered_splits(m, p, kPrefillRows, true) * kPrefillRows);
     };
     size_t in_n = 1, o_n = 1, gu_n = 1, down_n = 1, q_n = 1, uk_n = 1, uv_n = 1, dec = 1, latq = 1, rh = 1, rh_rank = 1, xo = 1, xi = 1, xq = 1,
-           xu = 1, xl = 1, act = 1;
+           xu = 1, xl = 1, rot = 1, act = 1;
     bool any_shift = false;
     const int max_tiles = (*std::max_element(c->max_seq.begin(), c->max_seq.end()) + 63) / 64;
     c->lat_splits = std::max(1, std::min({max_tiles, 64, (2 * m->num_sms + B - 1) / B}));
@@ -355,6 +358,8 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
                 uv_n = std::max(uv_n, floats(x.uv));
                 xu = std::max(xu, (size_t)x.heads * x.uk.K);
                 xl = std::max(xl, (size_t)x.heads * x.uv.K);
+                rot = std::max(rot, (size_t)x.heads * x.rot);
+                TRY(latent_mma_setup(x));
             }
         } else {
             const size_t n = (size_t)B * x.heads * x.dim * x.vdim;
@@ -390,12 +395,12 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
     TRY(dalloc(c, &c->q_buf, q_n));
     TRY(bytes_alloc(&c->x_q, (size_t)R * xq * xes));
     TRY(dalloc(c, &c->lat_q, (size_t)R * latq));
+    TRY(dalloc(c, &c->lat_rot, (size_t)R * rot));
     TRY(dalloc(c, &c->uk_buf, uk_n));
     TRY(dalloc(c, &c->uv_buf, uv_n));
     TRY(bytes_alloc(&c->x_u, (size_t)R * xu * 2));
     TRY(bytes_alloc(&c->x_l, (size_t)R * xl * 2));
-    // split-KV partials: a decode step has B rows and up to lat_splits splits, a chunk 256 rows and up to kChunkSplits
-    const size_t part_rows = std::max((size_t)B * c->lat_splits, (size_t)R * 4);
+    const size_t part_rows = std::max((size_t)B * c->lat_splits, (size_t)R * kLatentChunkSplits);
     TRY(dalloc(c, &c->lat_o, part_rows * rh_rank));
     TRY(dalloc(c, &c->lat_ml, part_rows * rh * 2));
     return OXG4_OK;
@@ -422,6 +427,31 @@ static LatentAttnFn pick_latent_attn(int rank) {
     if (rank <= 128) return latent_attn_kernel<KT, 4>;
     if (rank <= 256) return latent_attn_kernel<KT, 8>;
     return latent_attn_kernel<KT, 16>;
+}
+
+typedef void (*LatentMmaFn)(const LatentMmaArgs);
+// the tensor-core kernel for `rows` (token, head) rows per run and cache rows of `ld` elements, null when it does not fit
+static LatentMmaFn pick_latent_mma(int rank, int ld, int rows, int* tile_rows, size_t* smem) {
+    LatentMmaFn fn;
+#define LM(MT, NB)                                                                                              \
+    {                                                                                                           \
+        fn = rank <= 128 ? latent_mma_kernel<MT, 2, NB> : rank <= 256 ? latent_mma_kernel<MT, 4, NB> : latent_mma_kernel<MT, 8, NB>; \
+        *tile_rows = MT * 16;                                                                                   \
+        *smem = latent_mma_smem<MT, NB>(ld);                                                                    \
+    }
+    if (rows <= 16) LM(1, 64) else if (rows <= 32) LM(2, 32) else LM(4, 32)
+#undef LM
+    return *smem <= 226 * 1024 ? fn : nullptr;
+}
+
+static int32_t latent_mma_setup(const MixPlan& x) {
+    for (int rows : {16, 32, 64}) {
+        int tr;
+        size_t smem;
+        LatentMmaFn fn = pick_latent_mma(x.rank, x.ld, rows, &tr, &smem);
+        if (fn) TRY(allow_big_smem(fn));
+    }
+    return OXG4_OK;
 }
 
 namespace {
@@ -652,10 +682,53 @@ struct LayeredPass {
             q = project("uq", x.uq, c->x_q, c->q_buf);
         }
         LatentPart part{c->lat_o, c->lat_ml, rs.chunk ? 1 : c->lat_splits, (size_t)R * x.heads};
+        int tile_rows = 0;
+        size_t mma_smem = 0;
+        int longest = 1;
+        for (int n : rs.run_len) longest = std::max(longest, n);
+        const LatentMmaFn mma = sizeof(WT) == 2 && sizeof(KT) == 2 ? pick_latent_mma(x.rank, x.ld, longest * x.heads, &tile_rows, &mma_smem) : nullptr;
+        LatentMmaArgs ma{};
+        int mma_tiles = 0;
+        if (mma) {
+            for (int n : rs.run_len) mma_tiles += (n * x.heads + tile_rows - 1) / tile_rows;
+            if (rs.chunk) {
+                // as many splits as fill the GPU in whole rounds
+                double best = 0.0;
+                for (int s = 1; s <= kLatentChunkSplits; ++s) {
+                    const double units = (double)mma_tiles * s, eff = units / (std::ceil(units / m->num_sms) * m->num_sms);
+                    if (eff > best + 0.05) { best = eff; part.splits = s; }
+                }
+            }
+            ma.heads = x.heads; ma.rank = x.rank; ma.rot = x.rot;
+            ma.scale = x.scale;
+            ma.rows = a.rows;
+            ma.runs = (int)rs.run_len.size();
+            ma.cache = a.cache;
+            ma.part = part;
+        }
+        if (mma && tc) {
+            // many rows: per-head products with W_uk^T and W_uv on the tensor cores
+            ln.go("latsplit", latent_split_query_kernel, dim3(R), dim3(256), 0, a, R, q, (uint16_t*)c->x_u, x.uk.K, c->lat_rot);
+            ln.tc("uk", c, R, x.uk.w, nullptr, (const uint16_t*)c->x_u, x.uk.N, x.uk.K, 1, c->uk_buf, x.uk.N, 0, x.uk.seg_rows / kTcTileM);
+            ma.q_abs = c->uk_buf; ma.abs_row = x.uk.N; ma.abs_head = x.uk.seg_rows;
+            ma.q_rot = c->lat_rot; ma.rot_row = (size_t)x.heads * x.rot; ma.rot_head = x.rot;
+            ln.go("attn", mma, dim3(mma_tiles, part.splits), dim3(kLmThreads), mma_smem, ma);
+            ln.go("latmerge", latent_merge_kernel, dim3(x.heads, R), dim3(128), sizeof(float) * part.splits, R, x.heads, x.rank, part,
+                  (uint16_t*)c->x_l, x.uv.K);
+            const SplitIn o = project("uv", x.uv, c->x_l, c->uv_buf);
+            output(x, o, x.vpad, 0, nullptr, in, ACT_SIGMOID);
+            return;
+        }
         ln.go("latq", latent_query_kernel<WT, KT>, dim3(x.heads + (fused ? 1 : 0), R, (x.rank + 255) / 256), dim3(256),
               sizeof(float) * (x.dim + x.rot), a, q, (const WT*)x.w_uk, c->lat_q, (int)fused);
-        LatentAttnFn fn = pick_latent_attn<KT>(x.rank);
-        ln.go("attn", fn, dim3(x.heads, R, part.splits), dim3(256), sizeof(float) * (x.rank + x.rot + 8 * x.rank + 16), a, (const float*)c->lat_q, part);
+        if (mma) {
+            ma.q_abs = c->lat_q; ma.abs_row = (size_t)x.heads * (x.rank + x.rot); ma.abs_head = x.rank + x.rot;
+            ma.q_rot = c->lat_q + x.rank; ma.rot_row = ma.abs_row; ma.rot_head = ma.abs_head;
+            ln.go("attn", mma, dim3(mma_tiles, part.splits), dim3(kLmThreads), mma_smem, ma);
+        } else {
+            LatentAttnFn fn = pick_latent_attn<KT>(x.rank);
+            ln.go("attn", fn, dim3(x.heads, R, part.splits), dim3(256), sizeof(float) * (x.rank + x.rot + 8 * x.rank + 16), a, (const float*)c->lat_q, part);
+        }
         ln.go("latout", latent_out_kernel<WT>, dim3(x.heads, R, (x.vdim + 31) / 32), dim3(256), sizeof(float) * (x.rank + part.splits), x.heads,
               x.rank, x.vdim, part, (const WT*)x.w_uv, x.rank, in, x.c_g, rs.tok, c->attn_out, x.owp);
         // the gate has been applied by the kernel that leaves latent space

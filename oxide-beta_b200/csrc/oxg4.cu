@@ -27,6 +27,7 @@
 #include "batch_ops.cuh"
 #include "tc_gemm.cuh"
 #include "layered_ops.cuh"
+#include "latent_mma.cuh"
 #include "tp.h"
 
 using namespace oxg4;
@@ -176,6 +177,7 @@ struct oxg4_model {
     std::vector<struct oxg4_cache*> caches;     // live cache tables: destroyed with the model if the caller has not
     std::map<std::string, ProfileSlot> profile;
     bool profiling = false;
+    bool profile_ingest = false;  // oxg4_profile_extend: chunks of prompts fill `profile` too
     std::vector<std::pair<std::string, std::pair<cudaEvent_t, cudaEvent_t>>> prof_events;
 };
 
@@ -765,6 +767,7 @@ struct oxg4_cache {
     void *mix_x = nullptr, *mix_y = nullptr, *x_q = nullptr, *x_u = nullptr, *x_l = nullptr;
     float *xf = nullptr, *in_buf = nullptr, *q_buf = nullptr, *uk_buf = nullptr, *uv_buf = nullptr, *wdec = nullptr, *lat_q = nullptr,
           *lat_o = nullptr, *lat_ml = nullptr;
+    float* lat_rot = nullptr;
     int lat_splits = 1;
 
     int32_t *dec_grp_row0 = nullptr, *dec_grp_n = nullptr;      // decode: one group per sequence
@@ -2326,6 +2329,20 @@ extern "C" int32_t oxg4_decode_sampled(oxg4_model* m, oxg4_cache* c, const uint3
     return OXG4_OK;
 }
 
+// adds the event pairs of the launches so far (all complete) to the per-kind totals
+static void collect_profile(oxg4_model* m) {
+    for (auto& pe : m->prof_events) {
+        float ms = 0;
+        cudaEventElapsedTime(&ms, pe.second.first, pe.second.second);
+        ProfileSlot& ps = m->profile[pe.first];
+        ps.ms += ms;
+        ps.count += 1;
+        cudaEventDestroy(pe.second.first);
+        cudaEventDestroy(pe.second.second);
+    }
+    m->prof_events.clear();
+}
+
 extern "C" int32_t oxg4_profile_step(oxg4_model* m, oxg4_cache* c, const uint32_t* tokens) {
     if (!m || !c || !tokens || c->m != m) return fail(OXG4_INVALID_ARGUMENT, "null or mismatched handle");
     TRY(bind_device(m));
@@ -2339,16 +2356,7 @@ extern "C" int32_t oxg4_profile_step(oxg4_model* m, oxg4_cache* c, const uint32_
     CK(cudaStreamSynchronize(m->stream));
     TRY(check_tc(c));
     m->profile.clear();
-    for (auto& pe : m->prof_events) {
-        float ms = 0;
-        cudaEventElapsedTime(&ms, pe.second.first, pe.second.second);
-        ProfileSlot& ps = m->profile[pe.first];
-        ps.ms += ms;
-        ps.count += 1;
-        cudaEventDestroy(pe.second.first);
-        cudaEventDestroy(pe.second.second);
-    }
-    m->prof_events.clear();
+    collect_profile(m);
     advance_host(c, tokens);
     return OXG4_OK;
 }
@@ -2696,7 +2704,7 @@ static int32_t ingest(oxg4_model* m, oxg4_cache* c, const uint32_t* tokens, cons
         CK(cudaMemcpyAsync(c->pf_run_row0, h_run0, sizeof(int32_t) * rs.run_len.size(), cudaMemcpyHostToDevice, st));
         CK(cudaMemcpyAsync(c->pf_run_n, h_runn, sizeof(int32_t) * rs.run_len.size(), cudaMemcpyHostToDevice, st));
         const bool prof = getenv("GEMMA4_PROFILE") != nullptr && getenv("OXG4_PROFILE_PREFILL") != nullptr;
-        m->profiling = prof;           // events around every launch of the chunk (a measurement aid, like the reference's GEMMA4_PROFILE)
+        m->profiling = prof || m->profile_ingest;           // events around every launch of the chunk (a measurement aid, like the reference's GEMMA4_PROFILE)
         Launcher ln{m};
         rs.R = R;
         rs.run_row0 = c->pf_run_row0;
@@ -2730,7 +2738,9 @@ static int32_t ingest(oxg4_model* m, oxg4_cache* c, const uint32_t* tokens, cons
         TRY(ln.status);
         m->launches += ln.kernels;
         CK(cudaStreamSynchronize(st));                         // the pinned staging is reused by the next chunk
-        if (prof) {
+        if (m->profile_ingest) {
+            collect_profile(m);
+        } else if (prof) {
             std::map<std::string, double> sum;
             for (auto& pe : m->prof_events) {
                 float ms = 0;
@@ -2791,6 +2801,16 @@ extern "C" int32_t oxg4_prefill(oxg4_model* m, oxg4_cache* c, const uint32_t* to
     std::vector<uint8_t> want((size_t)off[B], 0);
     for (int b = 0; b < B; ++b) want[off[b + 1] - 1] = 1;
     return ingest(m, c, tokens, lens, want.data(), last_logits);
+}
+
+extern "C" int32_t oxg4_profile_extend(oxg4_model* m, oxg4_cache* c, const uint32_t* tokens, const int32_t* lens) {
+    if (!m || !c || !tokens || !lens || c->m != m) return fail(OXG4_INVALID_ARGUMENT, "null or mismatched handle");
+    m->profile.clear();
+    m->prof_events.clear();
+    m->profile_ingest = true;
+    const int32_t s = ingest(m, c, tokens, lens, nullptr, nullptr);
+    m->profile_ingest = false;
+    return s;
 }
 
 // Portions of prompts: see ingest.

@@ -409,8 +409,8 @@ class Gemma4CudaState:
                                             repetition_penalty, _ptr(s), _ptr(out), C.byref(ms)))
         return out, s, ms.value
 
-    PROFILE_KINDS = ["qkv", "shift", "decay", "recur", "outnorm", "latent", "uq", "latsplit", "latq", "latmerge", "latuv", "latout",
-                     "qkv_post", "attn", "attn_merge", "o", "gateup", "down", "lmhead", "norm", "geglu", "sum",
+    PROFILE_KINDS = ["qkv", "shift", "decay", "recur", "outnorm", "latent", "uq", "latsplit", "uk", "latq", "latmerge", "uv",
+                     "latout", "qkv_post", "attn", "attn_merge", "o", "gateup", "down", "lmhead", "norm", "geglu", "sum",
                      "topk1", "topk2", "tp_pick", "allreduce", "allgather", "step_begin", "step_end"]
 
     def profile_step(self, tokens, table: Gemma4CudaCacheTable, totals: bool = False) -> dict:
@@ -418,6 +418,16 @@ class Gemma4CudaState:
         launch of every kind that ran, or with `totals` the ms per STEP of every kind (mean x launches)."""
         t = _as_u32(np.atleast_1d(tokens))
         N.check(N.lib().oxg4_profile_step(self._h, table._h, _ptr(t)))
+        return self._profile(totals)
+
+    def profile_extend(self, tokens, table: Gemma4CudaCacheTable, lens=None, totals: bool = False) -> dict:
+        """The same for portions of prompts: every launch of every chunk."""
+        t = _as_u32(tokens).reshape(-1)
+        ln = np.ascontiguousarray([t.size] if lens is None else lens, dtype=np.int32)
+        N.check(N.lib().oxg4_profile_extend(self._h, table._h, _ptr(t), _ptr(ln)))
+        return self._profile(totals)
+
+    def _profile(self, totals: bool) -> dict:
         out = {}
         for k in self.PROFILE_KINDS:
             n = N.lib().oxg4_profile_count(self._h, k.encode())
