@@ -44,7 +44,9 @@ inline size_t latent_mma_smem(int ld) {
     return (rows + 2 * NB) * ldp * 2 + 2 * rows * (NB + 8) * 2 + rows * (NB + 4) * 4 + 3 * rows * 4 + 64;
 }
 
-template <int MT, int NT, int NB>
+// KQ > 0: the query fragments of a warp's score tile stay in registers (KQ steps of 16 columns, rows of at most 16 KQ
+// elements), which leaves shared memory to the cache rows.
+template <int MT, int NT, int NB, int KQ>
 __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentMmaArgs a) {
     constexpr int ROWS = MT * 16;
     constexpr int SN = NB / 8;                       // score columns in MMA tiles
@@ -108,13 +110,16 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentM
     }
     const uint16_t* pool = (const uint16_t*)a.cache.pool;
     auto load_tile = [&](int tile, int stage) {
-        const int chunks = ld / 8;
-        for (int i = warp; i < NB; i += kLmWarps) {
-            const int p = tile * NB + i;
-            const bool ok = p < visible;
-            const uint16_t* src = pool + a.cache.row(seq, ok ? p : 0);
-            const uint32_t dst = smem_u32(skv + ((size_t)stage * NB + i) * ldp);
-            for (int c = lane; c < chunks; c += 32) cp_async16(dst + c * 16, src + c * 8, ok);
+        constexpr int RPW = NB / kLmWarps;                           // rows per warp; one lane looks up each row's page
+        const int chunks = ld / 8, p = tile * NB + warp * RPW + lane;
+        const bool mine = lane < RPW && p < visible;
+        const size_t off = mine ? a.cache.row(seq, p) : 0;
+        const unsigned valid = __ballot_sync(0xffffffffu, mine);
+        const uint32_t dst = smem_u32(skv + ((size_t)stage * NB + warp * RPW) * ldp);
+#pragma unroll
+        for (int i = 0; i < RPW; ++i) {
+            const uint16_t* src = pool + __shfl_sync(0xffffffffu, off, i);
+            for (int c = lane; c < chunks; c += 32) cp_async16(dst + i * ldp * 2 + c * 16, src + c * 8, (valid >> i) & 1);
         }
     };
     load_tile(tile0, 0);
@@ -141,6 +146,7 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentM
     const int s_mi = warp % MT, s_n0 = (warp / MT) * SPW;
     const uint32_t q_base = smem_u32(sq) + ((s_mi * 16 + (lane & 15)) * ldp + (lane >> 4) * 8) * 2;
     const int v_col0 = warp * NT * 8;
+    uint32_t qf[KQ > 0 ? KQ : 1][4];
     for (int tile = tile0; tile < tile1; ++tile) {
         const int stage = (tile - tile0) & 1;
         cp_async_wait<0>();
@@ -154,7 +160,29 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentM
             float s[SPW][4];
 #pragma unroll
             for (int j = 0; j < SPW; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
-            if constexpr (SPW == 1) {
+            if constexpr (SPW == 1 && KQ > 0) {
+                if (tile == tile0) {
+#pragma unroll
+                    for (int k = 0; k < KQ; ++k)
+                        if (k * 16 < ld) ldmatrix_x4(qf[k], q_base + k * 32);
+                }
+                const uint32_t kb = kv + ((s_n0 * 8 + (lane & 7)) * ldp + (lane >> 3) * 8) * 2;
+                float s2[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+                for (int k = 0; k < KQ; k += 2) {
+                    uint32_t b[4];
+                    if (k * 16 + 32 <= ld) {
+                        ldmatrix_x4(b, kb + k * 32);
+                        mma_bf16_16816(s[0], qf[k], b[0], b[1]);
+                        mma_bf16_16816(s2, qf[k + 1], b[2], b[3]);
+                    } else if (k * 16 < ld) {                        // ld is a multiple of 16
+                        ldmatrix_x4(b, kv + ((s_n0 * 8 + (lane & 7)) * ldp + ((lane >> 3) & 1) * 8 + k * 16) * 2);
+                        mma_bf16_16816(s[0], qf[k], b[0], b[1]);
+                    }
+                }
+#pragma unroll
+                for (int q = 0; q < 4; ++q) s[0][q] += s2[q];
+            } else if constexpr (SPW == 1) {
                 // one column tile: a load brings its 8 positions for two k-steps
                 const uint32_t kb = kv + ((s_n0 * 8 + (lane & 7)) * ldp + (lane >> 3) * 8) * 2;
                 float s2[4] = {0.0f, 0.0f, 0.0f, 0.0f};

@@ -329,7 +329,7 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
            xu = 1, xl = 1, rot = 1, act = 1;
     bool any_shift = false;
     const int max_tiles = (*std::max_element(c->max_seq.begin(), c->max_seq.end()) + 63) / 64;
-    c->lat_splits = std::max(1, std::min({max_tiles, 64, (2 * m->num_sms + B - 1) / B}));
+    c->lat_splits = std::max(1, std::min({max_tiles, 64, (4 * m->num_sms + B - 1) / B}));
     for (int l = 0; l < L; ++l) {
         const MixPlan& x = m->layers[l].mix;
         in_n = std::max(in_n, floats(x.in));
@@ -409,16 +409,23 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
 // ---- a pass over the layers -----------------------------------------------------------------------------------
 typedef void (*RecurFn)(const RecurArgs);
 template <int KIND, typename WT>
-static RecurFn pick_recur(int dim, int* ks, int* kpt) {
+static RecurFn pick_recur(int dim, bool step, int* ks, int* kpt) {
 #define PR(KS, KPT)                                    \
     if (dim <= KS * KPT) {                             \
         *ks = KS;                                      \
         *kpt = KPT;                                    \
-        return recur_kernel<KIND, WT, KS, KPT>;        \
+        return step ? recur_kernel<KIND, WT, KS, KPT, 1> : recur_kernel<KIND, WT, KS, KPT, rec_tile(KS * KPT)>; \
     }
     PR(4, 8) PR(8, 8) PR(8, 16) PR(16, 16) PR(32, 16)
 #undef PR
     return nullptr;
+}
+
+static int32_t group_norm_setup() {
+    TRY((allow_big_smem(group_norm_rows_kernel<uint16_t, 1>)));
+    TRY((allow_big_smem(group_norm_rows_kernel<uint16_t, 4>)));
+    TRY((allow_big_smem(group_norm_rows_kernel<float, 1>)));
+    return allow_big_smem(group_norm_rows_kernel<float, 4>);
 }
 
 typedef void (*LatentAttnFn)(const LatentArgs, const float*, LatentPart);
@@ -431,11 +438,14 @@ static LatentAttnFn pick_latent_attn(int rank) {
 
 typedef void (*LatentMmaFn)(const LatentMmaArgs);
 // the tensor-core kernel for `rows` (token, head) rows per run and cache rows of `ld` elements, null when it does not fit
-static LatentMmaFn pick_latent_mma(int rank, int ld, int rows, int* tile_rows, size_t* smem) {
+static LatentMmaFn pick_latent_mma(int rank, int ld, int rows, int* tile_rows, int* tile_pos, size_t* smem) {
     LatentMmaFn fn;
 #define LM(MT, NB)                                                                                              \
     {                                                                                                           \
-        fn = rank <= 128 ? latent_mma_kernel<MT, 2, NB> : rank <= 256 ? latent_mma_kernel<MT, 4, NB> : latent_mma_kernel<MT, 8, NB>; \
+        if (rank <= 128) fn = MT < 4 && ld <= 192 ? latent_mma_kernel<MT, 2, NB, MT < 4 ? 12 : 0> : latent_mma_kernel<MT, 2, NB, 0>;       \
+        else if (rank <= 256) fn = MT < 4 && ld <= 320 ? latent_mma_kernel<MT, 4, NB, MT < 4 ? 20 : 0> : latent_mma_kernel<MT, 4, NB, 0>;  \
+        else fn = MT < 4 && ld <= 576 ? latent_mma_kernel<MT, 8, NB, MT < 4 ? 36 : 0> : latent_mma_kernel<MT, 8, NB, 0>;                   \
+        *tile_pos = NB;                                                                                         \
         *tile_rows = MT * 16;                                                                                   \
         *smem = latent_mma_smem<MT, NB>(ld);                                                                    \
     }
@@ -446,12 +456,25 @@ static LatentMmaFn pick_latent_mma(int rank, int ld, int rows, int* tile_rows, s
 
 static int32_t latent_mma_setup(const MixPlan& x) {
     for (int rows : {16, 32, 64}) {
-        int tr;
+        int tr, tp;
         size_t smem;
-        LatentMmaFn fn = pick_latent_mma(x.rank, x.ld, rows, &tr, &smem);
+        LatentMmaFn fn = pick_latent_mma(x.rank, x.ld, rows, &tr, &tp, &smem);
         if (fn) TRY(allow_big_smem(fn));
     }
     return OXG4_OK;
+}
+
+// Splits of `tiles` cache tiles when `units` row tiles share the GPU: the cheapest number of rounds times tiles per CTA, with
+// about three tiles' worth of start-up per CTA and a little for every partial the merge has to read.
+static int latent_splits(int units, int tiles, int most, int num_sms) {
+    int best = 1;
+    double best_cost = 1e30;
+    for (int s = 1; s <= std::min(most, std::max(1, tiles)); ++s) {
+        const double rounds = (units * s + num_sms - 1) / num_sms;
+        const double cost = rounds * ((tiles + s - 1) / s + 3) + 0.05 * s;
+        if (cost < best_cost - 1e-9) { best_cost = cost; best = s; }
+    }
+    return best;
 }
 
 namespace {
@@ -537,10 +560,15 @@ struct LayeredPass {
 
     void group_norm(const GroupNormArgs& g, void* x, int ld_x) {
         const size_t smem = sizeof(float) * g.n;
-        if (ln.status == OXG4_OK && smem > 48 * 1024)
-            ln.status = m->es == 2 ? allow_big_smem(group_norm_rows_kernel<uint16_t>) : allow_big_smem(group_norm_rows_kernel<float>);
-        if (m->es == 2) ln.go("outnorm", group_norm_rows_kernel<uint16_t>, dim3(R), dim3(256), smem, g, (uint16_t*)x, ld_x);
-        else ln.go("outnorm", group_norm_rows_kernel<float>, dim3(R), dim3(256), smem, g, (float*)x, ld_x);
+        if (ln.status == OXG4_OK && smem > 48 * 1024) ln.status = group_norm_setup();
+        const bool vec = (g.n | g.hs | g.hs_ld | g.o.ld | g.gate.ld | g.c_gate | ld_x) % 4 == 0 && (g.o.stride | g.gate.stride) % 4 == 0;
+        if (m->es == 2) {
+            if (vec) ln.go("outnorm", group_norm_rows_kernel<uint16_t, 4>, dim3(R), dim3(256), smem, g, (uint16_t*)x, ld_x);
+            else ln.go("outnorm", group_norm_rows_kernel<uint16_t, 1>, dim3(R), dim3(256), smem, g, (uint16_t*)x, ld_x);
+        } else {
+            if (vec) ln.go("outnorm", group_norm_rows_kernel<float, 4>, dim3(R), dim3(256), smem, g, (float*)x, ld_x);
+            else ln.go("outnorm", group_norm_rows_kernel<float, 1>, dim3(R), dim3(256), smem, g, (float*)x, ld_x);
+        }
     }
 
     // output norm, gate and output projection of a mixer; o: raw head outputs
@@ -626,7 +654,7 @@ struct LayeredPass {
             a.u = x.u;
             a.c_low = x.c_low; a.rank = x.low_rank; a.w2 = x.w2; a.w0 = x.w0;
             a.shift_src = c->xf; a.shift_dst = c->shift[l]; a.shift_n = H;
-            if (rs.chunk) {
+            if (!fused) {
                 const int N = x.heads * x.dim;
                 const dim3 grid((N + 255) / 256, (R + kDecayRows - 1) / kDecayRows);
                 const size_t smem = sizeof(float) * kDecayRows * x.low_rank;
@@ -641,10 +669,11 @@ struct LayeredPass {
         }
         int ks = 1, kpt = 1;
         RecurFn fn;
-        if (wkv) fn = m->es == 2 ? pick_recur<REC_WKV, uint16_t>(x.dim, &ks, &kpt) : pick_recur<REC_WKV, float>(x.dim, &ks, &kpt);
-        else fn = pick_recur<REC_LIGHTNING, float>(x.dim, &ks, &kpt);
-        const int vs = kRecThreads / ks, dp = ks * kpt;
-        const size_t smem = sizeof(float) * ((size_t)kRecTile * dp * (wkv ? 3 : 2) + kRecTile * vs + kRecTile + (wkv ? x.low_rank : 0));
+        const bool step = !rs.chunk;
+        if (wkv) fn = m->es == 2 ? pick_recur<REC_WKV, uint16_t>(x.dim, step, &ks, &kpt) : pick_recur<REC_WKV, float>(x.dim, step, &ks, &kpt);
+        else fn = pick_recur<REC_LIGHTNING, float>(x.dim, step, &ks, &kpt);
+        const int vs = kRecThreads / ks, dp = ks * kpt, tile = step ? 1 : rec_tile(dp);
+        const size_t smem = sizeof(float) * ((step ? 1 : 2) * ((size_t)tile * dp * (wkv ? 3 : 2) + tile * vs + pad_to(tile, 4)) + (wkv ? x.low_rank : 0));
         if (ln.status == OXG4_OK && smem > 48 * 1024) ln.status = allow_big_smem(fn);
         ln.go("recur", fn, dim3(x.heads, (x.vdim + vs - 1) / vs, (unsigned)rs.run_len.size()), dim3(kRecThreads), smem, a);
         output(x, one(c->attn_out, x.owp), x.vdim, wkv ? x.dim : x.ow, x.out_norm, in, wkv ? ACT_SILU : ACT_SIGMOID);
@@ -682,23 +711,17 @@ struct LayeredPass {
             q = project("uq", x.uq, c->x_q, c->q_buf);
         }
         LatentPart part{c->lat_o, c->lat_ml, rs.chunk ? 1 : c->lat_splits, (size_t)R * x.heads};
-        int tile_rows = 0;
+        int tile_rows = 0, tile_pos = 1;
         size_t mma_smem = 0;
         int longest = 1;
         for (int n : rs.run_len) longest = std::max(longest, n);
-        const LatentMmaFn mma = sizeof(WT) == 2 && sizeof(KT) == 2 ? pick_latent_mma(x.rank, x.ld, longest * x.heads, &tile_rows, &mma_smem) : nullptr;
+        const LatentMmaFn mma = sizeof(WT) == 2 && sizeof(KT) == 2 ? pick_latent_mma(x.rank, x.ld, longest * x.heads, &tile_rows, &tile_pos, &mma_smem) : nullptr;
         LatentMmaArgs ma{};
         int mma_tiles = 0;
         if (mma) {
             for (int n : rs.run_len) mma_tiles += (n * x.heads + tile_rows - 1) / tile_rows;
-            if (rs.chunk) {
-                // as many splits as fill the GPU in whole rounds
-                double best = 0.0;
-                for (int s = 1; s <= kLatentChunkSplits; ++s) {
-                    const double units = (double)mma_tiles * s, eff = units / (std::ceil(units / m->num_sms) * m->num_sms);
-                    if (eff > best + 0.05) { best = eff; part.splits = s; }
-                }
-            }
+            part.splits = latent_splits(mma_tiles, (rs.max_visible + tile_pos - 1) / tile_pos, rs.chunk ? kLatentChunkSplits : c->lat_splits,
+                                        m->num_sms);
             ma.heads = x.heads; ma.rank = x.rank; ma.rot = x.rot;
             ma.scale = x.scale;
             ma.rows = a.rows;
@@ -719,8 +742,8 @@ struct LayeredPass {
             output(x, o, x.vpad, 0, nullptr, in, ACT_SIGMOID);
             return;
         }
-        ln.go("latq", latent_query_kernel<WT, KT>, dim3(x.heads + (fused ? 1 : 0), R, (x.rank + 255) / 256), dim3(256),
-              sizeof(float) * (x.dim + x.rot), a, q, (const WT*)x.w_uk, c->lat_q, (int)fused);
+        ln.go("latq", latent_query_kernel<WT, KT>, dim3(x.heads + (fused ? 1 : 0), R, (x.rank + kLqCols - 1) / kLqCols), dim3(256),
+              sizeof(float) * (x.dim + x.rot + 256), a, q, (const WT*)x.w_uk, c->lat_q, (int)fused);
         if (mma) {
             ma.q_abs = c->lat_q; ma.abs_row = (size_t)x.heads * (x.rank + x.rot); ma.abs_head = x.rank + x.rot;
             ma.q_rot = c->lat_q + x.rank; ma.rot_row = ma.abs_row; ma.rot_head = ma.abs_head;

@@ -8,6 +8,7 @@
 // BF16 projection. "Split input": the consumer of a tcgen05 projection adds its K-split partials itself, in split
 // order, so every reader takes (pointer, number of splits, distance between splits).
 #pragma once
+#include "batch_ops.cuh"
 #include "common.cuh"
 #include "gemv.cuh"
 
@@ -73,16 +74,8 @@ shift_mix_kernel(int R, int H, int S, const float* h, const float* state, const 
 }
 
 // ---- per-channel decay of the time mixing -------------------------------------------------------------------
-// w[n] = exp(-exp(W2[n, :] . tanh(low) + w0[n]))
-template <typename WT>
-DEVINL float channel_decay(const WT* w2_row, const float* tanh_low, int rank, float w0) {
-    float t = w0;
-    for (int j = 0; j < rank; ++j) t = fmaf(WTraits<WT>::elem(w2_row, j), tanh_low[j], t);
-    return expf(-expf(t));
-}
-
 constexpr int kDecayRows = 8;
-// out[r, n] for R rows and N channels; grid (ceil(N / 256), ceil(R / 8)), dynamic shared memory 8 * rank floats
+// out[r, n] = exp(-exp(W2[n, :] . tanh(low[r, :]) + w0[n])) for R rows and N channels; grid (ceil(N / 256), ceil(R / 8)), dynamic shared memory 8 * rank floats
 template <typename WT>
 __global__ void __launch_bounds__(256)
 wkv_decay_kernel(int R, int N, int rank, SplitIn low, int col, const WT* w2, const float* w0, float* out) {
@@ -91,18 +84,32 @@ wkv_decay_kernel(int R, int N, int rank, SplitIn low, int col, const WT* w2, con
     pdl_wait();
     pdl_launch();
     const int r0 = blockIdx.y * kDecayRows, nr = min(kDecayRows, R - r0);
-    for (int i = threadIdx.x; i < nr * rank; i += blockDim.x) th[i] = tanhf(low.at(r0 + i / rank, col + i % rank));
+    for (int i = threadIdx.x; i < kDecayRows * rank; i += blockDim.x)
+        th[i] = i / rank < nr ? tanhf(low.at(r0 + i / rank, col + i % rank)) : 0.0f;
     __syncthreads();
     const int n = blockIdx.x * 256 + threadIdx.x;
     if (n >= N) return;
     float t[kDecayRows];
 #pragma unroll
     for (int q = 0; q < kDecayRows; ++q) t[q] = w0[n];
-    for (int j = 0; j < rank; ++j) {
-        const float w = WTraits<WT>::elem(w2, (size_t)n * rank + j);
+    constexpr int EPL = WTraits<WT>::EPL;
+    if (rank % EPL == 0) {               // rows of W2 are whole 16-byte pieces
+#pragma unroll 2
+        for (int j = 0; j < rank; j += EPL) {
+            const uint4 p = *reinterpret_cast<const uint4*>(w2 + (size_t)n * rank + j);
 #pragma unroll
-        for (int q = 0; q < kDecayRows; ++q)
-            if (q < nr) t[q] = fmaf(w, th[q * rank + j], t[q]);
+            for (int e = 0; e < EPL; ++e) {
+                const float w = WTraits<WT>::elem(&p, e);
+#pragma unroll
+                for (int q = 0; q < kDecayRows; ++q) t[q] = fmaf(w, th[q * rank + j + e], t[q]);
+            }
+        }
+    } else {
+        for (int j = 0; j < rank; ++j) {
+            const float w = WTraits<WT>::elem(w2, (size_t)n * rank + j);
+#pragma unroll
+            for (int q = 0; q < kDecayRows; ++q) t[q] = fmaf(w, th[q * rank + j], t[q]);
+        }
     }
 #pragma unroll
     for (int q = 0; q < kDecayRows; ++q)
@@ -116,11 +123,11 @@ wkv_decay_kernel(int R, int N, int rank, SplitIn low, int col, const WT* w2, con
 // The bonus term is v * sum_k r_k u_k k_k, one scalar per token and head.
 // Grid (heads, slices of vdim, runs). A thread owns KPT consecutive key channels of one value column; the KS threads
 // that share a column are neighbouring lanes. Tokens are staged in shared memory in tiles, activations applied on
-// the way; the dot products of 8 tokens are reduced across the KS lanes together.
+// the way; the dot products of up to 8 tokens are reduced across the KS lanes together.
 // State in memory: [sequence][head][vdim][dim]. At position 0 the state starts at zero whatever the memory holds.
 enum { REC_LIGHTNING = 0, REC_WKV = 1 };
 constexpr int kRecThreads = 256;
-constexpr int kRecTile = 16;             // tokens staged at a time
+constexpr int rec_tile(int dp) { return dp <= 128 ? 16 : dp <= 256 ? 8 : 4; }   // tokens staged at a time
 
 struct RecurArgs {
     SplitIn in;                          // fused input projection
@@ -142,89 +149,142 @@ struct RecurArgs {
     int shift_n;
 };
 
-template <int KIND, typename WT, int KS, int KPT>
-__global__ void __launch_bounds__(kRecThreads) recur_kernel(const RecurArgs a) {
+// Sums acc[0 .. N) over the KS neighbouring lanes of a column, halving the tokens a lane keeps at every step: lane ks ends
+// with the totals of tokens `first` .. `first + left - 1` in acc[0 .. left), left = max(1, N / KS).
+template <int N, int KS>
+DEVINL void column_reduce(float (&acc)[N], int ks, int& first) {
+    int left = N;
+    first = 0;
+#pragma unroll
+    for (int o = KS / 2; o > 0; o >>= 1) {
+        if (left > 1) {
+            left /= 2;
+            const bool up = (ks & o) != 0;
+#pragma unroll
+            for (int t = 0; t < N / 2; ++t)
+                if (t < left) {
+                    const float keep = up ? acc[t + left] : acc[t], send = up ? acc[t] : acc[t + left];
+                    acc[t] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                }
+            if (up) first += left;
+        } else {
+            acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], o);
+        }
+    }
+}
+
+// TILE: tokens staged at a time; 1 for decode steps (runs of one token). Tiles of longer runs are double-buffered: the next
+// tile's values are fetched into registers while the current one is walked.
+template <int KIND, typename WT, int KS, int KPT, int TILE>
+__global__ void __launch_bounds__(kRecThreads, 2) recur_kernel(const RecurArgs a) {
+    constexpr bool WKV = KIND == REC_WKV;
     constexpr int DP = KS * KPT;         // key channels, padded
     constexpr int VS = kRecThreads / KS; // value columns of this CTA
+    constexpr int NK = (TILE * DP + kRecThreads - 1) / kRecThreads, NV = (TILE * VS + kRecThreads - 1) / kRecThreads;
+    constexpr int TB = TILE < 8 ? TILE : 8;
+    constexpr int TPAD = (TILE + 3) / 4 * 4;
+    constexpr int BUF = TILE * DP * (WKV ? 3 : 2) + TILE * VS + TPAD;
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    float* sq = reinterpret_cast<float*>(smem_raw);          // [tile][DP]
-    float* sk = sq + kRecTile * DP;
-    float* sw = sk + kRecTile * DP;                          // WKV only
-    float* sv = sw + (KIND == REC_WKV ? kRecTile * DP : 0);  // [tile][VS]
-    float* sb = sv + kRecTile * VS;                          // [tile] bonus (WKV)
+    float* bufs = reinterpret_cast<float*>(smem_raw);        // [2 (1 for TILE 1)][q | k | w (WKV) | v | bonus (WKV)]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int hd = blockIdx.x, v0 = blockIdx.y * VS, run = blockIdx.z;
     const int ks = tid % KS, vc = tid / KS, v = v0 + vc;
+    const int hk = hd * a.dim, hv = hd * a.vdim;
     pdl_wait();
     pdl_launch();
-    const int row0 = a.rows.row0[run], n = a.rows.n[run];
-    if (a.rows.tok[row0] == kInactiveToken) return;
+    const int row0 = a.rows.row0[run], n = TILE == 1 ? 1 : a.rows.n[run];
     const int seq = a.rows.seq_of(row0);
-    const bool fresh = a.rows.pos[row0] == 0;
+    const bool have_v = v < a.vdim;
+    float* st = a.state + (((size_t)seq * a.heads + hd) * a.vdim + v) * a.dim;
+    float S[KPT];
+    if (KPT % 4 == 0 && a.dim % 4 == 0) {
+#pragma unroll
+        for (int i = 0; i < KPT; i += 4) {
+            const int k = ks * KPT + i;
+            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (have_v && k < a.dim) x = *reinterpret_cast<const float4*>(st + k);
+            S[i] = x.x; S[i + 1] = x.y; S[i + 2] = x.z; S[i + 3] = x.w;
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < KPT; ++i) S[i] = (have_v && ks * KPT + i < a.dim) ? st[ks * KPT + i] : 0.0f;
+    }
+    if (a.rows.tok[row0] == kInactiveToken) return;
+    if (a.rows.pos[row0] == 0) {
+#pragma unroll
+        for (int i = 0; i < KPT; ++i) S[i] = 0.0f;
+    }
     if (a.shift_src != nullptr && hd == 0 && blockIdx.y == 0)
         for (int i = tid; i < a.shift_n; i += kRecThreads)
             a.shift_dst[(size_t)seq * a.shift_n + i] = a.shift_src[(size_t)(row0 + n - 1) * a.shift_n + i];
-    float* st = a.state + (((size_t)seq * a.heads + hd) * a.vdim + v) * a.dim;
-    const bool have_v = v < a.vdim;
-    float S[KPT];
+    const float dh = WKV ? 0.0f : a.decay[hd];
+
+    float fq[NK], fk[NK], fw[WKV ? NK : 1], fv[NV];
+    auto fetch = [&](int t0) {           // values of the tile at t0, zero past the run and past the key channels
 #pragma unroll
-    for (int i = 0; i < KPT; ++i) {
-        const int k = ks * KPT + i;
-        S[i] = (!fresh && have_v && k < a.dim) ? st[k] : 0.0f;
-    }
-    const float dh = KIND == REC_LIGHTNING ? a.decay[hd] : 0.0f;
-    const int hk = hd * a.dim, hv = hd * a.vdim;
-    for (int t0 = 0; t0 < n; t0 += kRecTile) {
-        const int nt = min(kRecTile, n - t0);
+        for (int j = 0; j < NK; ++j) {
+            const int i = tid + j * kRecThreads, t = t0 + i / DP, k = i % DP;
+            const bool ok = i < TILE * DP && t < n && k < a.dim;
+            fq[j] = ok ? a.in.at(row0 + t, a.c_q + hk + k) : 0.0f;
+            fk[j] = ok ? a.in.at(row0 + t, a.c_k + hk + k) : 0.0f;
+            if constexpr (WKV) fw[j] = ok && a.w != nullptr ? a.w[(size_t)(row0 + t) * a.heads * a.dim + hk + k] : 0.0f;
+        }
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = tid + j * kRecThreads, t = t0 + i / VS, c = v0 + i % VS;
+            fv[j] = (i < TILE * VS && t < n && c < a.vdim) ? a.in.at(row0 + t, a.c_v + hv + c) : 0.0f;
+        }
+    };
+    fetch(0);
+    int parity = 0;
+    for (int t0 = 0; t0 < n; t0 += TILE) {
+        const int nt = min(TILE, n - t0);
+        float* sq = bufs + parity * BUF;
+        float *sk = sq + TILE * DP, *sw = sk + TILE * DP, *sv = sw + (WKV ? TILE * DP : 0), *sb = sv + TILE * VS;
+#pragma unroll
+        for (int j = 0; j < NK; ++j) {
+            const int i = tid + j * kRecThreads;
+            if (i < TILE * DP) {
+                sq[i] = WKV ? fq[j] : silu(fq[j]);
+                sk[i] = WKV ? fk[j] : silu(fk[j]);
+                if constexpr (WKV) sw[i] = fw[j];
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = tid + j * kRecThreads;
+            if (i < TILE * VS) sv[i] = WKV ? fv[j] : silu(fv[j]);
+        }
+        if (t0 + TILE < n) fetch(t0 + TILE);
         __syncthreads();
-        for (int i = tid; i < kRecTile * DP; i += kRecThreads) {
-            const int t = i / DP, k = i % DP;
-            float q = 0.0f, kk = 0.0f, w = 0.0f;
-            if (t < nt && k < a.dim) {
-                const int r = row0 + t0 + t;
-                q = a.in.at(r, a.c_q + hk + k);
-                kk = a.in.at(r, a.c_k + hk + k);
-                if constexpr (KIND == REC_LIGHTNING) {
-                    q = silu(q);
-                    kk = silu(kk);
-                } else if (a.w != nullptr) {
-                    w = a.w[(size_t)r * a.heads * a.dim + hk + k];
-                }
-            }
-            sq[i] = q;
-            sk[i] = kk;
-            if constexpr (KIND == REC_WKV) sw[i] = w;
-        }
-        for (int i = tid; i < kRecTile * VS; i += kRecThreads) {
-            const int t = i / VS, c = v0 + i % VS;
-            float x = 0.0f;
-            if (t < nt && c < a.vdim) {
-                x = a.in.at(row0 + t0 + t, a.c_v + hv + c);
-                if constexpr (KIND == REC_LIGHTNING) x = silu(x);
-            }
-            sv[i] = x;
-        }
-        if constexpr (KIND == REC_WKV) {
-            if (a.w == nullptr) {                            // one-token run: decay of this head's channels
-                float* th = sb + kRecTile;                   // [rank]
+        if constexpr (WKV) {
+            if (TILE == 1 && a.w == nullptr) {               // decay of this head's channels, four lanes per channel
+                float* th = sb + TPAD;                       // [rank]
                 for (int j = tid; j < a.rank; j += kRecThreads) th[j] = tanhf(a.in.at(row0, a.c_low + j));
                 __syncthreads();
-                for (int k = tid; k < a.dim; k += kRecThreads)
-                    sw[k] = channel_decay((const WT*)a.w2 + (size_t)(hk + k) * a.rank, th, a.rank, a.w0[hk + k]);
+                for (int k0 = 0; k0 < a.dim; k0 += kRecThreads / 4) {
+                    const int k = k0 + (tid >> 2);
+                    float t = 0.0f;
+                    if (k < a.dim)
+#pragma unroll 8
+                        for (int j = tid & 3; j < a.rank; j += 4) t = fmaf(WTraits<WT>::elem(a.w2, (size_t)(hk + k) * a.rank + j), th[j], t);
+                    t += __shfl_xor_sync(0xffffffffu, t, 1);
+                    t += __shfl_xor_sync(0xffffffffu, t, 2);
+                    if (k < a.dim && (tid & 3) == 0) sw[k] = expf(-expf(t + a.w0[hk + k]));
+                }
             }
-            __syncthreads();
             for (int t = warp; t < nt; t += kRecThreads / 32) {
                 float b = 0.0f;
                 for (int k = lane; k < a.dim; k += 32) b += sq[t * DP + k] * a.u[hk + k] * sk[t * DP + k];
                 b = warp_sum(b);
                 if (lane == 0) sb[t] = b;
             }
+            __syncthreads();
         }
-        __syncthreads();
-        for (int tb = 0; tb < nt; tb += 8) {
-            float acc[8];
+        for (int tb = 0; tb < nt; tb += TB) {
+            float acc[TB];
 #pragma unroll
-            for (int t = 0; t < 8; ++t) {
+            for (int t = 0; t < TB; ++t) {
                 acc[t] = 0.0f;
                 if (tb + t >= nt) continue;
                 const float* q = sq + (tb + t) * DP + ks * KPT;
@@ -235,7 +295,7 @@ __global__ void __launch_bounds__(kRecThreads) recur_kernel(const RecurArgs a) {
 #pragma unroll
                 for (int i = 0; i < KPT; i += 4) {
                     const float4 q4 = *reinterpret_cast<const float4*>(q + i), k4 = *reinterpret_cast<const float4*>(k + i);
-                    if constexpr (KIND == REC_LIGHTNING) {
+                    if constexpr (!WKV) {
                         S[i] = fmaf(dh, S[i], k4.x * x); s = fmaf(q4.x, S[i], s);
                         S[i + 1] = fmaf(dh, S[i + 1], k4.y * x); s = fmaf(q4.y, S[i + 1], s);
                         S[i + 2] = fmaf(dh, S[i + 2], k4.z * x); s = fmaf(q4.z, S[i + 2], s);
@@ -250,28 +310,34 @@ __global__ void __launch_bounds__(kRecThreads) recur_kernel(const RecurArgs a) {
                 }
                 acc[t] = s;
             }
+            int first;
+            column_reduce<TB, KS>(acc, ks, first);
+            constexpr int LEFT = TB / KS > 0 ? TB / KS : 1;
+            // with more lanes than tokens the lanes that differ in the low bits hold the same total: one of them stores
+            const bool owner = KS <= TB || ks % (KS / TB > 0 ? KS / TB : 1) == 0;
+            if (have_v && owner) {
 #pragma unroll
-            for (int t = 0; t < 8; ++t) {
-#pragma unroll
-                for (int o = KS / 2; o > 0; o >>= 1) acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], o);
-            }
-            // lane ks of a column stores tokens ks, ks + KS, ...
-            if (have_v) {
-#pragma unroll
-                for (int t = 0; t < 8; ++t)
-                    if ((t % KS) == ks && tb + t < nt) {
+                for (int t = 0; t < LEFT; ++t) {
+                    const int tt = tb + first + t;
+                    if (tt < nt) {
                         float o = acc[t];
-                        if constexpr (KIND == REC_WKV) o = fmaf(sb[tb + t], sv[(tb + t) * VS + vc], o);
-                        a.out[(size_t)(row0 + t0 + tb + t) * a.ld_out + hv + v] = o;
+                        if constexpr (WKV) o = fmaf(sb[tt], sv[tt * VS + vc], o);
+                        a.out[(size_t)(row0 + t0 + tt) * a.ld_out + hv + v] = o;
                     }
+                }
             }
         }
+        parity ^= 1;
     }
     if (have_v) {
+        if (KPT % 4 == 0 && a.dim % 4 == 0) {
 #pragma unroll
-        for (int i = 0; i < KPT; ++i) {
-            const int k = ks * KPT + i;
-            if (k < a.dim) st[k] = S[i];
+            for (int i = 0; i < KPT; i += 4)
+                if (ks * KPT + i < a.dim) *reinterpret_cast<float4*>(st + ks * KPT + i) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
+        } else {
+#pragma unroll
+            for (int i = 0; i < KPT; ++i)
+                if (ks * KPT + i < a.dim) st[ks * KPT + i] = S[i];
         }
     }
 }
@@ -289,7 +355,19 @@ struct GroupNormArgs {
     float eps;
 };
 
-template <typename XT>
+// E consecutive values of a split input
+template <int E>
+DEVINL void split_load(const SplitIn& in, int row, int col, float (&v)[E]) {
+    if constexpr (E == 4) {
+        const float4 t = sum_splits4(in.p + (size_t)row * in.ld + col, in.stride, in.splits);
+        v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+    } else {
+        v[0] = in.at(row, col);
+    }
+}
+
+// E: values per access; 4 when every size and column offset is a multiple of 4
+template <typename XT, int E>
 __global__ void __launch_bounds__(256) group_norm_rows_kernel(const GroupNormArgs a, XT* x, int ld_x) {
     __shared__ float red[32];
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -298,10 +376,14 @@ __global__ void __launch_bounds__(256) group_norm_rows_kernel(const GroupNormArg
     pdl_launch();
     const int r = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     float ss[1] = {0.0f};
-    for (int j = tid; j < a.n; j += blockDim.x) {
-        const float t = a.o.at(r, (j / a.hs) * a.hs_ld + j % a.hs);
-        v[j] = t;
-        ss[0] += t * t;
+    for (int j = tid * E; j < a.n; j += blockDim.x * E) {
+        float t[E];
+        split_load<E>(a.o, r, a.hs == a.hs_ld ? j : (j / a.hs) * a.hs_ld + j % a.hs, t);
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+            v[j + e] = t[e];
+            ss[0] += t[e] * t[e];
+        }
     }
     float whole = 1.0f;
     if (a.group == a.n) {
@@ -317,15 +399,30 @@ __global__ void __launch_bounds__(256) group_norm_rows_kernel(const GroupNormArg
         }
     }
     __syncthreads();
-    for (int j = tid; j < ld_x; j += blockDim.x) {
-        float t = 0.0f;
+    for (int j = tid * E; j < ld_x; j += blockDim.x * E) {
+        float t[E];
+#pragma unroll
+        for (int e = 0; e < E; ++e) t[e] = 0.0f;
         if (j < a.n) {
-            t = v[j] * whole;
-            if (a.w) t *= a.w[j];
-            if (a.act == ACT_SIGMOID) t *= sigmoid(a.gate.at(r, a.c_gate + j));
-            else if (a.act == ACT_SILU) t *= silu(a.gate.at(r, a.c_gate + j));
+            if (a.act != ACT_NONE) {
+                split_load<E>(a.gate, r, a.c_gate + j, t);
+#pragma unroll
+                for (int e = 0; e < E; ++e) t[e] = a.act == ACT_SIGMOID ? sigmoid(t[e]) : silu(t[e]);
+            } else {
+#pragma unroll
+                for (int e = 0; e < E; ++e) t[e] = 1.0f;
+            }
+#pragma unroll
+            for (int e = 0; e < E; ++e) {
+                t[e] *= v[j + e] * whole;
+                if (a.w) t[e] *= a.w[j + e];
+            }
         }
-        store_act(x + (size_t)r * ld_x + j, t);
+        if constexpr (E == 4) {
+            store_x4(x + (size_t)r * ld_x + j, make_float4(t[0], t[1], t[2], t[3]));
+        } else {
+            store_act(x + (size_t)r * ld_x + j, t[0]);
+        }
     }
 }
 
@@ -406,17 +503,22 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a, XT
 }
 
 // Queries in latent space, few rows: q_abs[r, h, :] = q_unrotated . W_uk[h], followed by the rotated part; f32
-// [R, heads, rank + rot]. grid (heads + 1, R, slices of 256 latent columns); the CTAs of x == heads append the token to
-// the cache when `append` is set. dynamic shared memory: dim + rot floats
+// [R, heads, rank + rot]. grid (heads + 1, R, slices of kLqCols latent columns); the CTAs of x == heads append the token to
+// the cache when `append` is set. Two groups of threads share a column's sum. dynamic shared memory: dim + rot + 256 floats
+constexpr int kLqCols = 128;
 template <typename WT, typename KT>
 __global__ void __launch_bounds__(256)
 latent_query_kernel(const LatentArgs a, SplitIn q, const WT* w_uk, float* q_abs, int append) {
     __shared__ float red[32];
     extern __shared__ __align__(16) unsigned char smem_raw[];
     float* sq = reinterpret_cast<float*>(smem_raw);
+    const int hd = blockIdx.x, r = blockIdx.y, tid = threadIdx.x;
+    const int n = blockIdx.z * kLqCols + tid % kLqCols, part = tid / kLqCols;
+    if (hd < a.heads)                    // this CTA's block of W_uk depends on nothing the preceding kernel writes
+        for (int d = tid; d < a.dim; d += 256)
+            prefetch_l2(w_uk + ((size_t)hd * a.dim + d) * a.rank + min(blockIdx.z * kLqCols, a.rank - 1));
     pdl_wait();
     pdl_launch();
-    const int hd = blockIdx.x, r = blockIdx.y, tid = threadIdx.x;
     if (a.rows.tok[r] == kInactiveToken) return;
     if (hd == a.heads) {
         if (append && blockIdx.z == 0) latent_append<KT>(a, r, red);
@@ -426,20 +528,17 @@ latent_query_kernel(const LatentArgs a, SplitIn q, const WT* w_uk, float* q_abs,
     for (int j = tid; j < dq; j += 256) sq[j] = q.at(r, hd * dq + j);
     __syncthreads();
     float* dst = q_abs + ((size_t)r * a.heads + hd) * (a.rank + a.rot);
-    const int n = blockIdx.z * 256 + tid;
+    float* sum = sq + dq;                // [256]
+    float t = 0.0f;
     if (n < a.rank) {
-        float t0 = 0.0f, t1 = 0.0f, t2 = 0.0f, t3 = 0.0f;
         const size_t base = (size_t)hd * a.dim * a.rank + n;
-        int d = 0;
-        for (; d + 4 <= a.dim; d += 4) {
-            t0 = fmaf(sq[d], WTraits<WT>::elem(w_uk, base + (size_t)d * a.rank), t0);
-            t1 = fmaf(sq[d + 1], WTraits<WT>::elem(w_uk, base + (size_t)(d + 1) * a.rank), t1);
-            t2 = fmaf(sq[d + 2], WTraits<WT>::elem(w_uk, base + (size_t)(d + 2) * a.rank), t2);
-            t3 = fmaf(sq[d + 3], WTraits<WT>::elem(w_uk, base + (size_t)(d + 3) * a.rank), t3);
-        }
-        for (; d < a.dim; ++d) t0 = fmaf(sq[d], WTraits<WT>::elem(w_uk, base + (size_t)d * a.rank), t0);
-        dst[n] = (t0 + t1) + (t2 + t3);
+        const int half = (a.dim + 1) / 2, d1 = min(a.dim, (part + 1) * half);
+#pragma unroll 16
+        for (int d = part * half; d < d1; ++d) t = fmaf(sq[d], WTraits<WT>::elem(w_uk, base + (size_t)d * a.rank), t);
     }
+    sum[tid] = t;
+    __syncthreads();
+    if (part == 0 && n < a.rank) dst[n] = sum[tid] + sum[tid + kLqCols];
     if (blockIdx.z == 0) {
         const int pos = a.rows.pos[r];
         for (int i = tid; i < (a.rot + 1) / 2; i += 256) {
@@ -567,9 +666,17 @@ DEVINL void latent_part_factors(const LatentPart& part, size_t rh, float* sc) {
     __syncthreads();
 }
 DEVINL float latent_part_value(const LatentPart& part, size_t rh, int rank, int j, const float* sc) {
+    const float* o = part.o + rh * rank + j;
+    const size_t stride = part.rows * rank;
     float t = 0.0f;
-    for (int s = 0; s < part.splits; ++s)
-        if (sc[s] > 0.0f) t = fmaf(__ldcg(part.o + ((size_t)s * part.rows + rh) * rank + j), sc[s], t);
+    for (int s0 = 0; s0 < part.splits; s0 += 8) {
+        float v[8];
+#pragma unroll
+        for (int q = 0; q < 8; ++q) v[q] = s0 + q < part.splits && sc[s0 + q] > 0.0f ? __ldcg(o + (s0 + q) * stride) : 0.0f;
+#pragma unroll
+        for (int q = 0; q < 8; ++q)
+            if (s0 + q < part.splits) t = fmaf(v[q], sc[s0 + q], t);
+    }
     return t;
 }
 

@@ -1549,6 +1549,7 @@ struct RowSet {
     const int32_t* run_row0 = nullptr;
     const int32_t* run_n = nullptr;
     std::vector<int> run_len;            // host copy of run_n
+    int max_visible = 1;                 // bound on the visible positions of any row (launch geometry only)
 };
 
 // The residual update a pass over the layers leaves to the kernel that follows: h + rmsnorm(sum of raw, w_post),
@@ -2054,6 +2055,7 @@ static int32_t run_step(oxg4_cache* c, int kind, int top_k, float penalty, int* 
     rs.run_row0 = c->dec_grp_row0;
     rs.run_n = c->dec_grp_n;
     rs.run_len.assign(B, 1);
+    rs.max_visible = *std::max_element(c->max_seq.begin(), c->max_seq.end());
     const Pending pd = run_layers(c, ln, rs, c->use_tc, peer, kind != STEP_PREFILL, tr);
     if (kind != STEP_PREFILL) {
         if (c->use_tc) closing_norm_tc(c, ln, B, pd);
@@ -2690,6 +2692,7 @@ static int32_t ingest(oxg4_model* m, oxg4_cache* c, const uint32_t* tokens, cons
             rs.run_len.push_back(take);
             R += take;
             p += take;
+            rs.max_visible = std::max(rs.max_visible, c->pos_host[b] + p);
             if (p == lens[b]) { ++b; p = 0; }
         }
         if (R == 0) break;
