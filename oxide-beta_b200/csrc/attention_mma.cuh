@@ -133,10 +133,10 @@ DEVINL void mma_bf16_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, u
 }
 // (hi, lo) BF16 split of two f32 values, packed for an MMA operand (first value in the low half)
 DEVINL void split_pack(float x, float y, uint32_t& hi, uint32_t& lo) {
-    const uint32_t xh = f32_to_bf16_bits(x), yh = f32_to_bf16_bits(y);
-    const float xr = x - __uint_as_float(xh << 16), yr = y - __uint_as_float(yh << 16);
-    hi = xh | (yh << 16);
-    lo = f32_to_bf16_bits(xr) | (f32_to_bf16_bits(yr) << 16);
+    // round to nearest even, two values per instruction (the first source fills the high half)
+    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(hi) : "f"(y), "f"(x));
+    const float xr = x - bf16lo(hi), yr = y - bf16hi(hi);
+    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(lo) : "f"(yr), "f"(xr));
 }
 DEVINL void mbar_arrive(uint64_t* bar) {
     asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");

@@ -51,7 +51,7 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentM
     constexpr int ROWS = MT * 16;
     constexpr int SN = NB / 8;                       // score columns in MMA tiles
     constexpr int SPW = MT * SN / kLmWarps;          // score tiles per warp
-    static_assert(MT * SN % kLmWarps == 0 && NT % 2 == 0, "tile shape");
+    static_assert(MT * SN % kLmWarps == 0 && NT % 2 == 0 && NB % (2 * kLmThreads / ROWS) == 0, "tile shape");
     constexpr int TPR = kLmThreads / ROWS;           // threads per row in the softmax
     constexpr int PPT = NB / TPR;                    // positions per thread
     constexpr int PLD = NB + 8, SLD = NB + 4;
@@ -118,8 +118,13 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentM
         const uint32_t dst = smem_u32(skv + ((size_t)stage * NB + warp * RPW) * ldp);
 #pragma unroll
         for (int i = 0; i < RPW; ++i) {
-            const uint16_t* src = pool + __shfl_sync(0xffffffffu, off, i);
-            for (int c = lane; c < chunks; c += 32) cp_async16(dst + i * ldp * 2 + c * 16, src + c * 8, (valid >> i) & 1);
+            const uint16_t* src = pool + __shfl_sync(0xffffffffu, off, i) + lane * 8;
+            const bool ok = (valid >> i) & 1;
+            const uint32_t d = dst + i * ldp * 2 + lane * 16;
+#pragma unroll
+            for (int c = 0; c < 3; ++c)                              // cache rows of up to 768 elements
+                if (lane + 32 * c < chunks) cp_async16(d + c * 512, src + c * 256, ok);
+            for (int c = 3; lane + 32 * c < chunks; ++c) cp_async16(d + c * 512, src + c * 256, ok);
         }
     };
     load_tile(tile0, 0);
@@ -128,11 +133,18 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentM
         const size_t f = flat0 + i;
         const size_t row = f / a.heads;
         const int hd = (int)(f - row * a.heads);
-        for (int j = lane; j < ld; j += 32) {
-            float v = 0.0f;
-            if (i < n_here && j < DK)
-                v = j < a.rank ? a.q_abs[row * a.abs_row + (size_t)hd * a.abs_head + j] : a.q_rot[row * a.rot_row + (size_t)hd * a.rot_head + j - a.rank];
-            sq[(size_t)i * ldp + j] = (uint16_t)f32_to_bf16_bits(v);
+        const float* qa = a.q_abs + row * a.abs_row + (size_t)hd * a.abs_head;
+        const float* qr = a.q_rot + row * a.rot_row + (size_t)hd * a.rot_head - a.rank;
+        for (int j0 = 0; j0 < ld; j0 += 256) {
+            float v[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const int j = j0 + lane + 32 * e;
+                v[e] = i < n_here && j < DK ? (j < a.rank ? qa[j] : qr[j]) : 0.0f;
+            }
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+                if (j0 + lane + 32 * e < ld) sq[(size_t)i * ldp + j0 + lane + 32 * e] = (uint16_t)f32_to_bf16_bits(v[e]);
         }
     }
     float acc[MT][NT][4];
@@ -141,6 +153,7 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentM
 #pragma unroll
         for (int j = 0; j < NT; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.0f;
     const int srow = tid / TPR, sub = tid % TPR;
+    const float scale2 = a.scale * 1.4426950408889634f;              // scores in units of log 2
     float m_run = -INFINITY, l_run = 0.0f;                           // of row srow (the same in its TPR threads)
     // score tiles of this warp: one row tile, SPW neighbouring column tiles
     const int s_mi = warp % MT, s_n0 = (warp / MT) * SPW;
@@ -160,28 +173,50 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentM
             float s[SPW][4];
 #pragma unroll
             for (int j = 0; j < SPW; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
-            if constexpr (SPW == 1 && KQ > 0) {
+            if constexpr (KQ > 0) {
                 if (tile == tile0) {
 #pragma unroll
                     for (int k = 0; k < KQ; ++k)
                         if (k * 16 < ld) ldmatrix_x4(qf[k], q_base + k * 32);
                 }
-                const uint32_t kb = kv + ((s_n0 * 8 + (lane & 7)) * ldp + (lane >> 3) * 8) * 2;
-                float s2[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+                float s2[SPW][4];
 #pragma unroll
-                for (int k = 0; k < KQ; k += 2) {
-                    uint32_t b[4];
-                    if (k * 16 + 32 <= ld) {
-                        ldmatrix_x4(b, kb + k * 32);
-                        mma_bf16_16816(s[0], qf[k], b[0], b[1]);
-                        mma_bf16_16816(s2, qf[k + 1], b[2], b[3]);
-                    } else if (k * 16 < ld) {                        // ld is a multiple of 16
-                        ldmatrix_x4(b, kv + ((s_n0 * 8 + (lane & 7)) * ldp + ((lane >> 3) & 1) * 8 + k * 16) * 2);
-                        mma_bf16_16816(s[0], qf[k], b[0], b[1]);
+                for (int j = 0; j < SPW; ++j) s2[j][0] = s2[j][1] = s2[j][2] = s2[j][3] = 0.0f;
+                if constexpr (SPW == 1) {
+                    // one column tile: a load brings its 8 positions for two k-steps
+                    float s3[4] = {0.0f, 0.0f, 0.0f, 0.0f}, s4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+                    const uint32_t kb = kv + ((s_n0 * 8 + (lane & 7)) * ldp + (lane >> 3) * 8) * 2;
+#pragma unroll
+                    for (int k = 0; k < KQ; k += 2) {
+                        uint32_t b[4];
+                        if (k * 16 + 32 <= ld) {
+                            ldmatrix_x4(b, kb + k * 32);
+                            mma_bf16_16816((k & 2) ? s3 : s[0], qf[k], b[0], b[1]);
+                            mma_bf16_16816((k & 2) ? s4 : s2[0], qf[k + 1], b[2], b[3]);
+                        } else if (k * 16 < ld) {                    // ld is a multiple of 16
+                            ldmatrix_x4(b, kv + ((s_n0 * 8 + (lane & 7)) * ldp + ((lane >> 3) & 1) * 8 + k * 16) * 2);
+                            mma_bf16_16816(s[0], qf[k], b[0], b[1]);
+                        }
                     }
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) s[0][q] += s3[q] + s4[q];
+                } else {
+                    // a pair of column tiles: a load brings 16 positions for one k-step
+                    static_assert(SPW <= 2, "score tiles per warp");
+                    const uint32_t kb = kv + ((s_n0 * 8 + (lane >> 4) * 8 + (lane & 7)) * ldp + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+                    for (int k = 0; k < KQ; ++k)
+                        if (k * 16 < ld) {
+                            uint32_t b[4];
+                            ldmatrix_x4(b, kb + k * 32);
+                            mma_bf16_16816((k & 1) ? s2[0] : s[0], qf[k], b[0], b[1]);
+                            mma_bf16_16816((k & 1) ? s2[1] : s[1], qf[k], b[2], b[3]);
+                        }
                 }
 #pragma unroll
-                for (int q = 0; q < 4; ++q) s[0][q] += s2[q];
+                for (int j = 0; j < SPW; ++j)
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) s[j][q] += s2[j][q];
             } else if constexpr (SPW == 1) {
                 // one column tile: a load brings its 8 positions for two k-steps
                 const uint32_t kb = kv + ((s_n0 * 8 + (lane & 7)) * ldp + (lane >> 3) * 8) * 2;
@@ -237,24 +272,28 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentM
             const int lim = s_pos[srow] - tile * NB;                 // last visible column of this row
             float v[PPT], mx = -INFINITY;
 #pragma unroll
-            for (int j = 0; j < PPT; ++j) {
-                const int c = sub + j * TPR;
-                v[j] = c <= lim ? ss[srow * SLD + c] * a.scale : -INFINITY;
-                mx = fmaxf(mx, v[j]);
+            for (int j = 0; j < PPT; j += 2) {                       // pairs of neighbouring positions
+                const int c = 2 * sub + j * TPR;
+                const float2 x = *reinterpret_cast<const float2*>(ss + srow * SLD + c);
+                v[j] = c <= lim ? x.x * scale2 : -INFINITY;
+                v[j + 1] = c + 1 <= lim ? x.y * scale2 : -INFINITY;
+                mx = fmaxf(mx, fmaxf(v[j], v[j + 1]));
             }
 #pragma unroll
             for (int o = TPR / 2; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
             const float m_new = fmaxf(m_run, mx);
-            const float alpha = m_new == m_run ? 1.0f : expf(m_run - m_new);
+            const float base = m_new == -INFINITY ? 0.0f : m_new;    // a row without a visible position so far
+            const float alpha = m_new == m_run ? 1.0f : exp2f(m_run - base);
             float sum = 0.0f;
 #pragma unroll
-            for (int j = 0; j < PPT; ++j) {
-                const float e = v[j] > -INFINITY ? expf(v[j] - m_new) : 0.0f;
-                sum += e;
-                const uint32_t hi = f32_to_bf16_bits(e);
-                const int c = sub + j * TPR;
-                sp[srow * PLD + c] = (uint16_t)hi;
-                sp[(ROWS + srow) * PLD + c] = (uint16_t)f32_to_bf16_bits(e - __uint_as_float(hi << 16));
+            for (int j = 0; j < PPT; j += 2) {
+                const float e0 = exp2f(v[j] - base), e1 = exp2f(v[j + 1] - base);
+                sum += e0 + e1;
+                uint32_t hi, lo;
+                split_pack(e0, e1, hi, lo);
+                const int c = 2 * sub + j * TPR;
+                *reinterpret_cast<uint32_t*>(sp + srow * PLD + c) = hi;
+                *reinterpret_cast<uint32_t*>(sp + (ROWS + srow) * PLD + c) = lo;
             }
 #pragma unroll
             for (int o = TPR / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
@@ -308,7 +347,7 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_mma_kernel(const LatentM
             }
         }
     }
-    if (sub == 0 && srow < n_here) { part_ml[2 * srow] = m_run; part_ml[2 * srow + 1] = l_run; }
+    if (sub == 0 && srow < n_here) { part_ml[2 * srow] = m_run * 0.6931471805599453f; part_ml[2 * srow + 1] = l_run; }
     float* po = a.part.o + ((size_t)blockIdx.y * a.part.rows + flat0) * a.rank;
 #pragma unroll
     for (int i = 0; i < MT; ++i)

@@ -449,7 +449,8 @@ static LatentMmaFn pick_latent_mma(int rank, int ld, int rows, int* tile_rows, i
         *tile_rows = MT * 16;                                                                                   \
         *smem = latent_mma_smem<MT, NB>(ld);                                                                    \
     }
-    if (rows <= 16) LM(1, 64) else if (rows <= 32) LM(2, 32) else LM(4, 32)
+    if (rows <= 16) LM(1, 64) else if (rows <= 32) LM(2, 64) else LM(4, 32)
+    if (*smem > 226 * 1024 && rows <= 32 && rows > 16) LM(2, 32)
 #undef LM
     return *smem <= 226 * 1024 ? fn : nullptr;
 }
@@ -672,8 +673,9 @@ struct LayeredPass {
         const bool step = !rs.chunk;
         if (wkv) fn = m->es == 2 ? pick_recur<REC_WKV, uint16_t>(x.dim, step, &ks, &kpt) : pick_recur<REC_WKV, float>(x.dim, step, &ks, &kpt);
         else fn = pick_recur<REC_LIGHTNING, float>(x.dim, step, &ks, &kpt);
-        const int vs = kRecThreads / ks, dp = ks * kpt, tile = step ? 1 : rec_tile(dp);
-        const size_t smem = sizeof(float) * ((step ? 1 : 2) * ((size_t)tile * dp * (wkv ? 3 : 2) + tile * vs + pad_to(tile, 4)) + (wkv ? x.low_rank : 0));
+        const int vs = kRecThreads / ks * kRecCols, dp = ks * kpt, tile = step ? 1 : rec_tile(dp);
+        const size_t smem = sizeof(float) * ((step ? 1 : 2) * ((size_t)tile * dp * (wkv ? 3 : 2) + tile * vs + pad_to(tile, 4)) +
+                                             (wkv ? dp + x.low_rank : 0));
         if (ln.status == OXG4_OK && smem > 48 * 1024) ln.status = allow_big_smem(fn);
         ln.go("recur", fn, dim3(x.heads, (x.vdim + vs - 1) / vs, (unsigned)rs.run_len.size()), dim3(kRecThreads), smem, a);
         output(x, one(c->attn_out, x.owp), x.vdim, wkv ? x.dim : x.ow, x.out_norm, in, wkv ? ACT_SILU : ACT_SIGMOID);
@@ -752,7 +754,7 @@ struct LayeredPass {
             LatentAttnFn fn = pick_latent_attn<KT>(x.rank);
             ln.go("attn", fn, dim3(x.heads, R, part.splits), dim3(256), sizeof(float) * (x.rank + x.rot + 8 * x.rank + 16), a, (const float*)c->lat_q, part);
         }
-        ln.go("latout", latent_out_kernel<WT>, dim3(x.heads, R, (x.vdim + 31) / 32), dim3(256), sizeof(float) * (x.rank + part.splits), x.heads,
+        ln.go("latout", latent_out_kernel<WT>, dim3(x.heads, R, (x.vdim + 31) / 32), dim3(256), sizeof(float) * (pad_to(x.rank, 4) + part.splits), x.heads,
               x.rank, x.vdim, part, (const WT*)x.w_uv, x.rank, in, x.c_g, rs.tok, c->attn_out, x.owp);
         // the gate has been applied by the kernel that leaves latent space
         output(x, one(c->attn_out, x.owp), x.vdim, 0, nullptr, in, ACT_NONE);

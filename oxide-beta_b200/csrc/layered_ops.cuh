@@ -121,12 +121,13 @@ wkv_decay_kernel(int R, int N, int rank, SplitIn low, int col, const WT* w2, con
 //   REC_LIGHTNING  q, k, v = silu(.);  S = decay_h S + k v^T;  o = S^T q
 //   REC_WKV        o = (S + diag(u) k v^T)^T r;  S = diag(w) S + k v^T, w per token and key channel
 // The bonus term is v * sum_k r_k u_k k_k, one scalar per token and head.
-// Grid (heads, slices of vdim, runs). A thread owns KPT consecutive key channels of one value column; the KS threads
-// that share a column are neighbouring lanes. Tokens are staged in shared memory in tiles, activations applied on
+// Grid (heads, slices of vdim, runs). A thread owns KPT key channels of two value columns; the KS threads that share
+// a column are neighbouring lanes. Tokens are staged in shared memory in tiles, activations applied on
 // the way; the dot products of up to 8 tokens are reduced across the KS lanes together.
 // State in memory: [sequence][head][vdim][dim]. At position 0 the state starts at zero whatever the memory holds.
 enum { REC_LIGHTNING = 0, REC_WKV = 1 };
-constexpr int kRecThreads = 256;
+constexpr int kRecThreads = 128;
+constexpr int kRecCols = 2;              // value columns per thread
 constexpr int rec_tile(int dp) { return dp <= 128 ? 16 : dp <= 256 ? 8 : 4; }   // tokens staged at a time
 
 struct RecurArgs {
@@ -173,69 +174,99 @@ DEVINL void column_reduce(float (&acc)[N], int ks, int& first) {
     }
 }
 
-// TILE: tokens staged at a time; 1 for decode steps (runs of one token). Tiles of longer runs are double-buffered: the next
-// tile's values are fetched into registers while the current one is walked.
+// TILE: tokens staged at a time; 1 for decode steps (row r is sequence r's one token). Tiles of longer runs are
+// double-buffered: the next tile's values are fetched into registers while the current one is walked. A thread's key
+// channels come in groups of four, KS * 4 apart, so that the lanes of a column read neighbouring 16-byte pieces.
 template <int KIND, typename WT, int KS, int KPT, int TILE>
-__global__ void __launch_bounds__(kRecThreads, 2) recur_kernel(const RecurArgs a) {
+__global__ void __launch_bounds__(kRecThreads) recur_kernel(const RecurArgs a) {
     constexpr bool WKV = KIND == REC_WKV;
     constexpr int DP = KS * KPT;         // key channels, padded
-    constexpr int VS = kRecThreads / KS; // value columns of this CTA
+    constexpr int VG = kRecThreads / KS; // threads along the value columns
+    constexpr int VS = VG * kRecCols;    // value columns of this CTA
     constexpr int NK = (TILE * DP + kRecThreads - 1) / kRecThreads, NV = (TILE * VS + kRecThreads - 1) / kRecThreads;
     constexpr int TB = TILE < 8 ? TILE : 8;
     constexpr int TPAD = (TILE + 3) / 4 * 4;
     constexpr int BUF = TILE * DP * (WKV ? 3 : 2) + TILE * VS + TPAD;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     float* bufs = reinterpret_cast<float*>(smem_raw);        // [2 (1 for TILE 1)][q | k | w (WKV) | v | bonus (WKV)]
+    float* su = bufs + (TILE == 1 ? 1 : 2) * BUF;            // WKV: [DP] u of this head, then [rank] for one-token runs
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int hd = blockIdx.x, v0 = blockIdx.y * VS, run = blockIdx.z;
-    const int ks = tid % KS, vc = tid / KS, v = v0 + vc;
+    const int ks = tid % KS, vg = tid / KS;
     const int hk = hd * a.dim, hv = hd * a.vdim;
+    auto channel = [&](int i) { return (i / 4) * (KS * 4) + ks * 4 + i % 4; };
+    if constexpr (WKV)
+        for (int k = tid; k < DP; k += kRecThreads) su[k] = k < a.dim ? a.u[hk + k] : 0.0f;
     pdl_wait();
     pdl_launch();
-    const int row0 = a.rows.row0[run], n = TILE == 1 ? 1 : a.rows.n[run];
+    const int row0 = TILE == 1 ? run : a.rows.row0[run], n = TILE == 1 ? 1 : a.rows.n[run];
     const int seq = a.rows.seq_of(row0);
-    const bool have_v = v < a.vdim;
-    float* st = a.state + (((size_t)seq * a.heads + hd) * a.vdim + v) * a.dim;
-    float S[KPT];
-    if (KPT % 4 == 0 && a.dim % 4 == 0) {
+    const uint32_t tok = a.rows.tok[row0];
+    const int pos = a.rows.pos[row0];
+    float* st = a.state + (((size_t)seq * a.heads + hd) * a.vdim + v0 + vg) * a.dim;     // column j: VG * dim further
+    float S[kRecCols][KPT];
 #pragma unroll
-        for (int i = 0; i < KPT; i += 4) {
-            const int k = ks * KPT + i;
-            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            if (have_v && k < a.dim) x = *reinterpret_cast<const float4*>(st + k);
-            S[i] = x.x; S[i + 1] = x.y; S[i + 2] = x.z; S[i + 3] = x.w;
+    for (int j = 0; j < kRecCols; ++j) {
+        const bool have = v0 + vg + j * VG < a.vdim;
+        const float* sj = st + (size_t)j * VG * a.dim;
+        if (a.dim % 4 == 0) {
+#pragma unroll
+            for (int i = 0; i < KPT; i += 4) {
+                float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                if (have && channel(i) < a.dim) x = *reinterpret_cast<const float4*>(sj + channel(i));
+                S[j][i] = x.x; S[j][i + 1] = x.y; S[j][i + 2] = x.z; S[j][i + 3] = x.w;
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < KPT; ++i) S[j][i] = (have && channel(i) < a.dim) ? sj[channel(i)] : 0.0f;
         }
-    } else {
-#pragma unroll
-        for (int i = 0; i < KPT; ++i) S[i] = (have_v && ks * KPT + i < a.dim) ? st[ks * KPT + i] : 0.0f;
     }
-    if (a.rows.tok[row0] == kInactiveToken) return;
-    if (a.rows.pos[row0] == 0) {
+    float fq[NK], fk[NK], fw[WKV ? NK : 1], fv[NV];
+    auto fetch = [&](int t0) {           // values of the tile at t0, zero past the run and past the key channels
+        const float* base = a.in.p + (size_t)(row0 + t0) * a.in.ld;
 #pragma unroll
-        for (int i = 0; i < KPT; ++i) S[i] = 0.0f;
+        for (int j = 0; j < NK; ++j) {
+            const int i = tid + j * kRecThreads, t = i / DP, k = i % DP;
+            const bool ok = i < TILE * DP && t0 + t < n && k < a.dim;
+            const float* p = base + (size_t)t * a.in.ld + hk + k;
+            fq[j] = ok ? p[a.c_q] : 0.0f;
+            fk[j] = ok ? p[a.c_k] : 0.0f;
+            if constexpr (WKV) fw[j] = ok && a.w != nullptr ? a.w[(size_t)(row0 + t0 + t) * a.heads * a.dim + hk + k] : 0.0f;
+        }
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = tid + j * kRecThreads, t = i / VS, c = v0 + i % VS;
+            fv[j] = (i < TILE * VS && t0 + t < n && c < a.vdim) ? base[(size_t)t * a.in.ld + a.c_v + hv + c] : 0.0f;
+        }
+        for (int s = 1; s < a.in.splits; ++s) {
+            const float* part = base + s * a.in.stride;
+#pragma unroll
+            for (int j = 0; j < NK; ++j) {
+                const int i = tid + j * kRecThreads, t = i / DP, k = i % DP;
+                if (i < TILE * DP && t0 + t < n && k < a.dim) {
+                    fq[j] += part[(size_t)t * a.in.ld + a.c_q + hk + k];
+                    fk[j] += part[(size_t)t * a.in.ld + a.c_k + hk + k];
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                const int i = tid + j * kRecThreads, t = i / VS, c = v0 + i % VS;
+                if (i < TILE * VS && t0 + t < n && c < a.vdim) fv[j] += part[(size_t)t * a.in.ld + a.c_v + hv + c];
+            }
+        }
+    };
+    fetch(0);
+    if (tok == kInactiveToken) return;
+    if (pos == 0) {
+#pragma unroll
+        for (int j = 0; j < kRecCols; ++j)
+#pragma unroll
+            for (int i = 0; i < KPT; ++i) S[j][i] = 0.0f;
     }
     if (a.shift_src != nullptr && hd == 0 && blockIdx.y == 0)
         for (int i = tid; i < a.shift_n; i += kRecThreads)
             a.shift_dst[(size_t)seq * a.shift_n + i] = a.shift_src[(size_t)(row0 + n - 1) * a.shift_n + i];
     const float dh = WKV ? 0.0f : a.decay[hd];
-
-    float fq[NK], fk[NK], fw[WKV ? NK : 1], fv[NV];
-    auto fetch = [&](int t0) {           // values of the tile at t0, zero past the run and past the key channels
-#pragma unroll
-        for (int j = 0; j < NK; ++j) {
-            const int i = tid + j * kRecThreads, t = t0 + i / DP, k = i % DP;
-            const bool ok = i < TILE * DP && t < n && k < a.dim;
-            fq[j] = ok ? a.in.at(row0 + t, a.c_q + hk + k) : 0.0f;
-            fk[j] = ok ? a.in.at(row0 + t, a.c_k + hk + k) : 0.0f;
-            if constexpr (WKV) fw[j] = ok && a.w != nullptr ? a.w[(size_t)(row0 + t) * a.heads * a.dim + hk + k] : 0.0f;
-        }
-#pragma unroll
-        for (int j = 0; j < NV; ++j) {
-            const int i = tid + j * kRecThreads, t = t0 + i / VS, c = v0 + i % VS;
-            fv[j] = (i < TILE * VS && t < n && c < a.vdim) ? a.in.at(row0 + t, a.c_v + hv + c) : 0.0f;
-        }
-    };
-    fetch(0);
     int parity = 0;
     for (int t0 = 0; t0 < n; t0 += TILE) {
         const int nt = min(TILE, n - t0);
@@ -256,10 +287,9 @@ __global__ void __launch_bounds__(kRecThreads, 2) recur_kernel(const RecurArgs a
             if (i < TILE * VS) sv[i] = WKV ? fv[j] : silu(fv[j]);
         }
         if (t0 + TILE < n) fetch(t0 + TILE);
-        __syncthreads();
-        if constexpr (WKV) {
-            if (TILE == 1 && a.w == nullptr) {               // decay of this head's channels, four lanes per channel
-                float* th = sb + TPAD;                       // [rank]
+        if constexpr (WKV && TILE == 1) {
+            if (a.w == nullptr) {                            // decay of this head's channels, four lanes per channel
+                float* th = su + DP;                         // [rank]
                 for (int j = tid; j < a.rank; j += kRecThreads) th[j] = tanhf(a.in.at(row0, a.c_low + j));
                 __syncthreads();
                 for (int k0 = 0; k0 < a.dim; k0 += kRecThreads / 4) {
@@ -273,71 +303,98 @@ __global__ void __launch_bounds__(kRecThreads, 2) recur_kernel(const RecurArgs a
                     if (k < a.dim && (tid & 3) == 0) sw[k] = expf(-expf(t + a.w0[hk + k]));
                 }
             }
+        }
+        __syncthreads();
+        if constexpr (WKV && TILE > 1) {                     // bonus of every token: sum over k of r u k
             for (int t = warp; t < nt; t += kRecThreads / 32) {
                 float b = 0.0f;
-                for (int k = lane; k < a.dim; k += 32) b += sq[t * DP + k] * a.u[hk + k] * sk[t * DP + k];
+                for (int k = lane; k < DP; k += 32) b += sq[t * DP + k] * su[k] * sk[t * DP + k];
                 b = warp_sum(b);
                 if (lane == 0) sb[t] = b;
             }
             __syncthreads();
         }
         for (int tb = 0; tb < nt; tb += TB) {
-            float acc[TB];
+            float acc[kRecCols][TB];
 #pragma unroll
             for (int t = 0; t < TB; ++t) {
-                acc[t] = 0.0f;
+#pragma unroll
+                for (int j = 0; j < kRecCols; ++j) acc[j][t] = 0.0f;
                 if (tb + t >= nt) continue;
-                const float* q = sq + (tb + t) * DP + ks * KPT;
-                const float* k = sk + (tb + t) * DP + ks * KPT;
-                const float* w = sw + (tb + t) * DP + ks * KPT;
-                const float x = sv[(tb + t) * VS + vc];
-                float s = 0.0f;
+                const float* q = sq + (tb + t) * DP + ks * 4;
+                const float* k = sk + (tb + t) * DP + ks * 4;
+                const float* w = sw + (tb + t) * DP + ks * 4;
+                float x[kRecCols];
+#pragma unroll
+                for (int j = 0; j < kRecCols; ++j) x[j] = sv[(tb + t) * VS + vg + j * VG];
 #pragma unroll
                 for (int i = 0; i < KPT; i += 4) {
-                    const float4 q4 = *reinterpret_cast<const float4*>(q + i), k4 = *reinterpret_cast<const float4*>(k + i);
+                    const float4 q4 = *reinterpret_cast<const float4*>(q + i * KS), k4 = *reinterpret_cast<const float4*>(k + i * KS);
+                    const float qe[4] = {q4.x, q4.y, q4.z, q4.w}, ke[4] = {k4.x, k4.y, k4.z, k4.w};
                     if constexpr (!WKV) {
-                        S[i] = fmaf(dh, S[i], k4.x * x); s = fmaf(q4.x, S[i], s);
-                        S[i + 1] = fmaf(dh, S[i + 1], k4.y * x); s = fmaf(q4.y, S[i + 1], s);
-                        S[i + 2] = fmaf(dh, S[i + 2], k4.z * x); s = fmaf(q4.z, S[i + 2], s);
-                        S[i + 3] = fmaf(dh, S[i + 3], k4.w * x); s = fmaf(q4.w, S[i + 3], s);
+#pragma unroll
+                        for (int j = 0; j < kRecCols; ++j)
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                S[j][i + e] = fmaf(dh, S[j][i + e], ke[e] * x[j]);
+                                acc[j][t] = fmaf(qe[e], S[j][i + e], acc[j][t]);
+                            }
                     } else {
-                        const float4 w4 = *reinterpret_cast<const float4*>(w + i);
-                        s = fmaf(q4.x, S[i], s); S[i] = fmaf(w4.x, S[i], k4.x * x);
-                        s = fmaf(q4.y, S[i + 1], s); S[i + 1] = fmaf(w4.y, S[i + 1], k4.y * x);
-                        s = fmaf(q4.z, S[i + 2], s); S[i + 2] = fmaf(w4.z, S[i + 2], k4.z * x);
-                        s = fmaf(q4.w, S[i + 3], s); S[i + 3] = fmaf(w4.w, S[i + 3], k4.w * x);
+                        const float4 w4 = *reinterpret_cast<const float4*>(w + i * KS);
+                        const float we[4] = {w4.x, w4.y, w4.z, w4.w};
+                        if constexpr (TILE == 1) {
+                            const float4 u4 = *reinterpret_cast<const float4*>(su + ks * 4 + i * KS);
+                            const float ue[4] = {u4.x, u4.y, u4.z, u4.w};
+#pragma unroll
+                            for (int j = 0; j < kRecCols; ++j)
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) acc[j][t] = fmaf(qe[e] * ue[e] * ke[e], x[j], acc[j][t]);
+                        }
+#pragma unroll
+                        for (int j = 0; j < kRecCols; ++j)
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                acc[j][t] = fmaf(qe[e], S[j][i + e], acc[j][t]);
+                                S[j][i + e] = fmaf(we[e], S[j][i + e], ke[e] * x[j]);
+                            }
                     }
                 }
-                acc[t] = s;
             }
-            int first;
-            column_reduce<TB, KS>(acc, ks, first);
             constexpr int LEFT = TB / KS > 0 ? TB / KS : 1;
             // with more lanes than tokens the lanes that differ in the low bits hold the same total: one of them stores
             const bool owner = KS <= TB || ks % (KS / TB > 0 ? KS / TB : 1) == 0;
-            if (have_v && owner) {
 #pragma unroll
-                for (int t = 0; t < LEFT; ++t) {
-                    const int tt = tb + first + t;
-                    if (tt < nt) {
-                        float o = acc[t];
-                        if constexpr (WKV) o = fmaf(sb[tt], sv[tt * VS + vc], o);
-                        a.out[(size_t)(row0 + t0 + tt) * a.ld_out + hv + v] = o;
+            for (int j = 0; j < kRecCols; ++j) {
+                int first;
+                column_reduce<TB, KS>(acc[j], ks, first);
+                const int c = vg + j * VG;
+                if (v0 + c < a.vdim && owner) {
+#pragma unroll
+                    for (int t = 0; t < LEFT; ++t) {
+                        const int tt = tb + first + t;
+                        if (tt < nt) {
+                            float o = acc[j][t];
+                            if constexpr (WKV && TILE > 1) o = fmaf(sb[tt], sv[tt * VS + c], o);
+                            a.out[(size_t)(row0 + t0 + tt) * a.ld_out + hv + v0 + c] = o;
+                        }
                     }
                 }
             }
         }
         parity ^= 1;
     }
-    if (have_v) {
-        if (KPT % 4 == 0 && a.dim % 4 == 0) {
+#pragma unroll
+    for (int j = 0; j < kRecCols; ++j) {
+        if (v0 + vg + j * VG >= a.vdim) continue;
+        float* sj = st + (size_t)j * VG * a.dim;
+        if (a.dim % 4 == 0) {
 #pragma unroll
             for (int i = 0; i < KPT; i += 4)
-                if (ks * KPT + i < a.dim) *reinterpret_cast<float4*>(st + ks * KPT + i) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
+                if (channel(i) < a.dim) *reinterpret_cast<float4*>(sj + channel(i)) = make_float4(S[j][i], S[j][i + 1], S[j][i + 2], S[j][i + 3]);
         } else {
 #pragma unroll
             for (int i = 0; i < KPT; ++i)
-                if (ks * KPT + i < a.dim) st[ks * KPT + i] = S[i];
+                if (channel(i) < a.dim) sj[channel(i)] = S[j][i];
         }
     }
 }
@@ -695,32 +752,58 @@ latent_merge_kernel(int R, int heads, int rank, LatentPart part, uint16_t* x, in
 }
 
 // few rows: merge, W_uv and the output gate: out[r, h * vdim + v] = (W_uv[h, v, :] . o) * sigmoid(gate). W_uv rows are
-// `ldw` elements apart. grid (heads, R, slices of 32 value columns), 256 threads, shared memory splits + rank floats
+// `ldw` elements apart. A warp owns four value columns; rows of whole 16-byte pieces are fetched before the dependency wait.
+// grid (heads, R, slices of 32 value columns), 256 threads, shared memory splits + rank floats (16-byte aligned)
 template <typename WT>
 __global__ void __launch_bounds__(256)
 latent_out_kernel(int heads, int rank, int vdim, LatentPart part, const WT* w_uv, int ldw, SplitIn gate, int c_gate,
                   const uint32_t* tok, float* out, int ld_out) {
+    constexpr int EPL = WTraits<WT>::EPL, PIECES = 512 / (32 * EPL);         // rank <= 512
     extern __shared__ __align__(16) unsigned char smem_raw[];
     float* so = reinterpret_cast<float*>(smem_raw);
-    float* sc = so + rank;
+    float* sc = so + (rank + 3) / 4 * 4;
+    const int hd = blockIdx.x, r = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int vb = blockIdx.z * 32 + warp * 4;
+    const bool vec = rank % EPL == 0 && ldw % EPL == 0;
+    uint4 w[4][PIECES];
+    if (vec) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int p = 0; p < PIECES; ++p) {
+                const int j = (p * 32 + lane) * EPL;
+                w[i][p] = make_uint4(0u, 0u, 0u, 0u);
+                if (vb + i < vdim && j < rank) w[i][p] = ldg_stream16(w_uv + ((size_t)hd * vdim + vb + i) * ldw + j);
+            }
+    }
     pdl_wait();
     pdl_launch();
-    const int hd = blockIdx.x, r = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     if (tok[r] == kInactiveToken) return;
     const size_t rh = (size_t)r * heads + hd;
     latent_part_factors(part, rh, sc);
     for (int j = threadIdx.x; j < rank; j += 256) so[j] = latent_part_value(part, rh, rank, j, sc);
     __syncthreads();
-    for (int i = warp; i < 32; i += 8) {
-        const int v = blockIdx.z * 32 + i;
-        if (v >= vdim) break;
-        const size_t base = ((size_t)hd * vdim + v) * ldw;
-        float t = 0.0f;
-        for (int j = lane; j < rank; j += 32) t = fmaf(WTraits<WT>::elem(w_uv, base + j), so[j], t);
-        t = warp_sum(t);
-        if (lane == 0) {
-            const int c = hd * vdim + v;
-            out[(size_t)r * ld_out + c] = t * sigmoid(gate.at(r, c_gate + c));
+    float t[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+    if (vec) {
+#pragma unroll
+        for (int p = 0; p < PIECES; ++p) {
+            const int j = (p * 32 + lane) * EPL;
+            if (j < rank)
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int e = 0; e < EPL; ++e) t[i] = fmaf(WTraits<WT>::elem(&w[i][p], e), so[j + e], t[i]);
+        }
+    } else {
+        for (int i = 0; i < 4 && vb + i < vdim; ++i)
+            for (int j = lane; j < rank; j += 32) t[i] = fmaf(WTraits<WT>::elem(w_uv, ((size_t)hd * vdim + vb + i) * ldw + j), so[j], t[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        t[i] = warp_sum(t[i]);
+        if (lane == 0 && vb + i < vdim) {
+            const int c = hd * vdim + vb + i;
+            out[(size_t)r * ld_out + c] = t[i] * sigmoid(gate.at(r, c_gate + c));
         }
     }
 }
