@@ -328,8 +328,8 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
     size_t in_n = 1, o_n = 1, gu_n = 1, down_n = 1, q_n = 1, uk_n = 1, uv_n = 1, dec = 1, latq = 1, rh = 1, rh_rank = 1, xo = 1, xi = 1, xq = 1,
            xu = 1, xl = 1, rot = 1, act = 1;
     bool any_shift = false;
-    const int max_tiles = (*std::max_element(c->max_seq.begin(), c->max_seq.end()) + 63) / 64;
-    c->lat_splits = std::max(1, std::min({max_tiles, 64, (4 * m->num_sms + B - 1) / B}));
+    const int max_tiles = (*std::max_element(c->max_seq.begin(), c->max_seq.end()) + kLmTile - 1) / kLmTile;
+    c->lat_splits = std::max(2, std::min({max_tiles, 64, (4 * m->num_sms + B - 1) / B}));
     for (int l = 0; l < L; ++l) {
         const MixPlan& x = m->layers[l].mix;
         in_n = std::max(in_n, floats(x.in));
@@ -438,41 +438,48 @@ static LatentAttnFn pick_latent_attn(int rank) {
 
 typedef void (*LatentMmaFn)(const LatentMmaArgs);
 // the tensor-core kernel for `rows` (token, head) rows per run and cache rows of `ld` elements, null when it does not fit
-static LatentMmaFn pick_latent_mma(int rank, int ld, int rows, int* tile_rows, int* tile_pos, size_t* smem) {
+static LatentMmaFn pick_latent_mma(int rank, int ld, int rows, int* tile_rows, int* groups, size_t* smem) {
     LatentMmaFn fn;
-#define LM(MT, NB)                                                                                              \
+#define LM(MT, NST, GR)                                                                                         \
     {                                                                                                           \
-        if (rank <= 128) fn = MT < 4 && ld <= 192 ? latent_mma_kernel<MT, 2, NB, MT < 4 ? 12 : 0> : latent_mma_kernel<MT, 2, NB, 0>;       \
-        else if (rank <= 256) fn = MT < 4 && ld <= 320 ? latent_mma_kernel<MT, 4, NB, MT < 4 ? 20 : 0> : latent_mma_kernel<MT, 4, NB, 0>;  \
-        else fn = MT < 4 && ld <= 576 ? latent_mma_kernel<MT, 8, NB, MT < 4 ? 36 : 0> : latent_mma_kernel<MT, 8, NB, 0>;                   \
-        *tile_pos = NB;                                                                                         \
+        fn = rank <= 128 ? latent_mma_kernel<MT, 2, NST, GR> : rank <= 256 ? latent_mma_kernel<MT, 4, NST, GR> : latent_mma_kernel<MT, 8, NST, GR>; \
         *tile_rows = MT * 16;                                                                                   \
-        *smem = latent_mma_smem<MT, NB>(ld);                                                                    \
+        *groups = GR;                                                                                           \
+        *smem = latent_mma_smem<MT, NST, GR>(ld);                                                               \
     }
-    if (rows <= 16) LM(1, 64) else if (rows <= 32) LM(2, 64) else LM(4, 32)
-    if (*smem > 226 * 1024 && rows <= 32 && rows > 16) LM(2, 32)
+    const size_t limit = 226 * 1024;
+    if (rows <= 16) {
+        LM(1, 2, 2)
+        if (*smem > limit) LM(1, 2, 1)
+    } else if (rows <= 32) {
+        LM(2, 2, 2)
+        if (*smem > limit) LM(2, 2, 1)
+    } else {
+        LM(4, 3, 1)
+        if (*smem > limit) LM(4, 2, 1)
+    }
 #undef LM
-    return *smem <= 226 * 1024 ? fn : nullptr;
+    return *smem <= limit ? fn : nullptr;
 }
 
 static int32_t latent_mma_setup(const MixPlan& x) {
     for (int rows : {16, 32, 64}) {
-        int tr, tp;
+        int tr, gr;
         size_t smem;
-        LatentMmaFn fn = pick_latent_mma(x.rank, x.ld, rows, &tr, &tp, &smem);
+        LatentMmaFn fn = pick_latent_mma(x.rank, x.ld, rows, &tr, &gr, &smem);
         if (fn) TRY(allow_big_smem(fn));
     }
     return OXG4_OK;
 }
 
 // Splits of `tiles` cache tiles when `units` row tiles share the GPU: the cheapest number of rounds times tiles per CTA, with
-// about three tiles' worth of start-up per CTA and a little for every partial the merge has to read.
+// about four tiles' worth of start-up per CTA and a little for every partial the merge has to read.
 static int latent_splits(int units, int tiles, int most, int num_sms) {
     int best = 1;
     double best_cost = 1e30;
     for (int s = 1; s <= std::min(most, std::max(1, tiles)); ++s) {
         const double rounds = (units * s + num_sms - 1) / num_sms;
-        const double cost = rounds * ((tiles + s - 1) / s + 3) + 0.05 * s;
+        const double cost = rounds * ((tiles + s - 1) / s + 4) + 0.1 * s;
         if (cost < best_cost - 1e-9) { best_cost = cost; best = s; }
     }
     return best;
@@ -713,17 +720,17 @@ struct LayeredPass {
             q = project("uq", x.uq, c->x_q, c->q_buf);
         }
         LatentPart part{c->lat_o, c->lat_ml, rs.chunk ? 1 : c->lat_splits, (size_t)R * x.heads};
-        int tile_rows = 0, tile_pos = 1;
+        int tile_rows = 0, groups = 1;
         size_t mma_smem = 0;
         int longest = 1;
         for (int n : rs.run_len) longest = std::max(longest, n);
-        const LatentMmaFn mma = sizeof(WT) == 2 && sizeof(KT) == 2 ? pick_latent_mma(x.rank, x.ld, longest * x.heads, &tile_rows, &tile_pos, &mma_smem) : nullptr;
+        const LatentMmaFn mma = sizeof(WT) == 2 && sizeof(KT) == 2 ? pick_latent_mma(x.rank, x.ld, longest * x.heads, &tile_rows, &groups, &mma_smem) : nullptr;
         LatentMmaArgs ma{};
         int mma_tiles = 0;
         if (mma) {
             for (int n : rs.run_len) mma_tiles += (n * x.heads + tile_rows - 1) / tile_rows;
-            part.splits = latent_splits(mma_tiles, (rs.max_visible + tile_pos - 1) / tile_pos, rs.chunk ? kLatentChunkSplits : c->lat_splits,
-                                        m->num_sms);
+            const int most = rs.chunk ? kLatentChunkSplits : c->lat_splits, visible_tiles = (rs.max_visible + kLmTile - 1) / kLmTile;
+            part.splits = groups * latent_splits(mma_tiles, (visible_tiles + groups - 1) / groups, std::max(1, most / groups), m->num_sms);
             ma.heads = x.heads; ma.rank = x.rank; ma.rot = x.rot;
             ma.scale = x.scale;
             ma.rows = a.rows;
@@ -737,7 +744,7 @@ struct LayeredPass {
             ln.tc("uk", c, R, x.uk.w, nullptr, (const uint16_t*)c->x_u, x.uk.N, x.uk.K, 1, c->uk_buf, x.uk.N, 0, x.uk.seg_rows / kTcTileM);
             ma.q_abs = c->uk_buf; ma.abs_row = x.uk.N; ma.abs_head = x.uk.seg_rows;
             ma.q_rot = c->lat_rot; ma.rot_row = (size_t)x.heads * x.rot; ma.rot_head = x.rot;
-            ln.go("attn", mma, dim3(mma_tiles, part.splits), dim3(kLmThreads), mma_smem, ma);
+            ln.go("attn", mma, dim3(mma_tiles, part.splits / groups), dim3(kLmThreads * groups), mma_smem, ma);
             ln.go("latmerge", latent_merge_kernel, dim3(x.heads, R), dim3(128), sizeof(float) * part.splits, R, x.heads, x.rank, part,
                   (uint16_t*)c->x_l, x.uv.K);
             const SplitIn o = project("uv", x.uv, c->x_l, c->uv_buf);
@@ -749,7 +756,7 @@ struct LayeredPass {
         if (mma) {
             ma.q_abs = c->lat_q; ma.abs_row = (size_t)x.heads * (x.rank + x.rot); ma.abs_head = x.rank + x.rot;
             ma.q_rot = c->lat_q + x.rank; ma.rot_row = ma.abs_row; ma.rot_head = ma.abs_head;
-            ln.go("attn", mma, dim3(mma_tiles, part.splits), dim3(kLmThreads), mma_smem, ma);
+            ln.go("attn", mma, dim3(mma_tiles, part.splits / groups), dim3(kLmThreads * groups), mma_smem, ma);
         } else {
             LatentAttnFn fn = pick_latent_attn<KT>(x.rank);
             ln.go("attn", fn, dim3(x.heads, R, part.splits), dim3(256), sizeof(float) * (x.rank + x.rot + 8 * x.rank + 16), a, (const float*)c->lat_q, part);
