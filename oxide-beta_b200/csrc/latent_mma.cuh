@@ -7,8 +7,8 @@
 // stages, each row read once: the first `rank` elements of a row are the value, all of it is the key. GR groups of 8 warps
 // share the query tile and are otherwise independent: each walks its own split of the positions with its own ring and its
 // own barrier, so one group's barriers and softmax hide behind the other's products. A group of 8 warps:
-//   S = Q K^T   16 x 8 tiles of the score block dealt to the warps (with one row tile two warps share a score tile, half of
-//               the columns each), f32 accumulation, into shared memory
+//   S = Q K^T   a warp takes all rows, 16 positions and a quarter of the columns, so that shared memory is read little more
+//               than once; f32 accumulation, the four partial scores meet in shared memory
 //   softmax     256 / (16 MT) neighbouring threads per row; running maximum and sum in f32; the weights are split into BF16
 //               high and low parts, so their products with the BF16 values lose nothing that f32 would keep
 //   O += P V    every warp owns NT * 8 latent columns of all rows
@@ -31,6 +31,7 @@ struct LatentMmaArgs {
     float scale;
     RunRows rows;
     int runs;
+    int step_tiles;                      // > 0: a decode step (run r is row r, one token): row tiles per run
     LatentCache cache;
     LatentPart part;
 };
@@ -42,13 +43,15 @@ DEVINL void cp_async16(uint32_t dst, const void* src, bool valid) {
 DEVINL void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> DEVINL void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// warps that share a score tile, each with a part of the columns
-template <int MT> struct LmGeom { static constexpr int KSP = MT * (kLmTile / 8) < kLmWarps ? kLmWarps / (MT * (kLmTile / 8)) : 1; };
+constexpr int kLmKS = 4;                             // quarters of the columns in the score products
+// A row's scores, four partial sums of 36 floats each; the row's weights (high and low BF16 parts) replace them. The stride is
+// an odd number of 16-byte pieces: ldmatrix without bank conflicts.
+constexpr int kLmRowBytes = 592, kLmScoreLd = 36, kLmLowBytes = 80;
 
-// shared memory of a group besides the query tile: ring, weights (high, low), scores, rescale factors
+// shared memory of a group besides the query tile: ring, scores / weights, rescale factors
 template <int MT, int NST>
 __host__ __device__ constexpr size_t latent_mma_group_bytes(int ld) {
-    return (size_t)NST * kLmTile * (ld + 8) * 2 + 2 * MT * 16 * (kLmTile + 8) * 2 + LmGeom<MT>::KSP * MT * 16 * (kLmTile + 4) * 4 + MT * 16 * 4;
+    return (size_t)NST * kLmTile * (ld + 8) * 2 + MT * 16 * kLmRowBytes + MT * 16 * 4;
 }
 template <int MT, int NST, int GR>
 inline size_t latent_mma_smem(int ld) {
@@ -59,29 +62,27 @@ inline size_t latent_mma_smem(int ld) {
 template <int MT, int NT, int NST, int GR>
 __global__ void __launch_bounds__(kLmThreads * GR, 1) latent_mma_kernel(const LatentMmaArgs a) {
     constexpr int ROWS = MT * 16, NB = kLmTile;
-    constexpr int SN = NB / 8;                       // score columns in MMA tiles
-    constexpr int KSP = LmGeom<MT>::KSP;
-    constexpr int SPW = MT * SN * KSP / kLmWarps;    // score tiles per warp
-    static_assert(MT * SN * KSP % kLmWarps == 0 && SPW <= 2 && NT % 2 == 0, "tile shape");
+    // one row tile: the warp's query fragments stay in registers (two groups fit only for cache rows below 768 elements)
+    constexpr bool QREG = MT == 1 && GR == 2;
+    constexpr int QSTEPS = QREG ? 768 / 16 / kLmKS : 1;
+    static_assert(kLmWarps == 2 * kLmKS && NB == 32 && NT % 2 == 0, "tile shape");
     constexpr int TPR = kLmThreads / ROWS;           // threads per row in the softmax
     constexpr int PPT = NB / TPR;                    // positions per thread
     constexpr int RPW = NB / kLmWarps;               // cache rows a warp loads per tile
-    constexpr int PLD = NB + 8, SLD = NB + 4;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int ld = a.cache.ld, ldp = ld + 8, DK = a.rank + a.rot;
     const int grp = GR > 1 ? threadIdx.x / kLmThreads : 0, tid = threadIdx.x % kLmThreads, lane = tid & 31, warp = tid >> 5;
     uint16_t* sq = reinterpret_cast<uint16_t*>(smem_raw);            // [ROWS][ldp]
     int* s_pos = reinterpret_cast<int*>(sq + (size_t)ROWS * ldp);    // [ROWS] last visible position, -1: no row
     uint16_t* skv = reinterpret_cast<uint16_t*>(reinterpret_cast<unsigned char*>(s_pos + ROWS) + grp * latent_mma_group_bytes<MT, NST>(ld));
-    uint16_t* sp = skv + (size_t)NST * NB * ldp;                     // ring [NST][NB][ldp], then [2 (hi, lo)][ROWS][PLD]
-    float* ss = reinterpret_cast<float*>(sp + 2 * ROWS * PLD);       // [KSP][ROWS][SLD]
-    float* s_alpha = ss + KSP * ROWS * SLD;                          // [ROWS]
+    unsigned char* sp = reinterpret_cast<unsigned char*>(skv + (size_t)NST * NB * ldp);   // [ROWS] rows of kLmRowBytes
+    float* s_alpha = reinterpret_cast<float*>(sp + ROWS * kLmRowBytes);      // [ROWS]
     __shared__ int s_run, s_first;
     pdl_wait();
     pdl_launch();
     // the longest rows are at the end of a run: they start first
     const int t = gridDim.x - 1 - blockIdx.x;
-    if (threadIdx.x < 32) {
+    if (a.step_tiles == 0 && threadIdx.x < 32) {
         int base = 0, run = -1, first = 0;
         for (int r0 = 0; r0 < a.runs && run < 0; r0 += 32) {
             const int r = r0 + lane;
@@ -103,10 +104,19 @@ __global__ void __launch_bounds__(kLmThreads * GR, 1) latent_mma_kernel(const La
         }
         if (lane == 0) { s_run = run; s_first = first; }
     }
-    __syncthreads();
-    const int run = s_run, first = s_first;
-    if (run < 0) return;
-    const int row0 = a.rows.row0[run], n_flat = a.rows.n[run] * a.heads;
+    int run, first, row0, n_flat;
+    if (a.step_tiles > 0) {
+        run = row0 = t / a.step_tiles;
+        first = t % a.step_tiles * ROWS;
+        n_flat = a.heads;
+    } else {
+        __syncthreads();
+        run = s_run;
+        first = s_first;
+        if (run < 0) return;
+        row0 = a.rows.row0[run];
+        n_flat = a.rows.n[run] * a.heads;
+    }
     if (a.rows.tok[row0] == kInactiveToken) return;
     const int seq = a.rows.seq_of(row0);
     const int n_here = min(ROWS, n_flat - first);
@@ -182,12 +192,16 @@ __global__ void __launch_bounds__(kLmThreads * GR, 1) latent_mma_kernel(const La
     const float scale2 = a.scale * 1.4426950408889634f;              // scores in units of log 2
     float m_run = -INFINITY, l_run = 0.0f;                           // of row srow (the same in its TPR threads)
     const int my_pos = s_pos[srow];
-    // score tiles of this warp: one row tile, SPW neighbouring column tiles, nk steps of 16 columns from s_k0 on
-    const int s_mi = warp % MT, s_n0 = (warp / MT) % (SN / SPW) * SPW, s_kh = warp / (MT * (SN / SPW));
-    const int half = (ld / 32 + KSP - 1) / KSP * 32;
-    const int s_k0 = KSP > 1 ? min(ld, s_kh * half) : 0, s_k1 = KSP > 1 && s_kh == 0 ? min(ld, half) : ld;
-    const int nk = (s_k1 - s_k0) / 16;                               // ld is a multiple of 16
-    const uint32_t q_base = smem_u32(sq) + ((s_mi * 16 + (lane & 15)) * ldp + (lane >> 4) * 8 + s_k0) * 2;
+    // scores of this warp: 16 positions from s_n0 on, nk steps of 16 columns from s_k0 on (ld is a multiple of 16)
+    const int steps = (ld / 16 + kLmKS - 1) / kLmKS, s_kq = warp / 2, s_n0 = (warp & 1) * 16;
+    const int s_k0 = min(ld, s_kq * steps * 16), nk = min(ld - s_k0, steps * 16) / 16;
+    const uint32_t q_base = smem_u32(sq) + ((lane & 15) * ldp + (lane >> 4) * 8 + s_k0) * 2;
+    uint32_t qf[QSTEPS][4];
+    if constexpr (QREG) {
+#pragma unroll
+        for (int k = 0; k < QSTEPS; ++k)
+            if (k < nk) ldmatrix_x4(qf[k], q_base + k * 32);
+    }
     const int v_col0 = warp * NT * 8;
     int stage = 0;
     for (int tile = tile0; tile < tile1; ++tile) {
@@ -202,52 +216,43 @@ __global__ void __launch_bounds__(kLmThreads * GR, 1) latent_mma_kernel(const La
         const uint32_t kv = smem_u32(skv + (size_t)stage * NB * ldp);
         stage = stage + 1 == NST ? 0 : stage + 1;
         {
-            float s[SPW][4], s2[SPW][4];
+            float s[MT][2][4];
 #pragma unroll
-            for (int j = 0; j < SPW; ++j) {
-                s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
-                s2[j][0] = s2[j][1] = s2[j][2] = s2[j][3] = 0.0f;
-            }
-            if constexpr (SPW == 1) {
-                // one column tile: a load brings its 8 positions for two k-steps
-                const uint32_t kb = kv + ((s_n0 * 8 + (lane & 7)) * ldp + (lane >> 3) * 8 + s_k0) * 2;
-                int k = 0;
-#pragma unroll 3
-                for (; k + 2 <= nk; k += 2) {
-                    uint32_t q0[4], q1[4], b[4];
-                    ldmatrix_x4(b, kb + k * 32);
-                    ldmatrix_x4(q0, q_base + k * 32);
-                    ldmatrix_x4(q1, q_base + k * 32 + 32);
-                    mma_bf16_16816(s[0], q0, b[0], b[1]);
-                    mma_bf16_16816(s2[0], q1, b[2], b[3]);
-                }
-                if (k < nk) {
-                    // a single step: the upper half of the lanes addresses the same columns again, no read behind the row
-                    uint32_t q0[4], b[4];
-                    ldmatrix_x4(b, kv + ((s_n0 * 8 + (lane & 7)) * ldp + ((lane >> 3) & 1) * 8 + s_k0) * 2 + k * 32);
-                    ldmatrix_x4(q0, q_base + k * 32);
-                    mma_bf16_16816(s[0], q0, b[0], b[1]);
-                }
+            for (int i = 0; i < MT; ++i)
+#pragma unroll
+                for (int j = 0; j < 2; ++j) s[i][j][0] = s[i][j][1] = s[i][j][2] = s[i][j][3] = 0.0f;
+            const uint32_t kb = kv + ((s_n0 + (lane >> 4) * 8 + (lane & 7)) * ldp + ((lane >> 3) & 1) * 8 + s_k0) * 2;
+            if constexpr (QREG) {
+#pragma unroll
+                for (int k = 0; k < QSTEPS; ++k)
+                    if (k < nk) {
+                        uint32_t b[4];
+                        ldmatrix_x4(b, kb + k * 32);
+                        mma_bf16_16816(s[0][0], qf[k], b[0], b[1]);
+                        mma_bf16_16816(s[0][1], qf[k], b[2], b[3]);
+                    }
             } else {
-                // a pair of column tiles: a load brings 16 positions for one k-step
-                const uint32_t kb = kv + ((s_n0 * 8 + (lane >> 4) * 8 + (lane & 7)) * ldp + ((lane >> 3) & 1) * 8 + s_k0) * 2;
-#pragma unroll 4
+#pragma unroll 3
                 for (int k = 0; k < nk; ++k) {
-                    uint32_t q0[4], b[4];
-                    ldmatrix_x4(q0, q_base + k * 32);
+                    uint32_t b[4], q[MT][4];
                     ldmatrix_x4(b, kb + k * 32);
-                    mma_bf16_16816((k & 1) ? s2[0] : s[0], q0, b[0], b[1]);
-                    mma_bf16_16816((k & 1) ? s2[SPW - 1] : s[SPW - 1], q0, b[2], b[3]);
+#pragma unroll
+                    for (int i = 0; i < MT; ++i) ldmatrix_x4(q[i], q_base + i * 16 * ldp * 2 + k * 32);
+#pragma unroll
+                    for (int i = 0; i < MT; ++i) {
+                        mma_bf16_16816(s[i][0], q[i], b[0], b[1]);
+                        mma_bf16_16816(s[i][1], q[i], b[2], b[3]);
+                    }
                 }
             }
-            const int r0 = s_mi * 16 + (lane >> 2);
-            float* dst = ss + (KSP > 1 ? s_kh : 0) * ROWS * SLD;
 #pragma unroll
-            for (int j = 0; j < SPW; ++j) {
-                const int c = (s_n0 + j) * 8 + (lane & 3) * 2;
-                *reinterpret_cast<float2*>(dst + r0 * SLD + c) = make_float2(s[j][0] + s2[j][0], s[j][1] + s2[j][1]);
-                *reinterpret_cast<float2*>(dst + (r0 + 8) * SLD + c) = make_float2(s[j][2] + s2[j][2], s[j][3] + s2[j][3]);
-            }
+            for (int i = 0; i < MT; ++i)
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    float* dst = reinterpret_cast<float*>(sp + (i * 16 + (lane >> 2)) * kLmRowBytes) + s_kq * kLmScoreLd + s_n0 + j * 8 + (lane & 3) * 2;
+                    *reinterpret_cast<float2*>(dst) = make_float2(s[i][j][0], s[i][j][1]);
+                    *reinterpret_cast<float2*>(dst + 8 * kLmRowBytes / 4) = make_float2(s[i][j][2], s[i][j][3]);
+                }
         }
         group_sync();
         {
@@ -256,10 +261,11 @@ __global__ void __launch_bounds__(kLmThreads * GR, 1) latent_mma_kernel(const La
 #pragma unroll
             for (int j = 0; j < PPT; j += 2) {                       // pairs of neighbouring positions
                 const int c = 2 * sub + j * TPR;
-                float2 x = *reinterpret_cast<const float2*>(ss + srow * SLD + c);
+                const float* src = reinterpret_cast<const float*>(sp + srow * kLmRowBytes) + c;
+                float2 x = *reinterpret_cast<const float2*>(src);
 #pragma unroll
-                for (int q = 1; q < KSP; ++q) {
-                    const float2 y = *reinterpret_cast<const float2*>(ss + (q * ROWS + srow) * SLD + c);
+                for (int q = 1; q < kLmKS; ++q) {
+                    const float2 y = *reinterpret_cast<const float2*>(src + q * kLmScoreLd);
                     x.x += y.x;
                     x.y += y.y;
                 }
@@ -273,6 +279,7 @@ __global__ void __launch_bounds__(kLmThreads * GR, 1) latent_mma_kernel(const La
             const float base = m_new == -INFINITY ? 0.0f : m_new;    // a row without a visible position so far
             const float alpha = m_new == m_run ? 1.0f : exp2f(m_run - base);
             float sum = 0.0f;
+            __syncwarp();                                            // a row's threads are one warp's: its scores are all read
 #pragma unroll
             for (int j = 0; j < PPT; j += 2) {
                 const float e0 = exp2f(v[j] - base), e1 = exp2f(v[j + 1] - base);
@@ -280,8 +287,8 @@ __global__ void __launch_bounds__(kLmThreads * GR, 1) latent_mma_kernel(const La
                 uint32_t hi, lo;
                 split_pack(e0, e1, hi, lo);
                 const int c = 2 * sub + j * TPR;
-                *reinterpret_cast<uint32_t*>(sp + srow * PLD + c) = hi;
-                *reinterpret_cast<uint32_t*>(sp + (ROWS + srow) * PLD + c) = lo;
+                *reinterpret_cast<uint32_t*>(sp + srow * kLmRowBytes + c * 2) = hi;
+                *reinterpret_cast<uint32_t*>(sp + srow * kLmRowBytes + kLmLowBytes + c * 2) = lo;
             }
             l_run = l_run * alpha + sum;                             // this thread's positions only; added up at the end
             m_run = m_new;
@@ -306,15 +313,15 @@ __global__ void __launch_bounds__(kLmThreads * GR, 1) latent_mma_kernel(const La
                         acc[i][j][2] *= al[i][1]; acc[i][j][3] *= al[i][1];
                     }
             }
-            const uint32_t p_base = smem_u32(sp) + ((lane & 15) * PLD + (lane >> 4) * 8) * 2;
+            const uint32_t p_base = smem_u32(sp) + (lane & 15) * kLmRowBytes + (lane >> 4) * 16;
             const uint32_t v_base = kv + ((lane & 15) * ldp + v_col0 + (lane >> 4) * 8) * 2;
 #pragma unroll
             for (int k = 0; k < NB; k += 16) {
                 uint32_t ph[MT][4], pl[MT][4];
 #pragma unroll
                 for (int i = 0; i < MT; ++i) {
-                    ldmatrix_x4(ph[i], p_base + (i * 16 * PLD + k) * 2);
-                    ldmatrix_x4(pl[i], p_base + ((ROWS + i * 16) * PLD + k) * 2);
+                    ldmatrix_x4(ph[i], p_base + i * 16 * kLmRowBytes + k * 2);
+                    ldmatrix_x4(pl[i], p_base + i * 16 * kLmRowBytes + kLmLowBytes + k * 2);
                 }
 #pragma unroll
                 for (int j = 0; j < NT; j += 2) {

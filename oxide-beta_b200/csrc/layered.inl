@@ -735,6 +735,7 @@ struct LayeredPass {
             ma.scale = x.scale;
             ma.rows = a.rows;
             ma.runs = (int)rs.run_len.size();
+            ma.step_tiles = rs.chunk ? 0 : (x.heads + tile_rows - 1) / tile_rows;
             ma.cache = a.cache;
             ma.part = part;
         }
