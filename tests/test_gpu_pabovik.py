@@ -35,6 +35,9 @@ MECHANISMS = {
     "latent_one_head": [latent(1, 8, 8, 8, 16, 4, ff=16)],
     "latent_rank_200": [latent(7, 32, 48, 96, 200, 16)],
     "latent_rank_512": [latent(9, 32, 24, 64, 512, 64)],
+    "latent_shared_tensors": [latent(4, 16, 16, 24, 40, 8, ff=32), wkv(2, 12), latent(4, 16, 16, 24, 40, 8, ff=32, weights_of=0)],
+    "wkv_many_heads": [wkv(150, 8)],
+    "lightning_many_heads": [lightning(149, 8, 6, np.linspace(0.3, 1.0, 149))],
     "latent_many_heads": [latent(33, 16, 16, 64, 96, 8)],
     "latent_wide_rotation": [latent(3, 16, 16, 32, 304, 300)],
     "feed_forward": [wkv(1, 8, ff=300)],
