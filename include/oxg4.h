@@ -74,15 +74,26 @@ typedef struct {
     int32_t vocab_size_per_layer_input;  /* rows of embed_tokens_per_layer.weight                        */
 } oxg4_config;
 
-/* Models whose layers are listed one by one, each with its own mixer, sizes and (optional) feed-forward, between
- * norms before and after every sublayer: x += norm_b(f(norm(x))). No counterpart in the reference. Everything but
- * model creation goes through the same entry points as a Gemma 4 model. */
+/* Models whose layers are listed one by one, each with its own mixer, sizes and (optional) feed-forward. No counterpart
+ * in the reference. Everything but model creation goes through the same entry points as a Gemma 4 model. */
 typedef enum {
     OXG4_MIXER_GQA = 0,               /* the attention of the Gemma 4 models; not valid in a layer list */
     OXG4_MIXER_LATENT_ATTENTION = 1,  /* low-rank queries, one cached latent and one rotated key part per token */
     OXG4_MIXER_LIGHTNING = 2,         /* linear attention with a fixed decay per head                          */
-    OXG4_MIXER_WKV = 3                /* RWKV-style time mixing: token shift, decay per token and channel      */
+    OXG4_MIXER_WKV = 3,               /* RWKV-style time mixing: token shift, decay per token and channel      */
+    OXG4_MIXER_RETENTION = 4,         /* linear attention with a fixed decay per head, rotated queries and keys,
+                                         every head's output normed and gated                                  */
+    OXG4_MIXER_ATTENTION = 5          /* grouped-query attention: biases, q and k normed over all heads at once,
+                                         position-dependent query factor, a sink in the softmax; no rotation   */
 } oxg4_mixer;
+
+/* How mixer and feed-forward of a listed layer meet the residual stream. */
+typedef enum {
+    OXG4_BLOCK_SANDWICH = 0,          /* x += norm1b(mixer(norm1(x))); x += norm2b(ff(norm2(x)))               */
+    OXG4_BLOCK_PARALLEL = 1           /* h = norm1(x); x += mixer(h) + ff(h)                                   */
+} oxg4_block;
+
+typedef enum { OXG4_ACT_GELU_TANH = 0, OXG4_ACT_SILU = 1, OXG4_ACT_RELU = 4 } oxg4_activation;
 
 typedef struct {
     int32_t mixer;                    /* oxg4_mixer                                                            */
@@ -92,12 +103,16 @@ typedef struct {
     int32_t q_rank;                   /* latent attention: query latent                                        */
     int32_t kv_rank;                  /*                   cached latent                                       */
     int32_t rot_dim;                  /*                   rotated part of queries and keys                    */
-    int32_t rot_dims;                 /*                   how many of its dimensions turn                     */
+    int32_t rot_dims;                 /*                   how many of its dimensions turn; retention: the first
+                                                           rot_dims of every head of q and k                   */
     float rot_base;
-    float scale;                      /*                   factor on the scores                                */
-    const float* decay;               /* lightning: [heads]                                                    */
-    int32_t ff;                       /* SiLU-gated feed-forward of this width after the mixer; 0 = none       */
+    float scale;                      /* both attentions: factor on the scores                                 */
+    const float* decay;               /* lightning, retention: [heads]                                         */
+    int32_t ff;                       /* gated feed-forward of this width; 0 = none                            */
     int32_t weights_of;               /* -1, or the layer whose tensors this layer uses (own cache and state)  */
+    int32_t kv_heads;                 /* attention: key/value heads                                            */
+    float q_temp_coef;                /*            queries at position p are multiplied by                    */
+    int32_t q_temp_every;             /*            1 + coef * ln(floor((p + 1) / every) + 1)                  */
 } oxg4_layer_spec;
 
 typedef struct {
@@ -106,6 +121,9 @@ typedef struct {
     int32_t num_layers;
     float norm_eps;
     int32_t weight_dtype;             /* as in oxg4_config                                                     */
+    int32_t block;                    /* oxg4_block                                                            */
+    int32_t act;                      /* oxg4_activation of the feed-forward's gate                            */
+    int32_t norm_weight_offset;       /* 1: the weights of the block and final norms are stored around zero    */
     const oxg4_layer_spec* layers;    /* [num_layers]                                                          */
 } oxg4_layered_config;
 

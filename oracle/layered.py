@@ -1,5 +1,6 @@
-"""Plain restatement, in numpy and double precision, of models whose layers are listed one by one (the Pabovik
-design): latent attention, lightning attention and RWKV-style time mixing between sandwich norms. One function per
+"""Plain restatement, in numpy and double precision, of models whose layers are listed one by one. Pabovik: latent
+attention, lightning attention and RWKV-style time mixing between sandwich norms. Nozurax: retention and grouped-query
+attention with a sink, in parallel with the feed-forward behind one norm. One function per
 mechanism, whole sequences at a time, no cache and no chunks. Test infrastructure only: nothing of the product
 path is imported, and nothing of this file is used by it.
 
@@ -33,15 +34,32 @@ def rotate_interleaved(x, positions, dims, base):
     return out
 
 
-def causal_softmax_attention(q, k, v, scale):
-    """q, k [T, H, D], v [T, H, Dv] -> [T, H, Dv]."""
+def rotate_half(x, positions, dims, base):
+    """x [T, ..., D]: the pairs (i, i + dims / 2) of the first `dims` entries turn by position * base^(-2i / dims)."""
+    out = np.array(x, dtype=np.float64)
+    half = dims // 2
+    for i in range(half):
+        a = np.asarray(positions, dtype=np.float64) * float(base) ** (-2.0 * i / dims)
+        a = a.reshape((-1,) + (1,) * (x.ndim - 2))
+        u, v = x[..., i], x[..., i + half]
+        out[..., i] = u * np.cos(a) - v * np.sin(a)
+        out[..., i + half] = v * np.cos(a) + u * np.sin(a)
+    return out
+
+
+def causal_softmax_attention(q, k, v, scale, sink=None):
+    """q, k [T, H, D], v [T, H, Dv] -> [T, H, Dv]. sink [H]: one more term exp(sink) of the denominator, without a value."""
     T = q.shape[0]
     s = np.einsum("thd,shd->hts", q, k) * scale
     s = np.where(np.tril(np.ones((T, T), dtype=bool))[None], s, -np.inf)
-    s -= s.max(axis=-1, keepdims=True)
-    e = np.exp(s)
-    e /= e.sum(axis=-1, keepdims=True)
-    return np.einsum("hts,shd->thd", e, v)
+    top = s.max(axis=-1, keepdims=True)
+    if sink is not None:
+        top = np.maximum(top, np.asarray(sink)[:, None, None])
+    e = np.exp(s - top)
+    total = e.sum(axis=-1, keepdims=True)
+    if sink is not None:
+        total = total + np.exp(np.asarray(sink)[:, None, None] - top)
+    return np.einsum("hts,shd->thd", e / total, v)
 
 
 def latent_attention(h, W, p, c, eps):
@@ -113,11 +131,44 @@ def wkv(h, W, p, c, eps):
     return o @ W[p + "mix.o"].T
 
 
-def dense_ff(h, W, p):
-    return (silu(h @ W[p + "mlp.gate"].T) * (h @ W[p + "mlp.up"].T)) @ W[p + "mlp.down"].T
+def retention(h, W, p, c, eps):
+    """Linear attention with a fixed decay per head, rotated queries and keys, every head's output normed and gated."""
+    T, H, D = h.shape[0], c["heads"], c["dim"]
+    pos, rot = np.arange(T), c["rot"]
+    q = rotate_half((h @ W[p + "mix.q"].T).reshape(T, H, D), pos, rot["dims"], rot["base"])
+    k = rotate_half((h @ W[p + "mix.k"].T).reshape(T, H, D), pos, rot["dims"], rot["base"]) * D ** -0.5
+    v = (h @ W[p + "mix.v"].T).reshape(T, H, c["vdim"])
+    o = rms_norm(lightning_scan(q, k, v, c["decay"]), None, eps).reshape(T, H * c["vdim"])
+    return (o * silu(h @ W[p + "mix.g"].T)) @ W[p + "mix.o"].T
 
 
-MIXERS = {"latent_attention": latent_attention, "lightning": lightning, "wkv": wkv}
+def query_temperature(positions, coef, every):
+    return 1.0 + coef * np.log(np.floor((np.asarray(positions) + 1) / every) + 1.0)
+
+
+def sink_attention(h, W, p, c, eps):
+    """Grouped-query attention without rotation: biases, q and k normed over all their heads at once, queries scaled with
+    the logarithm of the position, a learned sink per head in the denominator."""
+    T, H, G, D = h.shape[0], c["heads"], c["kv_heads"], c["dim"]
+    q = rms_norm(h @ W[p + "mix.q"].T + W[p + "mix.q.b"], W[p + "mix.q.norm"], eps).reshape(T, H, D)
+    k = rms_norm(h @ W[p + "mix.k"].T + W[p + "mix.k.b"], W[p + "mix.k.norm"], eps).reshape(T, G, D)
+    v = (h @ W[p + "mix.v"].T + W[p + "mix.v.b"]).reshape(T, G, c["vdim"])
+    q = q * query_temperature(np.arange(T), c["q_temp"]["coef"], c["q_temp"]["every"])[:, None, None]
+    shared = np.arange(H) // (H // G)
+    o = causal_softmax_attention(q, k[:, shared], v[:, shared], c["scale"], W[p + "mix.sink"])
+    return o.reshape(T, H * c["vdim"]) @ W[p + "mix.o"].T
+
+
+def relu(z):
+    return np.maximum(z, 0.0)
+
+
+def dense_ff(h, W, p, act=silu):
+    return (act(h @ W[p + "mlp.gate"].T) * (h @ W[p + "mlp.up"].T)) @ W[p + "mlp.down"].T
+
+
+MIXERS = {"latent_attention": latent_attention, "lightning": lightning, "wkv": wkv, "retention": retention,
+          "attention": sink_attention}
 
 
 def weights_layer(layers, i):
@@ -126,18 +177,32 @@ def weights_layer(layers, i):
     return i
 
 
+def sandwich_layer(x, layer, W, p, eps):
+    y = MIXERS[layer["type"]](rms_norm(x, W[p + "norm1"], eps), W, p, layer["mixer"], eps)
+    x = x + rms_norm(y, W[p + "norm1b"], eps)
+    if layer.get("mlp"):
+        y = dense_ff(rms_norm(x, W[p + "norm2"], eps), W, p)
+        x = x + rms_norm(y, W[p + "norm2b"], eps)
+    return x
+
+
+def parallel_layer(x, layer, W, p, eps):
+    """One norm, its weight stored around zero; mixer and feed-forward read the same input."""
+    h = rms_norm(x, 1.0 + W[p + "norm1"], eps)
+    y = MIXERS[layer["type"]](h, W, p, layer["mixer"], eps)
+    return x + (y + dense_ff(h, W, p, relu) if layer.get("mlp") else y)
+
+
 def forward(cfg, W, tokens):
     """(logits [T, vocab], residual stream after every layer [layers, T, width])."""
     W = {n: np.asarray(a, dtype=np.float64) for n, a in W.items()}
     eps = cfg["norm"]["eps"]
+    parallel = cfg["architecture"] == "Nozurax"
     x = W["embed"][np.asarray(tokens)]
     after = []
     for i, layer in enumerate(cfg["layers"]):
         p = f"l{weights_layer(cfg['layers'], i)}."
-        y = MIXERS[layer["type"]](rms_norm(x, W[p + "norm1"], eps), W, p, layer["mixer"], eps)
-        x = x + rms_norm(y, W[p + "norm1b"], eps)
-        if layer.get("mlp"):
-            y = dense_ff(rms_norm(x, W[p + "norm2"], eps), W, p)
-            x = x + rms_norm(y, W[p + "norm2b"], eps)
+        x = (parallel_layer if parallel else sandwich_layer)(x, layer, W, p, eps)
         after.append(x)
-    return rms_norm(x, W["final.norm"], eps) @ W["head"].T, np.stack(after)
+    final = 1.0 + W["final.norm"] if parallel else W["final.norm"]
+    return rms_norm(x, final, eps) @ W["head"].T, np.stack(after)

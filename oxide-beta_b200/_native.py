@@ -33,16 +33,20 @@ class Config(C.Structure):
 class LayerSpec(C.Structure):
     _fields_ = [("mixer", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("q_rank", C.c_int32),
                 ("kv_rank", C.c_int32), ("rot_dim", C.c_int32), ("rot_dims", C.c_int32), ("rot_base", C.c_float),
-                ("scale", C.c_float), ("decay", C.POINTER(C.c_float)), ("ff", C.c_int32), ("weights_of", C.c_int32)]
+                ("scale", C.c_float), ("decay", C.POINTER(C.c_float)), ("ff", C.c_int32), ("weights_of", C.c_int32),
+                ("kv_heads", C.c_int32), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int32)]
 
 
 class LayeredConfig(C.Structure):
     _fields_ = [("vocab_size", C.c_int32), ("width", C.c_int32), ("num_layers", C.c_int32), ("norm_eps", C.c_float),
-                ("weight_dtype", C.c_int32), ("layers", C.POINTER(LayerSpec))]
+                ("weight_dtype", C.c_int32), ("block", C.c_int32), ("act", C.c_int32), ("norm_weight_offset", C.c_int32),
+                ("layers", C.POINTER(LayerSpec))]
 
 
-# oxg4_mixer
-MIXERS = {"latent_attention": 1, "lightning": 2, "wkv": 3}
+# oxg4_mixer, oxg4_block, oxg4_activation
+MIXERS = {"latent_attention": 1, "lightning": 2, "wkv": 3, "retention": 4, "attention": 5}
+BLOCK_SANDWICH, BLOCK_PARALLEL = 0, 1
+ACTIVATIONS = {"gelu_tanh": 0, "silu": 1, "relu": 4}
 
 
 class CacheInfo(C.Structure):

@@ -7,7 +7,8 @@
 //   rows_norm_kernel  the reference's rms_norm + add + mul_bf16_scalar + rms_norm_bf16 chain
 //                     (gemma4_cuda/decode.rs:14,19-20,61-65,161-171,362-367; kernel_module.rs:1133-1211):
 //                     h = (h_in + rmsnorm(sum of the projection's K-split partials, w_post)) * layer_scalar
-//                     (or h = embedding row * sqrt(H), or h = h_in), x = bf16(rmsnorm(h, w_norm))
+//                     (or h = embedding row * sqrt(H), or h = h_in, or without the norm where w_post is null),
+//                     x = bf16(rmsnorm(h, w_norm))
 //   geglu_rows_kernel gelu_mul_f32 + f32_to_bf16 (decode.rs:17, kernel_module.rs:1441-1458, 1338-1348)
 #pragma once
 #include "common.cuh"
@@ -57,7 +58,7 @@ struct RowsNormArgs {
     float* h_out;            // [B, H]
     const float* raw;        // [raw_splits, B, H] partial outputs of the previous projection, or null
     int raw_splits;
-    const float* w_post;
+    const float* w_post;     // null: raw is added as it is
     float scalar;
     const float* w_norm;
     const void* embed;       // [V, H] embedding table (BF16 or f32, the type of x), or null
@@ -156,13 +157,17 @@ __global__ void __launch_bounds__(kRowsThreads) rows_norm_kernel(const RowsNormA
             ss[0] += t[j].z * t[j].z;
             ss[0] += t[j].w * t[j].w;
         }
-        block_sum<1>(ss, red);
-        const float r = 1.0f / sqrtf(ss[0] / norm_n + a.eps);
+        float r = 1.0f;
+        if (a.w_post != nullptr) {
+            block_sum<1>(ss, red);
+            r = 1.0f / sqrtf(ss[0] / norm_n + a.eps);
+        }
 #pragma unroll
         for (int j = 0; j < kRowsMaxJ; ++j) {
             const int i4 = tid + j * kRowsThreads;
             if (i4 < H4) {
-                const float4 w = *reinterpret_cast<const float4*>(a.w_post + 4 * i4);
+                float4 w = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+                if (a.w_post != nullptr) w = *reinterpret_cast<const float4*>(a.w_post + 4 * i4);
                 hv[j].x = (hv[j].x + t[j].x * r * w.x) * a.scalar;
                 hv[j].y = (hv[j].y + t[j].y * r * w.y) * a.scalar;
                 hv[j].z = (hv[j].z + t[j].z * r * w.z) * a.scalar;
@@ -366,7 +371,7 @@ __global__ void pool_fill_kernel(uint4* __restrict__ pool, size_t n16, uint32_t 
     }
 }
 
-// x[b, i] = bf16(act(sum_s gu[s, b, i]) * sum_s gu[s, b, I + i]), act = tanh-GELU or SiLU; grid (ceil(I / 1024), B)
+// x[b, i] = bf16(act(sum_s gu[s, b, i]) * sum_s gu[s, b, I + i]), act = tanh-GELU, SiLU or ReLU; grid (ceil(I / 1024), B)
 __global__ void __launch_bounds__(kRowsThreads)
 geglu_rows_kernel(int B, int I, const float* gu, int splits, uint16_t* x, int act) {
     pdl_wait();

@@ -127,9 +127,11 @@ DEVINL float gelu_mul(float x, float up) {
 DEVINL float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 DEVINL float silu(float z) { return z / (1.0f + expf(-z)); }
 
-enum { ACT_GELU_TANH = 0, ACT_SILU = 1, ACT_SIGMOID = 2, ACT_NONE = 3 };
+enum { ACT_GELU_TANH = 0, ACT_SILU = 1, ACT_SIGMOID = 2, ACT_NONE = 3, ACT_RELU = 4 };
 
 // gate activation times the up projection
-DEVINL float glu_mul(int act, float gate, float up) { return act == ACT_SILU ? silu(gate) * up : gelu_mul(gate, up); }
+DEVINL float glu_mul(int act, float gate, float up) {
+    return act == ACT_SILU ? silu(gate) * up : act == ACT_RELU ? fmaxf(gate, 0.0f) * up : gelu_mul(gate, up);
+}
 
 }  // namespace oxg4

@@ -5,16 +5,20 @@
 // gemma4_cuda/decode.rs:4-21,43-174 and tensor_ops.rs:61-157:
 //   prologue  PRO_NORM : finish the previous block's residual update
 //                        h = (h_in + rmsnorm(previous projection, w_post)) * layer_scalar
-//                        (or h = embedding row * sqrt(H) for the first layer), store h once, then
+//                        (the projection itself is added where w_post is null; h = embedding row * sqrt(H)
+//                        for the first layer), store h once, then
 //                        x = bf16(rmsnorm(h, w_norm))
 //             PRO_PLAIN: x = bf16(in)
 //             PRO_SHIFT: PRO_NORM, then one input per segment of output rows: n + (previous token's n - n) * mu_s,
 //                        n = rmsnorm(h, w_norm) in f32 (token shift of a time-mixing layer; one row)
-//             PRO_GNORM: x = bf16(in / rms(its group) * w * act(gate)), each factor optional (one row)
+//             PRO_GNORM: x = bf16(in / rms(its group) * w * act(gate)), each factor optional, then (optional) further
+//                        columns that are taken as they are (one row)
 //   body      out[n] = sum_k x[k] * W[n,k], f32 accumulate, 16-byte coalesced streaming loads,
 //             warp-shuffle reductions
 //   epilogue  EPI_STORE : out[b, n]
-//             EPI_GATEUP: out[b, i] = act(gate_i . x) * (up_i . x), act = tanh-GELU or SiLU
+//             EPI_GATEUP: out[b, i] = act(gate_i . x) * (up_i . x), act = tanh-GELU, SiLU or ReLU
+//             EPI_STORE_GLU: EPI_STORE for the rows before `glu_from`; the rows behind are alternately gate and up rows
+//                        and each pair gives one value (mixer and feed-forward inputs of a layer in one matrix)
 //             EPI_LOGITS: optional logits store + running arg-max with repetition penalty
 //
 // Work split (EPI_STORE / EPI_GATEUP). Every CTA owns a contiguous block of output rows (for
@@ -31,7 +35,7 @@
 namespace oxg4 {
 
 enum { PRO_PLAIN = 0, PRO_NORM = 1, PRO_SHIFT = 2, PRO_GNORM = 3 };
-enum { EPI_STORE = 0, EPI_GATEUP = 1, EPI_LOGITS = 2 };
+enum { EPI_STORE = 0, EPI_GATEUP = 1, EPI_LOGITS = 2, EPI_STORE_GLU = 3 };
 
 constexpr int kGemvThreads = 512;
 constexpr int kGemvWarps = kGemvThreads / 32;
@@ -61,12 +65,15 @@ struct GemvArgs {
     int gn_n, gn_group;      // values and group size (0: no norm); x is zero from gn_n to K
     const float* gn_w;       // or null
     const float* gn_gate;    // or null
-    int act;                 // PRO_GNORM: gate activation; EPI_GATEUP: activation of the gate projection
+    const float* gn_tail;    // gn_tail_n values for x[gn_tail_at ..], or null
+    int gn_tail_n, gn_tail_at;
+    int act;                 // PRO_GNORM: gate activation; EPI_GATEUP, EPI_STORE_GLU: activation of the gate projection
+    int glu_from;            // EPI_STORE_GLU: first gate row (even)
     // PRO_NORM (K == hidden size)
     const float* h_in;       // [B, K] residual stream before the pending update (unused with embed)
     float* h_out;            // [B, K] residual stream after it (written by block 0)
     const float* raw;        // [B, K] previous projection output still to be normed and added, or null
-    const float* w_post;     // norm weight applied to `raw`
+    const float* w_post;     // norm weight applied to `raw`, or null: `raw` is added as it is
     float scalar;            // layer_scalar of the layer that just ended (1.0 otherwise)
     const float* w_norm;     // norm weight producing x
     const void* embed;       // embedding table [V, K] (same element type as W0), or null
@@ -80,7 +87,7 @@ struct GemvArgs {
     int pf_cap_kb;           // bytes of its own weight block a CTA prefetches into L2 before the dependency wait (KiB)
     unsigned long long* ts;  // optional timeline slots of this launch (4 entries) or null
     // epilogue
-    float* out;              // STORE: [B, N]; GATEUP: [B, N/2]; LOGITS: [B, n_total] or null
+    float* out;              // STORE: [B, N]; GATEUP: [B, N/2]; STORE_GLU: [B, (glu_from + N) / 2]; LOGITS: [B, n_total] or null
     const uint8_t* seen;     // LOGITS: [B, n_total] repetition bitmap or null
     float penalty;
     int row_offset;          // LOGITS: first vocabulary row of this rank's slice
@@ -151,6 +158,7 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int K = a.K;
     constexpr bool SEGS = (PRO == PRO_SHIFT || PRO == PRO_PLAIN) && EPI == EPI_STORE;  // may have several inputs
+    constexpr bool STORES = EPI == EPI_STORE || EPI == EPI_STORE_GLU;
     const int nseg = SEGS ? max(1, a.nseg) : 1;
     XT* xs = reinterpret_cast<XT*>(smem_raw);                                        // [nseg][NB][K]
     float* red = reinterpret_cast<float*>(smem_raw + (size_t)nseg * NB * K * sizeof(XT));   // [NB*32]
@@ -173,7 +181,11 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
         block_range(a.N / 2, gridDim.x, blockIdx.x, row_first, rows_cta);
         row_first *= 2;
         rows_cta *= 2;
-    } else if constexpr (EPI == EPI_STORE) {
+    } else if constexpr (EPI == EPI_STORE_GLU) {       // a gate row and its up row stay together
+        block_range(a.N / 2, gridDim.x, blockIdx.x, row_first, rows_cta);
+        row_first *= 2;
+        rows_cta *= 2;
+    } else if constexpr (STORES) {
         block_range(a.N, gridDim.x, blockIdx.x, row_first, rows_cta);
     }
     const int chunks_cta = rows_cta * a.cpr;
@@ -270,7 +282,13 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
                 for (int i = lane; i < a.gn_group; i += 32) put(g * a.gn_group + i, src[i] * s);
             }
         }
-        for (int i = a.gn_n + tid; i < K; i += kSimtThreads) T::store_x(xs + i, 0.0f);
+        if (a.gn_tail != nullptr) {
+            for (int i = a.gn_n + tid; i < a.gn_tail_at; i += kSimtThreads) T::store_x(xs + i, 0.0f);
+            for (int i = a.gn_tail_at + tid; i < K; i += kSimtThreads)
+                T::store_x(xs + i, i < a.gn_tail_at + a.gn_tail_n ? a.gn_tail[i - a.gn_tail_at] : 0.0f);
+        } else {
+            for (int i = a.gn_n + tid; i < K; i += kSimtThreads) T::store_x(xs + i, 0.0f);
+        }
     } else {
         const bool writer = (blockIdx.x == 0);
         const float norm_n = (float)(a.norm_n ? a.norm_n : K);
@@ -303,10 +321,15 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
                     hv[j] = (i < K) ? a.h_in[(size_t)(b0 + b) * K + i] : 0.0f;
                     ss[0] += t[j] * t[j];
                 }
-                block_sum<1>(ss, red);
-                const float r = 1.0f / sqrtf(ss[0] / norm_n + a.eps);
+                if (a.w_post != nullptr) {
+                    block_sum<1>(ss, red);
+                    const float r = 1.0f / sqrtf(ss[0] / norm_n + a.eps);
 #pragma unroll
-                for (int j = 0; j < kSimtMaxJ; ++j) hv[j] = (hv[j] + t[j] * r * wpost[j]) * a.scalar;
+                    for (int j = 0; j < kSimtMaxJ; ++j) hv[j] = (hv[j] + t[j] * r * wpost[j]) * a.scalar;
+                } else {
+#pragma unroll
+                    for (int j = 0; j < kSimtMaxJ; ++j) hv[j] = (hv[j] + t[j]) * a.scalar;
+                }
             }
             ss[0] = 0.0f;
 #pragma unroll
@@ -426,6 +449,14 @@ __global__ void __launch_bounds__(kSimtThreads, 1) gemv_kernel(const GemvArgs a)
             for (int idx = tid; idx < rows_cta * nb; idx += kSimtThreads) {
                 const int rl = idx % rows_cta, b = idx / rows_cta;
                 a.out[(size_t)(b0 + b) * a.N + row_first + rl] = row_total(rl, b);
+            }
+        } else if constexpr (EPI == EPI_STORE_GLU) {
+            const int ld = (a.glu_from + a.N) / 2;
+            for (int idx = tid; idx < rows_cta * nb; idx += kSimtThreads) {
+                const int rl = idx % rows_cta, b = idx / rows_cta, row = row_first + rl;
+                float* o = a.out + (size_t)(b0 + b) * ld;
+                if (row < a.glu_from) o[row] = row_total(rl, b);
+                else if (!(row & 1)) o[a.glu_from + (row - a.glu_from) / 2] = glu_mul(a.act, row_total(rl, b), row_total(rl + 1, b));
             }
         } else {
             const int pairs = rows_cta / 2;

@@ -32,8 +32,8 @@ struct LatentMmaArgs {
     RunRows rows;
     int runs;
     int step_tiles;                      // > 0: a decode step (run r is row r, one token): row tiles per run
-    LatentCache cache;
-    LatentPart part;
+    RowCache cache;
+    AttnPart part;
 };
 
 DEVINL void cp_async16(uint32_t dst, const void* src, bool valid) {
@@ -83,25 +83,8 @@ __global__ void __launch_bounds__(kLmThreads * GR, 1) latent_mma_kernel(const La
     // the longest rows are at the end of a run: they start first
     const int t = gridDim.x - 1 - blockIdx.x;
     if (a.step_tiles == 0 && threadIdx.x < 32) {
-        int base = 0, run = -1, first = 0;
-        for (int r0 = 0; r0 < a.runs && run < 0; r0 += 32) {
-            const int r = r0 + lane;
-            const int nt = r < a.runs ? (a.rows.n[r] * a.heads + ROWS - 1) / ROWS : 0;
-            int inc = nt;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const int v = __shfl_up_sync(0xffffffffu, inc, o);
-                if (lane >= o) inc += v;
-            }
-            const int lo = base + inc - nt;
-            const unsigned hit = __ballot_sync(0xffffffffu, t >= lo && t < lo + nt);
-            if (hit) {
-                const int src = __ffs(hit) - 1;
-                run = r0 + src;
-                first = (t - __shfl_sync(0xffffffffu, lo, src)) * ROWS;
-            }
-            base += __shfl_sync(0xffffffffu, inc, 31);
-        }
+        int run, first;
+        find_row_tile(a.rows, a.runs, a.heads, ROWS, t, run, first);
         if (lane == 0) { s_run = run; s_first = first; }
     }
     int run, first, row0, n_flat;

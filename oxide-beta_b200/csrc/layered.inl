@@ -1,5 +1,7 @@
 // Models whose layers are listed one by one (oxg4_model_create_layered): every layer names its mixer, its sizes and an
-// optional feed-forward, x += norm1b(mixer(norm1(x))), x += norm2b(ff(norm2(x))). This file turns the list into plans,
+// optional feed-forward. Two blocks: x += norm1b(mixer(norm1(x))), x += norm2b(ff(norm2(x))), and the parallel one,
+// h = norm1(x), x += mixer(h) + ff(h), whose input matrices (mixer, gate and up rows) are one matrix and whose output
+// matrices are one matrix over [mixer output | feed-forward activations]. This file turns the list into plans,
 // adds the caches and states of the mixers to the cache table and sequences a pass over the layers; positions, pages,
 // chunks of prompts, graphs, sampling and generation are those of oxg4.cu, which includes it.
 //
@@ -25,6 +27,10 @@ extern "C" int32_t oxg4_model_create_layered(const oxg4_layered_config* lc, int3
     if (lc->width > std::min(max_width, kGemvMaxJ * kGemvThreads))
         return fail(OXG4_UNSUPPORTED, "width above %d is not supported", std::min(max_width, kGemvMaxJ * kGemvThreads));
     const int L = lc->num_layers;
+    if (lc->block != OXG4_BLOCK_SANDWICH && lc->block != OXG4_BLOCK_PARALLEL) return fail(OXG4_INVALID_ARGUMENT, "unknown block %d", lc->block);
+    if (lc->act != OXG4_ACT_GELU_TANH && lc->act != OXG4_ACT_SILU && lc->act != OXG4_ACT_RELU)
+        return fail(OXG4_INVALID_ARGUMENT, "unknown activation %d", lc->act);
+    const bool parallel = lc->block == OXG4_BLOCK_PARALLEL;
     for (int l = 0; l < L; ++l) {
         const oxg4_layer_spec& s = lc->layers[l];
         if (s.heads <= 0 || s.dim <= 0 || s.vdim <= 0 || s.ff < 0) return fail(OXG4_INVALID_SHAPE, "layer %d: invalid sizes", l);
@@ -45,9 +51,24 @@ extern "C" int32_t oxg4_model_create_layered(const oxg4_layered_config* lc, int3
                 if (s.vdim != s.dim) return fail(OXG4_INVALID_SHAPE, "layer %d: invalid time-mixing sizes", l);
                 if (s.dim > 512) return fail(OXG4_UNSUPPORTED, "layer %d: key size above 512 is not supported", l);
                 break;
+            case OXG4_MIXER_RETENTION:
+                if (!s.decay) return fail(OXG4_INVALID_ARGUMENT, "layer %d: decay is missing", l);
+                if (s.rot_dims < 0 || s.rot_dims > s.dim || s.rot_dims % 2) return fail(OXG4_INVALID_SHAPE, "layer %d: invalid rotation", l);
+                if (s.dim > 512) return fail(OXG4_UNSUPPORTED, "layer %d: key size above 512 is not supported", l);
+                break;
+            case OXG4_MIXER_ATTENTION:
+                if (s.kv_heads <= 0 || s.heads % s.kv_heads) return fail(OXG4_INVALID_SHAPE, "layer %d: query heads must be a multiple of kv heads", l);
+                if (s.q_temp_every <= 0) return fail(OXG4_INVALID_ARGUMENT, "layer %d: q_temp_every must be positive", l);
+                if (s.vdim > 512) return fail(OXG4_UNSUPPORTED, "layer %d: value size above 512 is not supported", l);
+                if (s.dim > 1024) return fail(OXG4_UNSUPPORTED, "layer %d: key size above 1024 is not supported", l);
+                if ((size_t)s.heads * s.dim * 4 > 200 * 1024)
+                    return fail(OXG4_UNSUPPORTED, "layer %d: more than 51200 query values per token are not supported", l);
+                break;
             default:
                 return fail(OXG4_INVALID_ARGUMENT, "layer %d: unknown mixer %d", l, s.mixer);
         }
+        if (parallel != (s.mixer == OXG4_MIXER_RETENTION || s.mixer == OXG4_MIXER_ATTENTION))
+            return fail(OXG4_UNSUPPORTED, "layer %d: mixer %d is not available in block %d", l, s.mixer, lc->block);
     }
     // the rest of the model is created as a one-kind attention model of the same depth and vocabulary would be
     std::vector<int32_t> sliding(L, 0), rotary(L, 64);
@@ -70,11 +91,14 @@ extern "C" int32_t oxg4_model_create_layered(const oxg4_layered_config* lc, int3
     TRY(oxg4_model_create(&c, device, out));
     oxg4_model* m = *out;
     m->layered = true;
+    m->parallel = parallel;
+    m->ff_act = lc->act;
+    m->norm_offset = lc->norm_weight_offset ? 1.0f : 0.0f;
     m->Hn = lc->width;
     m->specs.assign(lc->layers, lc->layers + L);
     m->spec_decay.resize(L);
     for (int l = 0; l < L; ++l) {
-        if (m->specs[l].mixer == OXG4_MIXER_LIGHTNING)
+        if (m->specs[l].mixer == OXG4_MIXER_LIGHTNING || m->specs[l].mixer == OXG4_MIXER_RETENTION)
             m->spec_decay[l].assign(m->specs[l].decay, m->specs[l].decay + m->specs[l].heads);
         m->specs[l].decay = m->spec_decay[l].data();
     }
@@ -90,8 +114,8 @@ static int32_t owned_alloc(oxg4_model* m, void** d, size_t bytes) {
     return OXG4_OK;
 }
 
-// f32 copy of a small tensor (matrices of a BF16 model are widened), padded with zeros to n_pad values
-static int32_t small_f32(oxg4_model* m, const std::string& name, int64_t n, int64_t n_pad, const float** out) {
+// f32 copy of a small tensor (matrices of a BF16 model are widened) plus `offset`, padded with zeros to n_pad values
+static int32_t small_f32(oxg4_model* m, const std::string& name, int64_t n, int64_t n_pad, const float** out, float offset = 0.0f) {
     const Tensor* t;
     TRY(need(m, name, {n}, &t));
     std::vector<float> f((size_t)n_pad, 0.0f);
@@ -102,6 +126,7 @@ static int32_t small_f32(oxg4_model* m, const std::string& name, int64_t n, int6
         CK(cudaMemcpy(h.data(), t->d, 2 * n, cudaMemcpyDeviceToHost));
         for (int64_t i = 0; i < n; ++i) f[i] = host_bf16_to_f32(h[i]);
     }
+    for (int64_t i = 0; i < n; ++i) f[i] += offset;
     void* d;
     TRY(owned_alloc(m, &d, sizeof(float) * n_pad));
     CK(cudaMemcpy(d, f.data(), sizeof(float) * n_pad, cudaMemcpyHostToDevice));
@@ -113,12 +138,15 @@ struct StackPart {
     std::string name;
     int64_t rows;
     int64_t at;              // first row in the stacked matrix
+    int64_t step = 1;        // distance of its rows there
+    int64_t col = 0;         // first column
+    int64_t cols = 0;        // columns; 0: the stack's
 };
-// [N, K] matrix with the given tensors (each [rows, cols]) at their rows, everything else zero. A single tensor that needs
+// [N, K] matrix with the given tensors (each [rows, cols]) at their places, everything else zero. A single tensor that needs
 // no padding is used as it is; the parts of a stack are released.
 static int32_t stack_rows(oxg4_model* m, const std::vector<StackPart>& parts, int64_t cols, int64_t N, int64_t K, const void** out) {
     const Tensor* t;
-    for (auto& p : parts) TRY(need(m, p.name, {p.rows, cols}, &t));
+    for (auto& p : parts) TRY(need(m, p.name, {p.rows, p.cols ? p.cols : cols}, &t));
     if (parts.size() == 1 && parts[0].rows == N && cols == K) {
         *out = t->d;
         return OXG4_OK;
@@ -126,8 +154,9 @@ static int32_t stack_rows(oxg4_model* m, const std::vector<StackPart>& parts, in
     void* d;
     TRY(owned_alloc(m, &d, (size_t)N * K * m->es));
     for (auto& p : parts) {
-        TRY(need(m, p.name, {p.rows, cols}, &t));
-        CK(cudaMemcpy2D((char*)d + (size_t)p.at * K * m->es, (size_t)K * m->es, t->d, (size_t)cols * m->es, (size_t)cols * m->es,
+        const int64_t pc = p.cols ? p.cols : cols;
+        TRY(need(m, p.name, {p.rows, pc}, &t));
+        CK(cudaMemcpy2D((char*)d + ((size_t)p.at * K + p.col) * m->es, (size_t)p.step * K * m->es, t->d, (size_t)pc * m->es, (size_t)pc * m->es,
                         (size_t)p.rows, cudaMemcpyDeviceToDevice));
     }
     CK(cudaDeviceSynchronize());
@@ -160,12 +189,67 @@ __global__ void transpose_heads_kernel(const uint16_t* w, uint16_t* t, int heads
     }
 }
 
+// layer of the parallel block: one input matrix (mixer rows, then alternately gate and up rows), one output matrix over
+// [mixer output | feed-forward]
+static int32_t finalize_parallel(oxg4_model* m, const std::string& pre, const oxg4_layer_spec& s, MixPlan& x) {
+    const std::string mx = pre + "mix.";
+    const int H = m->Hn, Hp = m->H, HD = x.heads * x.dim;
+    const bool attention = x.kind == MIX_ATTENTION;
+    const int kn = attention ? x.kv_heads * x.dim : HD, vn = attention ? x.kv_heads * x.vdim : x.ow;
+    x.c_k = pad_to(HD, 8);
+    x.c_v = x.c_k + pad_to(kn, 8);
+    x.c_g = x.c_v + pad_to(vn, 8);
+    x.c_ff = x.c_g + (attention ? 0 : pad_to(x.ow, 8));
+    std::vector<StackPart> parts = {{mx + "q", HD, 0}, {mx + "k", kn, x.c_k}, {mx + "v", vn, x.c_v}};
+    if (!attention) parts.push_back({mx + "g", x.ow, x.c_g});
+    if (x.ff > 0) {
+        parts.push_back({pre + "mlp.gate", x.ff, x.c_ff, 2});
+        parts.push_back({pre + "mlp.up", x.ff, x.c_ff + 1, 2});
+    }
+    const void* w = nullptr;
+    const int N = x.c_ff + 2 * x.ffp;
+    TRY(stack_rows(m, parts, H, N, Hp, &w));
+    x.in = make_proj(m, w, N, Hp);
+    if (x.ff > 0) {
+        x.in.glu_from = x.c_ff;
+        x.in.gp = make_plan(N, Hp, m->es, m->num_sms, 2);
+    }
+    parts = {{mx + "o", H, 0, 1, 0, x.ow}};
+    if (x.ff > 0) parts.push_back({pre + "mlp.down", H, 0, 1, x.owp, x.ff});
+    TRY(stack_rows(m, parts, x.ow, Hp, x.owp + x.ffp, &w));
+    x.o = make_proj(m, w, Hp, x.owp + x.ffp);
+    void* d;
+    if (attention) {
+        TRY(small_f32(m, mx + "q.norm", HD, HD, &x.q_norm));
+        TRY(small_f32(m, mx + "k.norm", kn, kn, &x.k_norm));
+        TRY(small_f32(m, mx + "q.b", HD, HD, &x.q_b));
+        TRY(small_f32(m, mx + "k.b", kn, kn, &x.k_b));
+        TRY(small_f32(m, mx + "v.b", vn, vn, &x.v_b));
+        TRY(small_f32(m, mx + "sink", x.heads, x.heads, &x.sink));
+        return OXG4_OK;
+    }
+    TRY(owned_alloc(m, &d, sizeof(float) * x.heads));
+    CK(cudaMemcpy(d, s.decay, sizeof(float) * x.heads, cudaMemcpyHostToDevice));
+    x.decay = (const float*)d;
+    std::vector<float2> freq(std::max(1, x.rot_dims / 2));
+    for (int i = 0; i < x.rot_dims / 2; ++i) {
+        const double f = std::pow((double)s.rot_base, -2.0 * i / (double)x.rot_dims);
+        freq[i].x = (float)f;
+        freq[i].y = (float)(f - (double)freq[i].x);
+    }
+    TRY(owned_alloc(m, &d, sizeof(float2) * freq.size()));
+    CK(cudaMemcpy(d, freq.data(), sizeof(float2) * freq.size(), cudaMemcpyHostToDevice));
+    x.freq2 = (const float2*)d;
+    return OXG4_OK;
+}
+
 static int32_t finalize_mixer(oxg4_model* m, int l, const oxg4_layer_spec& s, MixPlan& x) {
     const std::string pre = "l" + std::to_string(l) + ".", mx = pre + "mix.";
     const int H = m->Hn, Hp = m->H;
     const Tensor* t;
-    TRY(small_f32(m, pre + "norm1", H, Hp, &x.norm1));
-    TRY(small_f32(m, pre + "norm1b", H, Hp, &x.norm1b));
+    TRY(small_f32(m, pre + "norm1", H, Hp, &x.norm1, m->norm_offset));
+    if (m->parallel) return finalize_parallel(m, pre, s, x);
+    TRY(small_f32(m, pre + "norm1b", H, Hp, &x.norm1b, m->norm_offset));
     const int HD = x.heads * x.dim;
     const void* w = nullptr;
     if (x.kind == MIX_WKV) {
@@ -247,8 +331,8 @@ static int32_t finalize_mixer(oxg4_model* m, int l, const oxg4_layer_spec& s, Mi
     TRY(stack_rows(m, {{mx + "o", H, 0}}, x.ow, Hp, x.owp, &w));
     x.o = make_proj(m, w, Hp, x.owp);
     if (x.ff > 0) {
-        TRY(small_f32(m, pre + "norm2", H, Hp, &x.norm2));
-        TRY(small_f32(m, pre + "norm2b", H, Hp, &x.norm2b));
+        TRY(small_f32(m, pre + "norm2", H, Hp, &x.norm2, m->norm_offset));
+        TRY(small_f32(m, pre + "norm2b", H, Hp, &x.norm2b, m->norm_offset));
         TRY(stack_rows(m, {{pre + "mlp.gate", x.ff, 0}}, H, x.ffp, Hp, &w));
         x.gateup = make_proj(m, w, x.ffp, Hp);
         TRY(stack_rows(m, {{pre + "mlp.up", x.ff, 0}}, H, x.ffp, Hp, &x.gateup.w1));
@@ -263,7 +347,7 @@ static int32_t finalize_layered(oxg4_model* m) {
     const int L = m->cfg.num_hidden_layers, H = m->Hn, Hp = m->H;
     TRY(stack_rows(m, {{"embed", m->V, 0}}, H, m->V, Hp, &m->embed));
     TRY(stack_rows(m, {{"head", m->V, 0}}, H, m->V, Hp, &m->head));
-    TRY(small_f32(m, "final.norm", H, Hp, &m->final_norm));
+    TRY(small_f32(m, "final.norm", H, Hp, &m->final_norm, m->norm_offset));
     m->p_lm = make_plan(m->V, Hp, m->es, m->num_sms, 1);
     m->p_lm_simt_grid = std::min(m->num_sms, std::max(1, (m->V + 2 * kSimtWarps - 1) / (2 * kSimtWarps)));
     m->layers.resize(L);
@@ -282,6 +366,13 @@ static int32_t finalize_layered(oxg4_model* m) {
         x.rot = s.rot_dim;
         x.rot_dims = s.rot_dims;
         x.ld = pad_to(s.kv_rank + s.rot_dim, 16);
+        if (x.kind == MIX_ATTENTION) {
+            x.kv_heads = s.kv_heads;
+            x.kd = pad_to(s.dim, 16);
+            x.ld = x.kd + pad_to(s.vdim, 16);
+            x.temp_coef = s.q_temp_coef;
+            x.temp_every = s.q_temp_every;
+        }
         x.scale = s.scale;
         x.ff = s.ff;
         x.ffp = pad_to(s.ff, 8);
@@ -295,7 +386,7 @@ static int32_t finalize_layered(oxg4_model* m) {
         if (j == l) continue;
         const oxg4_layer_spec &a = m->specs[l], &b = m->specs[j];
         if (a.mixer != b.mixer || a.heads != b.heads || a.dim != b.dim || a.vdim != b.vdim || a.q_rank != b.q_rank ||
-            a.kv_rank != b.kv_rank || a.rot_dim != b.rot_dim || a.ff != b.ff)
+            a.kv_rank != b.kv_rank || a.rot_dim != b.rot_dim || a.ff != b.ff || a.kv_heads != b.kv_heads)
             return fail(OXG4_INVALID_SHAPE, "layer %d uses the tensors of layer %d but differs in size", l, j);
         m->layers[l].mix = m->layers[j].mix;
     }
@@ -311,6 +402,7 @@ static int layered_splits(const oxg4_model* m, const Proj& p, int R, bool chunk)
 }
 
 static int32_t latent_mma_setup(const MixPlan& x);
+static int32_t head_attn_setup(const MixPlan& x);
 constexpr int kLatentChunkSplits = 4;     // most splits of the visible positions in a prompt chunk
 
 static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
@@ -334,9 +426,9 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
         const MixPlan& x = m->layers[l].mix;
         in_n = std::max(in_n, floats(x.in));
         o_n = std::max(o_n, floats(x.o));
-        xo = std::max(xo, (size_t)x.owp);
+        xo = std::max(xo, (size_t)x.o.K);
         act = std::max(act, (size_t)x.owp);
-        if (x.ff > 0) {
+        if (x.ff > 0 && !m->parallel) {
             gu_n = std::max(gu_n, floats(x.gateup));
             down_n = std::max(down_n, floats(x.down));
             xi = std::max(xi, (size_t)x.ffp);
@@ -361,6 +453,18 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
                 rot = std::max(rot, (size_t)x.heads * x.rot);
                 TRY(latent_mma_setup(x));
             }
+        } else if (x.kind == MIX_ATTENTION) {
+            uint8_t* pool;
+            const size_t bytes = (size_t)pages_full * x.kv_heads * c->PT * x.ld * kes;
+            TRY(dalloc(c, &pool, bytes));
+            c->kpool[l] = pool;
+            c->pool_bytes[l] = bytes;
+            c->kv_bytes += (int64_t)bytes;
+            xu = std::max(xu, (size_t)x.heads * x.kd);
+            latq = std::max(latq, (size_t)x.heads * x.dim);
+            rh = std::max(rh, (size_t)x.heads);
+            rh_rank = std::max(rh_rank, (size_t)x.ow);
+            TRY(head_attn_setup(x));
         } else {
             const size_t n = (size_t)B * x.heads * x.dim * x.vdim;
             TRY(dalloc(c, &c->state[l], n));
@@ -428,13 +532,14 @@ static int32_t group_norm_setup() {
     return allow_big_smem(group_norm_rows_kernel<float, 4>);
 }
 
-typedef void (*LatentAttnFn)(const LatentArgs, const float*, LatentPart);
-template <typename KT>
-static LatentAttnFn pick_latent_attn(int rank) {
-    if (rank <= 128) return latent_attn_kernel<KT, 4>;
-    if (rank <= 256) return latent_attn_kernel<KT, 8>;
-    return latent_attn_kernel<KT, 16>;
+typedef void (*RowAttnFn)(const RowAttnArgs);
+template <typename KT, bool LATENT>
+static RowAttnFn pick_row_attn(int vw) {
+    if (vw <= 128) return row_attn_kernel<KT, 4, LATENT>;
+    if (vw <= 256) return row_attn_kernel<KT, 8, LATENT>;
+    return row_attn_kernel<KT, 16, LATENT>;
 }
+static size_t row_attn_smem(int dk, int vw) { return sizeof(float) * ((size_t)dk + 8 * vw + 16); }
 
 typedef void (*LatentMmaFn)(const LatentMmaArgs);
 // the tensor-core kernel for `rows` (token, head) rows per run and cache rows of `ld` elements, null when it does not fit
@@ -470,6 +575,30 @@ static int32_t latent_mma_setup(const MixPlan& x) {
         if (fn) TRY(allow_big_smem(fn));
     }
     return OXG4_OK;
+}
+
+// Attention over [key | value] rows: the tensor-core kernel for `rows` (token, head) rows per run and kv head, null when the
+// heads are too wide for it
+typedef void (*HeadMmaFn)(const HeadMmaArgs);
+static HeadMmaFn pick_head_mma(const MixPlan& x, int rows, int* tile_rows, size_t* smem) {
+    const int vd = x.ld - x.kd, cols = std::max(x.kd, vd) <= 64 ? 64 : std::max(x.kd, vd) <= 128 ? 128 : 256, wr = rows <= 16 ? 1 : 4;
+    if (std::max(x.kd, vd) > 256) return nullptr;
+    *tile_rows = 16 * wr;
+    *smem = head_mma_smem(cols, wr, x.ld, x.kd, vd);
+    if (wr == 1) return cols == 64 ? head_mma_kernel<64, 1> : cols == 128 ? head_mma_kernel<128, 1> : head_mma_kernel<256, 1>;
+    return cols == 64 ? head_mma_kernel<64, 4> : cols == 128 ? head_mma_kernel<128, 4> : head_mma_kernel<256, 4>;
+}
+
+static int32_t head_attn_setup(const MixPlan& x) {
+    for (int rows : {16, 64}) {
+        int tr;
+        size_t smem;
+        HeadMmaFn fn = pick_head_mma(x, rows, &tr, &smem);
+        if (fn) TRY(allow_big_smem(fn));
+    }
+    TRY((allow_big_smem(head_prep_kernel<uint16_t, uint16_t>)));
+    TRY((allow_big_smem(head_prep_kernel<float, uint16_t>)));
+    return allow_big_smem((head_prep_kernel<float, float>));
 }
 
 // Splits of `tiles` cache tiles when `units` row tiles share the GPU: the cheapest number of rounds times tiles per CTA, with
@@ -527,6 +656,16 @@ struct LayeredPass {
             a.w_post = pd.w_post;
         }
     }
+    // what an output projection of the parallel block reads behind the mixer's columns; in: fused input projection
+    OutTail ff_tail(const MixPlan& x, const SplitIn& in) const {
+        OutTail t{};
+        t.in = in;
+        t.col = x.c_ff;
+        t.n = m->parallel ? x.ffp : 0;
+        t.at = x.owp;
+        t.act = tc ? m->ff_act : ACT_NONE;
+        return t;
+    }
     // row kernels: close the pending update, norm; x and / or x_f32 may be null
     void close_rows(const float* w_norm, void* x, float* x_f32) {
         RowsNormArgs n{};
@@ -560,22 +699,29 @@ struct LayeredPass {
         a.W0 = p.w;
         a.in = (const float*)x;
         a.out = out;
+        if (p.glu_from >= 0) {
+            a.glu_from = p.glu_from;
+            a.act = m->ff_act;
+            launch_gemv(ln, kind, c, R, a, p.gp, PRO_PLAIN, EPI_STORE_GLU);
+            return one(out, (p.glu_from + p.N) / 2);
+        }
         if (p.nseg > 1) { a.nseg = p.nseg; a.seg_rows = p.seg_rows; }
         launch_gemv(ln, kind, c, R, a, p.gp, PRO_PLAIN, EPI_STORE);
         return SplitIn{out, 1, 0, n};
     }
     SplitIn one(float* out, int n) const { return SplitIn{out, 1, 0, n}; }
 
-    void group_norm(const GroupNormArgs& g, void* x, int ld_x) {
+    void group_norm(const GroupNormArgs& g, const OutTail& tail, void* x, int ld_x) {
         const size_t smem = sizeof(float) * g.n;
+        const dim3 grid(R, 1 + tail.slices());
         if (ln.status == OXG4_OK && smem > 48 * 1024) ln.status = group_norm_setup();
-        const bool vec = (g.n | g.hs | g.hs_ld | g.o.ld | g.gate.ld | g.c_gate | ld_x) % 4 == 0 && (g.o.stride | g.gate.stride) % 4 == 0;
+        const bool vec = (g.n | g.n_pad | g.hs | g.hs_ld | g.o.ld | g.gate.ld | g.c_gate | ld_x) % 4 == 0 && (g.o.stride | g.gate.stride) % 4 == 0;
         if (m->es == 2) {
-            if (vec) ln.go("outnorm", group_norm_rows_kernel<uint16_t, 4>, dim3(R), dim3(256), smem, g, (uint16_t*)x, ld_x);
-            else ln.go("outnorm", group_norm_rows_kernel<uint16_t, 1>, dim3(R), dim3(256), smem, g, (uint16_t*)x, ld_x);
+            if (vec) ln.go("outnorm", group_norm_rows_kernel<uint16_t, 4>, grid, dim3(256), smem, g, tail, (uint16_t*)x, ld_x);
+            else ln.go("outnorm", group_norm_rows_kernel<uint16_t, 1>, grid, dim3(256), smem, g, tail, (uint16_t*)x, ld_x);
         } else {
-            if (vec) ln.go("outnorm", group_norm_rows_kernel<float, 4>, dim3(R), dim3(256), smem, g, (float*)x, ld_x);
-            else ln.go("outnorm", group_norm_rows_kernel<float, 1>, dim3(R), dim3(256), smem, g, (float*)x, ld_x);
+            if (vec) ln.go("outnorm", group_norm_rows_kernel<float, 4>, grid, dim3(256), smem, g, tail, (float*)x, ld_x);
+            else ln.go("outnorm", group_norm_rows_kernel<float, 1>, grid, dim3(256), smem, g, tail, (float*)x, ld_x);
         }
     }
 
@@ -590,6 +736,11 @@ struct LayeredPass {
             a.gn_w = w;
             a.gn_gate = act == ACT_NONE ? nullptr : gate.p + x.c_g;
             a.act = act;
+            if (m->parallel && x.ff > 0) {
+                a.gn_tail = gate.p + x.c_ff;
+                a.gn_tail_n = x.ffp;
+                a.gn_tail_at = x.owp;
+            }
             a.out = c->o_part;
             launch_gemv(ln, "o", c, R, a, x.o.gp, PRO_GNORM, EPI_STORE);
             pend(one(c->o_part, H), x.norm1b);
@@ -600,13 +751,14 @@ struct LayeredPass {
         g.hs = x.vdim;
         g.hs_ld = hs_ld;
         g.n = x.ow;
+        g.n_pad = x.owp;
         g.group = group;
         g.w = w;
         g.gate = gate;
         g.c_gate = x.c_g;
         g.act = act;
         g.eps = eps;
-        group_norm(g, c->mix_y, x.owp);
+        group_norm(g, ff_tail(x, gate), c->mix_y, x.o.K);
         pend(project("o", x.o, c->mix_y, c->o_part), x.norm1b);
     }
 
@@ -627,9 +779,13 @@ struct LayeredPass {
                 a.pos = rs.pos;
                 a.x_f32 = c->xf;
             }
-            launch_gemv(ln, "qkv", c, R, a, x.in.gp, shift ? PRO_SHIFT : PRO_NORM, EPI_STORE);
+            if (x.in.glu_from >= 0) {
+                a.glu_from = x.in.glu_from;
+                a.act = m->ff_act;
+            }
+            launch_gemv(ln, "qkv", c, R, a, x.in.gp, shift ? PRO_SHIFT : PRO_NORM, x.in.glu_from >= 0 ? EPI_STORE_GLU : EPI_STORE);
             advance();
-            in = one(c->in_buf, x.in.N);
+            in = one(c->in_buf, x.in.glu_from >= 0 ? (x.in.glu_from + x.in.N) / 2 : x.in.N);
         } else {
             close_rows(x.norm1, shift ? nullptr : c->mix_x, shift ? c->xf : nullptr);
             if (shift) {
@@ -657,7 +813,7 @@ struct LayeredPass {
         a.rows = runs();
         a.out = c->attn_out;
         a.ld_out = x.owp;
-        const bool wkv = x.kind == MIX_WKV;
+        const bool wkv = x.kind == MIX_WKV, ret = x.kind == MIX_RETENTION;
         if (wkv) {
             a.u = x.u;
             a.c_low = x.c_low; a.rank = x.low_rank; a.w2 = x.w2; a.w0 = x.w0;
@@ -674,18 +830,23 @@ struct LayeredPass {
             }
         } else {
             a.decay = x.decay;
+            a.freq = x.freq2;
+            a.rot_dims = x.rot_dims;
+            a.k_scale = 1.0f / sqrtf((float)x.dim);
         }
         int ks = 1, kpt = 1;
         RecurFn fn;
         const bool step = !rs.chunk;
         if (wkv) fn = m->es == 2 ? pick_recur<REC_WKV, uint16_t>(x.dim, step, &ks, &kpt) : pick_recur<REC_WKV, float>(x.dim, step, &ks, &kpt);
+        else if (ret) fn = pick_recur<REC_RETENTION, float>(x.dim, step, &ks, &kpt);
         else fn = pick_recur<REC_LIGHTNING, float>(x.dim, step, &ks, &kpt);
         const int vs = kRecThreads / ks * kRecCols, dp = ks * kpt, tile = step ? 1 : rec_tile(dp);
         const size_t smem = sizeof(float) * ((step ? 1 : 2) * ((size_t)tile * dp * (wkv ? 3 : 2) + tile * vs + pad_to(tile, 4)) +
                                              (wkv ? dp + x.low_rank : 0));
         if (ln.status == OXG4_OK && smem > 48 * 1024) ln.status = allow_big_smem(fn);
         ln.go("recur", fn, dim3(x.heads, (x.vdim + vs - 1) / vs, (unsigned)rs.run_len.size()), dim3(kRecThreads), smem, a);
-        output(x, one(c->attn_out, x.owp), x.vdim, wkv ? x.dim : x.ow, x.out_norm, in, wkv ? ACT_SILU : ACT_SIGMOID);
+        if (ret) output(x, one(c->attn_out, x.owp), x.vdim, x.vdim, nullptr, in, ACT_SILU);
+        else output(x, one(c->attn_out, x.owp), x.vdim, wkv ? x.dim : x.ow, x.out_norm, in, wkv ? ACT_SILU : ACT_SIGMOID);
     }
 
     LatentArgs latent_args(const MixPlan& x, int l, const SplitIn& in) const {
@@ -698,7 +859,7 @@ struct LayeredPass {
         a.eps = eps;
         a.scale = x.scale;
         a.rows = runs();
-        a.cache = LatentCache{c->kpool[l], c->pt_full, c->pps_full, c->PT, x.ld};
+        a.cache = RowCache{c->kpool[l], c->pt_full, c->pps_full, c->PT, x.ld, 1};
         return a;
     }
 
@@ -719,7 +880,7 @@ struct LayeredPass {
             ln.go("latent", latent_prep_kernel<WT, KT>, dim3(R), dim3(256), 0, a, (WT*)c->x_q, x.q_rankp);
             q = project("uq", x.uq, c->x_q, c->q_buf);
         }
-        LatentPart part{c->lat_o, c->lat_ml, rs.chunk ? 1 : c->lat_splits, (size_t)R * x.heads};
+        AttnPart part{c->lat_o, c->lat_ml, rs.chunk ? 1 : c->lat_splits, (size_t)R * x.heads};
         int tile_rows = 0, groups = 1;
         size_t mma_smem = 0;
         int longest = 1;
@@ -759,13 +920,73 @@ struct LayeredPass {
             ma.q_rot = c->lat_q + x.rank; ma.rot_row = ma.abs_row; ma.rot_head = ma.abs_head;
             ln.go("attn", mma, dim3(mma_tiles, part.splits / groups), dim3(kLmThreads * groups), mma_smem, ma);
         } else {
-            LatentAttnFn fn = pick_latent_attn<KT>(x.rank);
-            ln.go("attn", fn, dim3(x.heads, R, part.splits), dim3(256), sizeof(float) * (x.rank + x.rot + 8 * x.rank + 16), a, (const float*)c->lat_q, part);
+            const RowAttnArgs ra{c->lat_q, x.heads, x.heads, x.rank + x.rot, 0, x.rank, x.scale, a.rows, a.cache, part};
+            ln.go("attn", pick_row_attn<KT, true>(x.rank), dim3(x.heads, R, part.splits), dim3(256), row_attn_smem(ra.dk, ra.vw), ra);
         }
         ln.go("latout", latent_out_kernel<WT>, dim3(x.heads, R, (x.vdim + 31) / 32), dim3(256), sizeof(float) * (pad_to(x.rank, 4) + part.splits), x.heads,
               x.rank, x.vdim, part, (const WT*)x.w_uv, x.rank, in, x.c_g, rs.tok, c->attn_out, x.owp);
         // the gate has been applied by the kernel that leaves latent space
         output(x, one(c->attn_out, x.owp), x.vdim, 0, nullptr, in, ACT_NONE);
+    }
+
+    // grouped-query attention with whole-projection norms and a sink
+    template <typename WT, typename KT>
+    void attention(const MixPlan& x, int l, const SplitIn& in) {
+        HeadAttnArgs a{};
+        a.in = in;
+        a.c_q = x.c_q; a.c_k = x.c_k; a.c_v = x.c_v;
+        a.heads = x.heads; a.kv_heads = x.kv_heads; a.dim = x.dim; a.vdim = x.vdim; a.kd = x.kd;
+        a.q_b = x.q_b; a.k_b = x.k_b; a.v_b = x.v_b; a.q_norm = x.q_norm; a.k_norm = x.k_norm;
+        a.eps = eps;
+        a.temp_coef = x.temp_coef;
+        a.temp_every = x.temp_every;
+        a.rows = runs();
+        a.cache = RowCache{c->kpool[l], c->pt_full, c->pps_full, c->PT, x.ld, x.kv_heads};
+        const int group = x.heads / x.kv_heads;
+        AttnPart part{c->lat_o, c->lat_ml, rs.chunk ? 1 : c->lat_splits, (size_t)R * x.heads};
+        int longest = 1, tile_rows = 0;
+        for (int n : rs.run_len) longest = std::max(longest, n);
+        size_t mma_smem = 0;
+        const HeadMmaFn mma = sizeof(WT) == 2 && sizeof(KT) == 2 ? pick_head_mma(x, longest * group, &tile_rows, &mma_smem) : nullptr;
+        const size_t prep_smem = sizeof(float) * x.heads * x.dim;
+        if (mma) {
+            ln.go("qkv_post", head_prep_kernel<uint16_t, uint16_t>, dim3(R, 3), dim3(256), prep_smem, a, (uint16_t*)c->x_u, x.kd);
+            int units = 0;
+            for (int n : rs.run_len) units += (n * group + tile_rows - 1) / tile_rows;
+            const int most = rs.chunk ? kLatentChunkSplits : c->lat_splits;
+            part.splits = latent_splits(units * x.kv_heads, (rs.max_visible + kHmTile - 1) / kHmTile, most, 2 * m->num_sms);
+            HeadMmaArgs h{};
+            h.q = (const uint16_t*)c->x_u;
+            h.heads = x.heads; h.group = group; h.kd = x.kd; h.vd = x.ld - x.kd; h.vdim = x.vdim;
+            h.scale = x.scale;
+            h.rows = a.rows;
+            h.runs = (int)rs.run_len.size();
+            h.step_tiles = rs.chunk ? 0 : (group + tile_rows - 1) / tile_rows;
+            h.cache = a.cache;
+            h.part = part;
+            ln.go("attn", mma, dim3(units, x.kv_heads, part.splits), dim3(kHmThreads), mma_smem, h);
+        } else {
+            ln.go("qkv_post", head_prep_kernel<float, KT>, dim3(R, 3), dim3(256), prep_smem, a, c->lat_q, x.dim);
+            const RowAttnArgs ra{c->lat_q, x.heads, group, x.dim, x.kd, x.vdim, x.scale, a.rows, a.cache, part};
+            ln.go("attn", pick_row_attn<KT, false>(x.vdim), dim3(x.heads, R, part.splits), dim3(256), row_attn_smem(ra.dk, ra.vw), ra);
+        }
+        const size_t smem = sizeof(float) * part.splits;
+        if (fused) {
+            ln.go("attn_merge", head_merge_kernel<float>, dim3(x.heads, R), dim3(128), smem, x.heads, x.vdim, part, x.sink, OutTail{}, c->attn_out, x.owp);
+            output(x, one(c->attn_out, x.owp), x.vdim, 0, nullptr, in, ACT_NONE);
+            return;
+        }
+        const OutTail tail = ff_tail(x, in);
+        const dim3 grid(x.heads + tail.slices(), R);
+        if (tc) ln.go("attn_merge", head_merge_kernel<uint16_t>, grid, dim3(128), smem, x.heads, x.vdim, part, x.sink, tail, (uint16_t*)c->mix_y, x.o.K);
+        else ln.go("attn_merge", head_merge_kernel<float>, grid, dim3(128), smem, x.heads, x.vdim, part, x.sink, tail, (float*)c->mix_y, x.o.K);
+        pend(project("o", x.o, c->mix_y, c->o_part), nullptr);
+    }
+
+    template <typename WT, typename KT>
+    void attend(const MixPlan& x, int l, const SplitIn& in) {
+        if (x.kind == MIX_LATENT) latent<WT, KT>(x, l, in);
+        else attention<WT, KT>(x, l, in);
     }
 
     void feed_forward(const MixPlan& x) {
@@ -774,7 +995,7 @@ struct LayeredPass {
             a.W0 = x.gateup.w;
             a.W1 = x.gateup.w1;
             residual_args(a, x.norm2);
-            a.act = ACT_SILU;
+            a.act = m->ff_act;
             a.out = c->gu_part;
             launch_gemv(ln, "gateup", c, R, a, x.gateup.gp, PRO_NORM, EPI_GATEUP);
             advance();
@@ -789,7 +1010,7 @@ struct LayeredPass {
         close_rows(x.norm2, c->mix_x, nullptr);
         const SplitIn gu = project("gateup", x.gateup, c->mix_x, c->gu_part);
         ln.go("geglu", geglu_rows_kernel, dim3((x.ffp / 4 + kRowsThreads - 1) / kRowsThreads, R), dim3(kRowsThreads), 0, R, x.ffp,
-              (const float*)c->gu_part, gu.splits, (uint16_t*)c->mix_y, (int)ACT_SILU);
+              (const float*)c->gu_part, gu.splits, (uint16_t*)c->mix_y, m->ff_act);
         pend(project("down", x.down, c->mix_y, c->down_part), x.norm2b);
     }
 };
@@ -802,15 +1023,15 @@ static Pending run_layered(oxg4_cache* c, Launcher& ln, const RowSet& rs, bool u
     for (int l = 0; l < m->cfg.num_hidden_layers && ln.status == OXG4_OK; ++l) {
         const MixPlan& x = m->layers[l].mix;
         const SplitIn in = p.input(x, l);
-        if (x.kind != MIX_LATENT) p.recurrent(x, l, in);
+        if (x.kind != MIX_LATENT && x.kind != MIX_ATTENTION) p.recurrent(x, l, in);
         else if (m->es == 2) {
-            if (c->kv_dtype == OXG4_BF16) p.latent<uint16_t, uint16_t>(x, l, in);
-            else p.latent<uint16_t, float>(x, l, in);
+            if (c->kv_dtype == OXG4_BF16) p.attend<uint16_t, uint16_t>(x, l, in);
+            else p.attend<uint16_t, float>(x, l, in);
         } else {
-            if (c->kv_dtype == OXG4_BF16) p.latent<float, uint16_t>(x, l, in);
-            else p.latent<float, float>(x, l, in);
+            if (c->kv_dtype == OXG4_BF16) p.attend<float, uint16_t>(x, l, in);
+            else p.attend<float, float>(x, l, in);
         }
-        if (x.ff > 0) p.feed_forward(x);
+        if (x.ff > 0 && !m->parallel) p.feed_forward(x);
     }
     p.pd.h = p.cur;
     p.pd.h_out = p.nxt;

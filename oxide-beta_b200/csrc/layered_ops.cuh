@@ -1,6 +1,6 @@
 // Kernels of models whose layers are listed one by one (csrc/layered.inl): recurrent mixers with a matrix state per
-// head (lightning attention, RWKV-style time mixing), token shift, grouped output norms with a gate, and multi-head
-// latent attention over a paged cache of latents. They sit around the projections of gemv.cuh (one row, or f32
+// head (lightning attention, retention, RWKV-style time mixing), token shift, grouped output norms with a gate, and
+// attention over a paged cache of rows: multi-head latent attention, and grouped-query attention with a sink. They sit around the projections of gemv.cuh (one row, or f32
 // weights) and tc_gemm.cuh (BF16 weights, many rows); the sandwich norms and the residual stream are those of
 // rows_norm_kernel / the PRO_NORM prologue.
 //
@@ -37,6 +37,33 @@ struct RunRows {
     const uint32_t* tok;     // [R]; kInactiveToken rows are left out
     DEVINL int seq_of(int row) const { return seq ? seq[row] : row; }
 };
+
+// The rows of a run, per_token of them per token, laid end to end and cut into tiles of `tile_rows`: run and first row
+// (inside the run) of tile t over all runs, run -1 past the end. One warp.
+DEVINL void find_row_tile(const RunRows& rows, int runs, int per_token, int tile_rows, int t, int& run, int& first) {
+    const int lane = threadIdx.x & 31;
+    int base = 0;
+    run = -1;
+    first = 0;
+    for (int r0 = 0; r0 < runs && run < 0; r0 += 32) {
+        const int r = r0 + lane;
+        const int nt = r < runs ? (rows.n[r] * per_token + tile_rows - 1) / tile_rows : 0;
+        int inc = nt;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int v = __shfl_up_sync(0xffffffffu, inc, o);
+            if (lane >= o) inc += v;
+        }
+        const int lo = base + inc - nt;
+        const unsigned hit = __ballot_sync(0xffffffffu, t >= lo && t < lo + nt);
+        if (hit) {
+            const int src = __ffs(hit) - 1;
+            run = r0 + src;
+            first = (t - __shfl_sync(0xffffffffu, lo, src)) * tile_rows;
+        }
+        base += __shfl_sync(0xffffffffu, inc, 31);
+    }
+}
 
 template <typename XT> DEVINL void store_act(XT* p, float v);
 template <> DEVINL void store_act<float>(float* p, float v) { *p = v; }
@@ -119,13 +146,14 @@ wkv_decay_kernel(int R, int N, int rank, SplitIn low, int col, const WT* w2, con
 // ---- recurrence ---------------------------------------------------------------------------------------------
 // Per head a state S [dim, vdim] in f32, walked token by token:
 //   REC_LIGHTNING  q, k, v = silu(.);  S = decay_h S + k v^T;  o = S^T q
+//   REC_RETENTION  the same recurrence; q and k are rotated (channel i with i + rot_dims / 2) and k is scaled instead
 //   REC_WKV        o = (S + diag(u) k v^T)^T r;  S = diag(w) S + k v^T, w per token and key channel
 // The bonus term is v * sum_k r_k u_k k_k, one scalar per token and head.
 // Grid (heads, slices of vdim, runs). A thread owns KPT key channels of two value columns; the KS threads that share
 // a column are neighbouring lanes. Tokens are staged in shared memory in tiles, activations applied on
 // the way; the dot products of up to 8 tokens are reduced across the KS lanes together.
 // State in memory: [sequence][head][vdim][dim]. At position 0 the state starts at zero whatever the memory holds.
-enum { REC_LIGHTNING = 0, REC_WKV = 1 };
+enum { REC_LIGHTNING = 0, REC_WKV = 1, REC_RETENTION = 2 };
 constexpr int kRecThreads = 128;
 constexpr int kRecCols = 2;              // value columns per thread
 constexpr int rec_tile(int dp) { return dp <= 128 ? 16 : dp <= 256 ? 8 : 4; }   // tokens staged at a time
@@ -134,7 +162,10 @@ struct RecurArgs {
     SplitIn in;                          // fused input projection
     int c_q, c_k, c_v;                   // first columns of q (r), k and v, head by head
     int heads, dim, vdim;
-    const float* decay;                  // LIGHTNING: [heads]
+    const float* decay;                  // LIGHTNING, RETENTION: [heads]
+    const float2* freq;                  // RETENTION: [rot_dims / 2] angle per position, high and low part
+    int rot_dims;
+    float k_scale;
     const float* u;                      // WKV: [heads, dim]
     const float* w;                      // WKV: [R, heads * dim] decays, or null: computed here (runs of one token)
     int c_low, rank;                     //   from the low-rank columns
@@ -177,9 +208,18 @@ DEVINL void column_reduce(float (&acc)[N], int ks, int& first) {
 // TILE: tokens staged at a time; 1 for decode steps (row r is sequence r's one token). Tiles of longer runs are
 // double-buffered: the next tile's values are fetched into registers while the current one is walked. A thread's key
 // channels come in groups of four, KS * 4 apart, so that the lanes of a column read neighbouring 16-byte pieces.
+DEVINL void rotation(int pos, float2 freq, float& sn, float& cs) {
+    // the angle to more than f32: p * (hi + lo), its rounding error e turned into a first-order correction
+    const float a = (float)pos * freq.x, e = fmaf((float)pos, freq.x, -a) + (float)pos * freq.y;
+    float s, c;
+    sincosf(a, &s, &c);
+    sn = fmaf(c, e, s);
+    cs = fmaf(-s, e, c);
+}
+
 template <int KIND, typename WT, int KS, int KPT, int TILE>
 __global__ void __launch_bounds__(kRecThreads) recur_kernel(const RecurArgs a) {
-    constexpr bool WKV = KIND == REC_WKV;
+    constexpr bool WKV = KIND == REC_WKV, RET = KIND == REC_RETENTION;
     constexpr int DP = KS * KPT;         // key channels, padded
     constexpr int VG = kRecThreads / KS; // threads along the value columns
     constexpr int VS = VG * kRecCols;    // value columns of this CTA
@@ -276,17 +316,32 @@ __global__ void __launch_bounds__(kRecThreads) recur_kernel(const RecurArgs a) {
         for (int j = 0; j < NK; ++j) {
             const int i = tid + j * kRecThreads;
             if (i < TILE * DP) {
-                sq[i] = WKV ? fq[j] : silu(fq[j]);
-                sk[i] = WKV ? fk[j] : silu(fk[j]);
+                sq[i] = WKV || RET ? fq[j] : silu(fq[j]);
+                sk[i] = WKV ? fk[j] : RET ? fk[j] * a.k_scale : silu(fk[j]);
                 if constexpr (WKV) sw[i] = fw[j];
             }
         }
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
             const int i = tid + j * kRecThreads;
-            if (i < TILE * VS) sv[i] = WKV ? fv[j] : silu(fv[j]);
+            if (i < TILE * VS) sv[i] = WKV || RET ? fv[j] : silu(fv[j]);
         }
         if (t0 + TILE < n) fetch(t0 + TILE);
+        if constexpr (RET) {
+            __syncthreads();
+            const int half = a.rot_dims / 2;
+            for (int i = tid; i < nt * half; i += kRecThreads) {
+                const int t = i / half, d = i % half;
+                float sn, cs;
+                rotation(pos + t0 + t, a.freq[d], sn, cs);
+                float *q = sq + t * DP + d, *k = sk + t * DP + d;
+                const float qu = q[0], qv = q[half], ku = k[0], kv = k[half];
+                q[0] = qu * cs - qv * sn;
+                q[half] = qv * cs + qu * sn;
+                k[0] = ku * cs - kv * sn;
+                k[half] = kv * cs + ku * sn;
+            }
+        }
         if constexpr (WKV && TILE == 1) {
             if (a.w == nullptr) {                            // decay of this head's channels, four lanes per channel
                 float* th = su + DP;                         // [rank]
@@ -400,12 +455,37 @@ __global__ void __launch_bounds__(kRecThreads) recur_kernel(const RecurArgs a) {
 }
 
 // ---- output norm and gate of a mixer ------------------------------------------------------------------------
+// Further columns of an output projection's input, from `at` on: the feed-forward's activations where mixer and
+// feed-forward share the projection. In f32 multi-row passes they are finished values; behind a tcgen05 projection
+// alternately gate and up values, `act` and product still to come. Slices of kTailCols columns.
+constexpr int kTailCols = 1024;
+struct OutTail {
+    SplitIn in;
+    int col, n, at, act;                 // n columns (a multiple of 4; 0: none); act: ACT_NONE for finished values
+    int slices() const { return (n + kTailCols - 1) / kTailCols; }
+};
+
+template <typename XT> DEVINL void out_tail(const OutTail& t, int r, int slice, XT* x_row) {
+    const int end = min(t.n, (slice + 1) * kTailCols);
+    for (int j = slice * kTailCols + threadIdx.x * 4; j < end; j += blockDim.x * 4) {
+        const float* p = t.in.p + (size_t)r * t.in.ld + t.col;
+        float4 v;
+        if (t.act == ACT_NONE) {
+            v = sum_splits4(p + j, t.in.stride, t.in.splits);
+        } else {
+            const float4 a = sum_splits4(p + 2 * j, t.in.stride, t.in.splits), b = sum_splits4(p + 2 * j + 4, t.in.stride, t.in.splits);
+            v = make_float4(glu_mul(t.act, a.x, a.y), glu_mul(t.act, a.z, a.w), glu_mul(t.act, b.x, b.y), glu_mul(t.act, b.z, b.w));
+        }
+        store_x4(x_row + t.at + j, v);
+    }
+}
+
 // x[r, j] = o[r, j] / rms(group of j) * w[j] * act(gate[r, j]); group = 0: no norm, w = null: no weight. The values lie
-// in heads of `hs` columns that start `hs_ld` apart in `o`. One CTA per row, `n` values, padded with zeros to `ld_x`.
+// in heads of `hs` columns that start `hs_ld` apart in `o`. One CTA per row, `n` values, padded with zeros to `n_pad`.
 struct GroupNormArgs {
     SplitIn o;
     int hs, hs_ld;
-    int n, group;
+    int n, n_pad, group;
     const float* w;
     SplitIn gate;
     int c_gate, act;                     // act: ACT_NONE without a gate
@@ -423,15 +503,19 @@ DEVINL void split_load(const SplitIn& in, int row, int col, float (&v)[E]) {
     }
 }
 
-// E: values per access; 4 when every size and column offset is a multiple of 4
+// E: values per access; 4 when every size and column offset is a multiple of 4. grid (R, 1 + slices of the tail)
 template <typename XT, int E>
-__global__ void __launch_bounds__(256) group_norm_rows_kernel(const GroupNormArgs a, XT* x, int ld_x) {
+__global__ void __launch_bounds__(256) group_norm_rows_kernel(const GroupNormArgs a, const OutTail tail, XT* x, int ld_x) {
     __shared__ float red[32];
     extern __shared__ __align__(16) unsigned char smem_raw[];
     float* v = reinterpret_cast<float*>(smem_raw);           // [n]
     pdl_wait();
     pdl_launch();
     const int r = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    if (blockIdx.y > 0) {
+        out_tail(tail, r, blockIdx.y - 1, x + (size_t)r * ld_x);
+        return;
+    }
     float ss[1] = {0.0f};
     for (int j = tid * E; j < a.n; j += blockDim.x * E) {
         float t[E];
@@ -456,7 +540,7 @@ __global__ void __launch_bounds__(256) group_norm_rows_kernel(const GroupNormArg
         }
     }
     __syncthreads();
-    for (int j = tid * E; j < ld_x; j += blockDim.x * E) {
+    for (int j = tid * E; j < a.n_pad; j += blockDim.x * E) {
         float t[E];
 #pragma unroll
         for (int e = 0; e < E; ++e) t[e] = 0.0f;
@@ -487,13 +571,14 @@ __global__ void __launch_bounds__(256) group_norm_rows_kernel(const GroupNormArg
 // The cache row of a token is [latent (rank) | rotated key part (rot)], padded with zeros to `ld` elements; slot =
 // position, pages of `page_tokens` rows. Scores and values are taken in latent space: the query is carried through
 // W_uk ("absorbed") and the attention output through W_uv, so a cached token costs ld elements whatever the heads.
-struct LatentCache {
-    void* pool;                          // [pages][page_tokens][ld]
+struct RowCache {
+    void* pool;                          // [pages][kv_heads][page_tokens][ld]
     const int32_t* page_table;           // [sequences, pages_per_seq]
     int pages_per_seq, page_tokens, ld;
-    DEVINL size_t row(int seq, int pos) const {
+    int kv_heads;                        // rows of a token: 1 for latents
+    DEVINL size_t row(int seq, int pos, int kvh = 0) const {
         const int page = page_table[(size_t)seq * pages_per_seq + pos / page_tokens];
-        return ((size_t)page * page_tokens + pos % page_tokens) * ld;
+        return (((size_t)page * kv_heads + kvh) * page_tokens + pos % page_tokens) * ld;
     }
 };
 
@@ -504,7 +589,7 @@ struct LatentArgs {
     const float *dq_norm, *dkv_norm, *inv_freq;
     float eps, scale;
     RunRows rows;
-    LatentCache cache;
+    RowCache cache;
 };
 
 // rotation of the pair (u, v) = (x[2i], x[2i+1]) at `pos`
@@ -629,24 +714,37 @@ latent_split_query_kernel(const LatentArgs a, int R, SplitIn q, uint16_t* x_u, i
     }
 }
 
-// Split-KV partials of the latent attention: `o` un-normalised [splits][R * heads][rank], `ml` (running maximum,
+// Split-KV partials of attention, `rank` value columns: `o` un-normalised [splits][R * heads][rank], `ml` (running maximum,
 // denominator) [splits][R * heads][2]; a split without a visible key has denominator 0 and leaves `o` unwritten.
-struct LatentPart {
+struct AttnPart {
     float* o;
     float* ml;
     int splits;
     size_t rows;                         // R * heads
 };
 
-// Attention of one (row, head, split) per CTA on the CUDA cores: f32 caches, and BF16 weights with an f32 cache.
-// grid (heads, R, splits), 256 threads, dynamic shared memory (8 + 1) * (rank + rot) + 16 floats. rank <= 32 * RPL.
-template <typename KT, int RPL>
-__global__ void __launch_bounds__(256) latent_attn_kernel(const LatentArgs a, const float* q_abs, LatentPart part) {
+// Attention of one (row, head, split) per CTA on the CUDA cores: f32 caches, BF16 weights with an f32 cache, and heads
+// too wide for the tensor-core kernels. The key of a cache row is its first `dk` elements; its value is `vw` elements
+// from `v_at` on (latent attention: from 0 on, RPL registers hold them for both). Query heads share the cache rows of
+// kv head (head / group). Queries [R, heads, dk] f32. grid (heads, R, splits), 256 threads, dynamic shared memory
+// dk + 8 * vw + 16 floats. vw <= 32 * RPL.
+struct RowAttnArgs {
+    const float* q;
+    int heads, group, dk, v_at, vw;
+    float scale;
+    RunRows rows;
+    RowCache cache;
+    AttnPart part;
+};
+
+template <typename KT, int RPL, bool LATENT>
+__global__ void __launch_bounds__(256) row_attn_kernel(const RowAttnArgs a) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    const int DK = a.rank + a.rot;
+    const AttnPart& part = a.part;
+    const int DK = a.dk, VW = a.vw;
     float* sq = reinterpret_cast<float*>(smem_raw);          // [DK]
-    float* so = sq + DK;                                     // [8][rank]
-    float* sm = so + 8 * a.rank;                             // [8][2]
+    float* so = sq + DK;                                     // [8][VW]
+    float* sm = so + 8 * VW;                                 // [8][2]
     pdl_wait();
     pdl_launch();
     const int hd = blockIdx.x, r = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -659,22 +757,23 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const LatentArgs a, co
         if (tid == 0) { part.ml[2 * pr] = -INFINITY; part.ml[2 * pr + 1] = 0.0f; }
         return;
     }
-    const float* q = q_abs + ((size_t)r * a.heads + hd) * DK;
+    const float* q = a.q + ((size_t)r * a.heads + hd) * DK;
     for (int j = tid; j < DK; j += 256) sq[j] = q[j];
     __syncthreads();
+    const int kvh = hd / a.group;
     float m = -INFINITY, l = 0.0f, acc[RPL];
 #pragma unroll
     for (int i = 0; i < RPL; ++i) acc[i] = 0.0f;
     for (int p = p0 + warp; p < p1; p += 8) {
-        const KT* row = (const KT*)a.cache.pool + a.cache.row(seq, p);
+        const KT* row = (const KT*)a.cache.pool + a.cache.row(seq, p, kvh);
         float c[RPL], s = 0.0f;
 #pragma unroll
         for (int i = 0; i < RPL; ++i) {
             const int j = lane + 32 * i;
-            c[i] = j < a.rank ? WTraits<KT>::elem(row, j) : 0.0f;
-            if (j < a.rank) s = fmaf(sq[j], c[i], s);
+            c[i] = j < VW ? WTraits<KT>::elem(row, (LATENT ? 0 : a.v_at) + j) : 0.0f;
+            if (LATENT && j < VW) s = fmaf(sq[j], c[i], s);
         }
-        for (int j = a.rank + lane; j < DK; j += 32) s = fmaf(sq[j], WTraits<KT>::elem(row, j), s);
+        for (int j = (LATENT ? VW : 0) + lane; j < DK; j += 32) s = fmaf(sq[j], WTraits<KT>::elem(row, j), s);
         s = warp_sum(s) * a.scale;
         const float m2 = fmaxf(m, s), f = expf(m - m2), e = expf(s - m2);
         l = l * f + e;
@@ -684,26 +783,26 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const LatentArgs a, co
     }
 #pragma unroll
     for (int i = 0; i < RPL; ++i)
-        if (lane + 32 * i < a.rank) so[warp * a.rank + lane + 32 * i] = acc[i];
+        if (lane + 32 * i < VW) so[warp * VW + lane + 32 * i] = acc[i];
     if (lane == 0) { sm[2 * warp] = m; sm[2 * warp + 1] = l; }
     __syncthreads();
     float M = -INFINITY, L = 0.0f;
     for (int w = 0; w < 8; ++w) M = fmaxf(M, sm[2 * w]);
     for (int w = 0; w < 8; ++w) L += sm[2 * w + 1] > 0.0f ? sm[2 * w + 1] * expf(sm[2 * w] - M) : 0.0f;
-    for (int j = tid; j < a.rank; j += 256) {
+    for (int j = tid; j < VW; j += 256) {
         float t = 0.0f;
         for (int w = 0; w < 8; ++w)
-            if (sm[2 * w + 1] > 0.0f) t += so[w * a.rank + j] * expf(sm[2 * w] - M);
-        part.o[pr * a.rank + j] = t;
+            if (sm[2 * w + 1] > 0.0f) t += so[w * VW + j] * expf(sm[2 * w] - M);
+        part.o[pr * VW + j] = t;
     }
     if (tid == 0) { part.ml[2 * pr] = M; part.ml[2 * pr + 1] = L; }
 }
 
-// attention output of (row, head) in latent space: column j, partials added in split order; `sc` [splits] holds the
-// factors exp(m_s - M) / L of latent_part_factors
-DEVINL void latent_part_factors(const LatentPart& part, size_t rh, float* sc) {
+// attention output of (row, head): column j of `rank`, partials added in split order; `sc` [splits] holds the factors
+// exp(m_s - M) / L of attn_part_factors. `sink`: score of one more term of the denominator that has no value, or null.
+DEVINL void attn_part_factors(const AttnPart& part, size_t rh, float* sc, const float* sink = nullptr) {
     if (threadIdx.x < 32) {
-        float M = -INFINITY;
+        float M = sink ? *sink : -INFINITY;
         for (int s = threadIdx.x; s < part.splits; s += 32) {
             const float* ml = part.ml + 2 * ((size_t)s * part.rows + rh);
             if (__ldcg(ml + 1) > 0.0f) M = fmaxf(M, __ldcg(ml));
@@ -717,12 +816,13 @@ DEVINL void latent_part_factors(const LatentPart& part, size_t rh, float* sc) {
             L += l * f;
         }
         L = warp_sum(L);
+        if (sink) L += expf(*sink - M);
         __syncwarp();
         for (int s = threadIdx.x; s < part.splits; s += 32) sc[s] = L > 0.0f ? sc[s] / L : 0.0f;
     }
     __syncthreads();
 }
-DEVINL float latent_part_value(const LatentPart& part, size_t rh, int rank, int j, const float* sc) {
+DEVINL float attn_part_value(const AttnPart& part, size_t rh, int rank, int j, const float* sc) {
     const float* o = part.o + rh * rank + j;
     const size_t stride = part.rows * rank;
     float t = 0.0f;
@@ -739,16 +839,16 @@ DEVINL float latent_part_value(const LatentPart& part, size_t rh, int rank, int 
 
 // many rows: merged output as BF16 operands of the per-head products with W_uv, [heads][R][ld]. grid (heads, R)
 __global__ void __launch_bounds__(128)
-latent_merge_kernel(int R, int heads, int rank, LatentPart part, uint16_t* x, int ld) {
+latent_merge_kernel(int R, int heads, int rank, AttnPart part, uint16_t* x, int ld) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     float* sc = reinterpret_cast<float*>(smem_raw);
     pdl_wait();
     pdl_launch();
     const int hd = blockIdx.x, r = blockIdx.y;
     const size_t rh = (size_t)r * heads + hd;
-    latent_part_factors(part, rh, sc);
+    attn_part_factors(part, rh, sc);
     for (int j = threadIdx.x; j < ld; j += 128)
-        store_act(x + ((size_t)hd * R + r) * ld + j, j < rank ? latent_part_value(part, rh, rank, j, sc) : 0.0f);
+        store_act(x + ((size_t)hd * R + r) * ld + j, j < rank ? attn_part_value(part, rh, rank, j, sc) : 0.0f);
 }
 
 // few rows: merge, W_uv and the output gate: out[r, h * vdim + v] = (W_uv[h, v, :] . o) * sigmoid(gate). W_uv rows are
@@ -756,7 +856,7 @@ latent_merge_kernel(int R, int heads, int rank, LatentPart part, uint16_t* x, in
 // grid (heads, R, slices of 32 value columns), 256 threads, shared memory splits + rank floats (16-byte aligned)
 template <typename WT>
 __global__ void __launch_bounds__(256)
-latent_out_kernel(int heads, int rank, int vdim, LatentPart part, const WT* w_uv, int ldw, SplitIn gate, int c_gate,
+latent_out_kernel(int heads, int rank, int vdim, AttnPart part, const WT* w_uv, int ldw, SplitIn gate, int c_gate,
                   const uint32_t* tok, float* out, int ld_out) {
     constexpr int EPL = WTraits<WT>::EPL, PIECES = 512 / (32 * EPL);         // rank <= 512
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -780,8 +880,8 @@ latent_out_kernel(int heads, int rank, int vdim, LatentPart part, const WT* w_uv
     pdl_launch();
     if (tok[r] == kInactiveToken) return;
     const size_t rh = (size_t)r * heads + hd;
-    latent_part_factors(part, rh, sc);
-    for (int j = threadIdx.x; j < rank; j += 256) so[j] = latent_part_value(part, rh, rank, j, sc);
+    attn_part_factors(part, rh, sc);
+    for (int j = threadIdx.x; j < rank; j += 256) so[j] = attn_part_value(part, rh, rank, j, sc);
     __syncthreads();
     float t[4] = {0.0f, 0.0f, 0.0f, 0.0f};
     if (vec) {
@@ -806,6 +906,87 @@ latent_out_kernel(int heads, int rank, int vdim, LatentPart part, const WT* w_uv
             out[(size_t)r * ld_out + c] = t[i] * sigmoid(gate.at(r, c_gate + c));
         }
     }
+}
+
+// ---- grouped-query attention with whole-projection norms ------------------------------------------------------
+// The cache row of a (token, kv head) is [key, zero-padded to kd | value, zero-padded], no ring: slot = position. q and k
+// get their biases, are divided by the root mean square over all heads together and weighted; q is also multiplied by
+// 1 + coef * ln(floor((p + 1) / every) + 1).
+struct HeadAttnArgs {
+    SplitIn in;                          // fused input projection
+    int c_q, c_k, c_v;
+    int heads, kv_heads, dim, vdim, kd;
+    const float *q_b, *k_b, *v_b, *q_norm, *k_norm;
+    float eps, temp_coef;
+    int temp_every;
+    RunRows rows;
+    RowCache cache;
+};
+
+// Queries [R, heads, ld_q] (BF16 rows padded with zeros for the tensor-core kernel, f32 rows of dim values for the other one)
+// and the cache append. grid (R, 3): queries, keys, values. dynamic shared memory heads * dim floats.
+template <typename QT, typename KT>
+__global__ void __launch_bounds__(256) head_prep_kernel(const HeadAttnArgs a, QT* q_out, int ld_q) {
+    __shared__ float red[32];
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* v = reinterpret_cast<float*>(smem_raw);
+    pdl_wait();
+    pdl_launch();
+    const int r = blockIdx.x, part = blockIdx.y, tid = threadIdx.x;
+    if (a.rows.tok[r] == kInactiveToken) return;
+    const int pos = a.rows.pos[r];
+    KT* pool = (KT*)a.cache.pool;
+    if (part == 2) {
+        const int seq = a.rows.seq_of(r), vp = a.cache.ld - a.kd;
+        for (int i = tid; i < a.kv_heads * vp; i += blockDim.x) {
+            const int g = i / vp, d = i % vp, c = g * a.vdim + d;
+            store_act(pool + a.cache.row(seq, pos, g) + a.kd + d, d < a.vdim ? a.in.at(r, a.c_v + c) + a.v_b[c] : 0.0f);
+        }
+        return;
+    }
+    const bool key = part == 1;
+    const int n = (key ? a.kv_heads : a.heads) * a.dim, col = key ? a.c_k : a.c_q;
+    const float *bias = key ? a.k_b : a.q_b, *w = key ? a.k_norm : a.q_norm;
+    float ss[1] = {0.0f};
+    for (int i = tid; i < n; i += blockDim.x) {
+        const float t = a.in.at(r, col + i) + bias[i];
+        v[i] = t;
+        ss[0] += t * t;
+    }
+    block_sum<1>(ss, red);
+    float s = 1.0f / sqrtf(ss[0] / (float)n + a.eps);
+    if (key) {
+        const int seq = a.rows.seq_of(r);
+        for (int i = tid; i < a.kv_heads * a.kd; i += blockDim.x) {
+            const int g = i / a.kd, d = i % a.kd, c = g * a.dim + d;
+            store_act(pool + a.cache.row(seq, pos, g) + d, d < a.dim ? v[c] * s * w[c] : 0.0f);
+        }
+        return;
+    }
+    s *= 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.0f);
+    for (int i = tid; i < a.heads * ld_q; i += blockDim.x) {
+        const int h = i / ld_q, d = i % ld_q, c = h * a.dim + d;
+        store_act(q_out + ((size_t)r * a.heads + h) * ld_q + d, d < a.dim ? v[c] * s * w[c] : 0.0f);
+    }
+}
+
+// Merge of the split partials, with the sink, into the output projection's input; grid (heads + slices of the tail, R),
+// dynamic shared memory: splits floats
+template <typename XT>
+__global__ void __launch_bounds__(128)
+head_merge_kernel(int heads, int vdim, AttnPart part, const float* sink, const OutTail tail, XT* x, int ld_x) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* sc = reinterpret_cast<float*>(smem_raw);
+    pdl_wait();
+    pdl_launch();
+    const int hd = blockIdx.x, r = blockIdx.y;
+    if (hd >= heads) {
+        out_tail(tail, r, hd - heads, x + (size_t)r * ld_x);
+        return;
+    }
+    const size_t rh = (size_t)r * heads + hd;
+    attn_part_factors(part, rh, sc, sink + hd);
+    for (int j = threadIdx.x; j < vdim; j += 128) store_act(x + (size_t)r * ld_x + hd * vdim + j, attn_part_value(part, rh, vdim, j, sc));
 }
 
 }  // namespace oxg4

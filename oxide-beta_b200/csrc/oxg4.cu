@@ -28,6 +28,7 @@
 #include "tc_gemm.cuh"
 #include "layered_ops.cuh"
 #include "latent_mma.cuh"
+#include "head_mma.cuh"
 #include "tp.h"
 
 using namespace oxg4;
@@ -83,11 +84,12 @@ struct Proj {
     const void* w = nullptr;
     const void* w1 = nullptr; // gate/up: the up projection (N counts the gate rows only)
     int N = 0, K = 0, nseg = 1, seg_rows = 0;
+    int glu_from = -1;        // >= 0: from this (even) row on, gate and up rows alternate
     GemvPlan gp;
 };
 
 enum MixerKind { MIX_GQA = OXG4_MIXER_GQA, MIX_LATENT = OXG4_MIXER_LATENT_ATTENTION, MIX_LIGHTNING = OXG4_MIXER_LIGHTNING,
-                 MIX_WKV = OXG4_MIXER_WKV };
+                 MIX_WKV = OXG4_MIXER_WKV, MIX_RETENTION = OXG4_MIXER_RETENTION, MIX_ATTENTION = OXG4_MIXER_ATTENTION };
 
 // What a layer of a layered model (csrc/layered.inl) needs beyond the common part of LayerPlan.
 struct MixPlan {
@@ -97,12 +99,18 @@ struct MixPlan {
     int low_rank = 0, ff = 0, ffp = 0;
     int c_q = 0, c_k = 0, c_v = 0, c_g = 0, c_low = 0, c_dq = 0, c_dkv = 0;  // columns of the fused input projection
     int vpad = 0;             // latent attention: rows per head of the padded W_uv
+    int kv_heads = 1, kd = 0; // attention: kv heads, padded key columns of a cache row
+    int c_ff = 0;             // parallel block: first gate row of the input projection; its output goes behind owp columns
+    float temp_coef = 0;
+    int temp_every = 1;
     float scale = 1;
     Proj in, uq, uk, uv, o, gateup, down;
     const void *w_uk = nullptr, *w_uv = nullptr, *w2 = nullptr;             // checkpoint layout
     const float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
     const float *out_norm = nullptr, *mu = nullptr, *w0 = nullptr, *u = nullptr, *decay = nullptr, *dq_norm = nullptr,
-                *dkv_norm = nullptr, *inv_freq = nullptr;
+                *dkv_norm = nullptr, *inv_freq = nullptr, *q_norm = nullptr, *k_norm = nullptr, *q_b = nullptr, *k_b = nullptr,
+                *v_b = nullptr, *sink = nullptr;
+    const float2* freq2 = nullptr;   // retention: angle per position, high and low part
 };
 
 struct LayerPlan {            // Gemma4DecodeLayerPlan (gemma4_cuda/mod.rs:65-93)
@@ -156,6 +164,9 @@ struct oxg4_model {
     const void* head = nullptr;   // output projection: the embedding table, or a matrix of its own (layered models)
     const float* final_norm = nullptr;
     bool layered = false;         // layers listed one by one (csrc/layered.inl)
+    bool parallel = false;        // mixer and feed-forward side by side behind one norm (OXG4_BLOCK_PARALLEL)
+    int ff_act = ACT_SILU;        // listed layers: activation of the feed-forward's gate
+    float norm_offset = 0;        // listed layers: added to the weights of the block and final norms
     std::vector<oxg4_layer_spec> specs;
     std::vector<std::vector<float>> spec_decay;
     std::vector<void*> owned;     // device allocations of a layered model besides `tensors`
@@ -461,7 +472,9 @@ static int32_t set_gemv_attrs() {
     SETA(PRO_PLAIN, EPI_STORE);
     SETA(PRO_NORM, EPI_GATEUP);
     SETA(PRO_NORM, EPI_LOGITS);
+    if constexpr (sizeof(WT) == 4) SETA(PRO_PLAIN, EPI_STORE_GLU);
     if constexpr (NB == 1) {
+        SETA(PRO_NORM, EPI_STORE_GLU);
         SETA(PRO_SHIFT, EPI_STORE);
         SETA(PRO_GNORM, EPI_STORE);
     }
@@ -1418,10 +1431,13 @@ static void (*pick_gemv(int nb, int pro, int epi))(const GemvArgs) {
     if (pro == PRO_NORM && epi == EPI_LOGITS) return gemv_kernel<WT, NB, PRO_NORM, EPI_LOGITS>;
     if (nb == 1) {
         PICK(1)
+        if (pro == PRO_NORM && epi == EPI_STORE_GLU) return gemv_kernel<WT, 1, PRO_NORM, EPI_STORE_GLU>;
         if (pro == PRO_SHIFT && epi == EPI_STORE) return gemv_kernel<WT, 1, PRO_SHIFT, EPI_STORE>;
         if (pro == PRO_GNORM && epi == EPI_STORE) return gemv_kernel<WT, 1, PRO_GNORM, EPI_STORE>;
     }
     if constexpr (sizeof(WT) == 4) {      // BF16 weights with more than one row use the tensor-core kernel
+        if (pro == PRO_PLAIN && epi == EPI_STORE_GLU)
+            return nb == 1 ? gemv_kernel<WT, 1, PRO_PLAIN, EPI_STORE_GLU> : nb == 2 ? gemv_kernel<WT, 2, PRO_PLAIN, EPI_STORE_GLU> : gemv_kernel<WT, 4, PRO_PLAIN, EPI_STORE_GLU>;
         if (nb == 2) { PICK(2) }
         if (nb == 4) { PICK(4) }
     }
@@ -1552,8 +1568,8 @@ struct RowSet {
     int max_visible = 1;                 // bound on the visible positions of any row (launch geometry only)
 };
 
-// The residual update a pass over the layers leaves to the kernel that follows: h + rmsnorm(sum of raw, w_post),
-// times scalar, goes to h_out.
+// The residual update a pass over the layers leaves to the kernel that follows: h + rmsnorm(sum of raw, w_post) (without
+// the norm where w_post is null), times scalar, goes to h_out.
 struct Pending {
     const float* h = nullptr;
     float* h_out = nullptr;

@@ -5,10 +5,12 @@ from . import _native as N
 from . import synthetic
 from ._native import Oxg4Error
 from .gemma4 import Device, Gemma4ForCausalLM
+from .nozurax import NozuraxForCausalLM
 from .pabovik import PabovikForCausalLM
 
 # `architecture` (or `model_type`) of config.json -> model class
 MODELS = {
+    "Nozurax": NozuraxForCausalLM,
     "Pabovik": PabovikForCausalLM,
     "gemma4": Gemma4ForCausalLM,
     "gemma4_text": Gemma4ForCausalLM,

@@ -268,18 +268,20 @@ def read_checkpoint(directory: str):
     return cfg.get("text_config", cfg), {n[len(PREFIX):]: a for n, a in tensors.items() if n.startswith(PREFIX)}
 
 
-# ---- models of listed layers (pabovik.py) ------------------------------------------------------
+# ---- models of listed layers (layered.py) ------------------------------------------------------
 
 def layered_weight_names(cfg: dict, low_rank: int = 16):
-    """(name, shape, kind) of every tensor. kind: 'matrix' | 'norm' | 'mu' | 'w0' | 'u'."""
+    """(name, shape, kind) of every tensor. kind: 'matrix' | 'norm' (around one) | 'norm0' (around zero) | 'bias' | 'sink' |
+    'mu' | 'w0' | 'u'."""
     H, out = cfg["width"], [("embed", (cfg["vocab"], cfg["width"]), "matrix")]
+    parallel = cfg.get("architecture") == "Nozurax"          # one norm per layer, mixer and feed-forward side by side
     for i, layer in enumerate(cfg["layers"]):
         if layer.get("weights_of") is not None:
             continue
         p, c = f"l{i}.", layer["mixer"]
         heads, dim = c["heads"], c["dim"]
         hd, ow = heads * dim, heads * c.get("vdim", dim)
-        out += [(p + "norm1", (H,), "norm"), (p + "norm1b", (H,), "norm")]
+        out += [(p + "norm1", (H,), "norm0")] if parallel else [(p + "norm1", (H,), "norm"), (p + "norm1b", (H,), "norm")]
         if layer["type"] == "wkv":
             out += [(p + "mix.mu." + s, (H,), "mu") for s in "rkvgw"]
             out += [(p + "mix." + s, (hd, H), "matrix") for s in "rkvg"]
@@ -288,6 +290,13 @@ def layered_weight_names(cfg: dict, low_rank: int = 16):
         elif layer["type"] == "lightning":
             out += [(p + "mix.q", (hd, H), "matrix"), (p + "mix.k", (hd, H), "matrix"), (p + "mix.v", (ow, H), "matrix"),
                     (p + "mix.g", (ow, H), "matrix"), (p + "mix.norm", (ow,), "norm")]
+        elif layer["type"] == "retention":
+            out += [(p + "mix." + s, (n, H), "matrix") for s, n in (("q", hd), ("k", hd), ("v", ow), ("g", ow))]
+        elif layer["type"] == "attention":
+            kd, kw = c["kv_heads"] * dim, c["kv_heads"] * c.get("vdim", dim)
+            for s, n in (("q", hd), ("k", kd), ("v", kw)):
+                out += [(p + "mix." + s, (n, H), "matrix"), (p + "mix." + s + ".b", (n,), "bias")]
+            out += [(p + "mix.q.norm", (hd,), "norm"), (p + "mix.k.norm", (kd,), "norm"), (p + "mix.sink", (heads,), "sink")]
         else:
             rank, rot = c["kv_rank"], c["rot_dim"]
             out += [(p + "mix.dq", (c["q_rank"], H), "matrix"), (p + "mix.dq.norm", (c["q_rank"],), "norm"),
@@ -297,14 +306,14 @@ def layered_weight_names(cfg: dict, low_rank: int = 16):
         out.append((p + "mix.o", (H, ow), "matrix"))
         if layer.get("mlp"):
             ff = layer["mlp"]["ff"]
-            out += [(p + "norm2", (H,), "norm"), (p + "norm2b", (H,), "norm"), (p + "mlp.gate", (ff, H), "matrix"),
-                    (p + "mlp.up", (ff, H), "matrix"), (p + "mlp.down", (H, ff), "matrix")]
-    return out + [("final.norm", (H,), "norm"), ("head", (cfg["vocab"], H), "matrix")]
+            out += [] if parallel else [(p + "norm2", (H,), "norm"), (p + "norm2b", (H,), "norm")]
+            out += [(p + "mlp.gate", (ff, H), "matrix"), (p + "mlp.up", (ff, H), "matrix"), (p + "mlp.down", (H, ff), "matrix")]
+    return out + [("final.norm", (H,), "norm0" if parallel else "norm"), ("head", (cfg["vocab"], H), "matrix")]
 
 
 def layered_weights(cfg: dict, seed: int = 0, low_rank: int = 16, gain: float = 1.0):
-    """Yields (name, BF16 bit pattern array): matrices N(0, gain^2 / columns), norm weights around 1, shift mixes in
-    [0, 1], decay offsets that spread the decays between fast and slow channels."""
+    """Yields (name, BF16 bit pattern array): matrices N(0, gain^2 / columns), norm weights around 1 or 0, shift mixes
+    in [0, 1], decay offsets that spread the decays between fast and slow channels."""
     rng = np.random.default_rng(seed)
     for name, shape, kind in layered_weight_names(cfg, low_rank):
         a = rng.standard_normal(shape, dtype=np.float32)
@@ -312,6 +321,8 @@ def layered_weights(cfg: dict, seed: int = 0, low_rank: int = 16, gain: float = 
             a *= np.float32(gain if name == "embed" else gain / np.sqrt(shape[1]))
         elif kind == "norm":
             a = 1.0 + 0.2 * a
+        elif kind == "norm0":
+            a *= np.float32(0.2)
         elif kind == "mu":
             a = rng.random(shape, dtype=np.float32)
         elif kind == "w0":

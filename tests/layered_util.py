@@ -31,8 +31,21 @@ def latent(heads, dim, vdim, q_rank, kv_rank, rot_dim, scale=None, base=10000.0,
                            "scale": (dim + rot_dim) ** -0.5 if scale is None else scale}}, **kw)
 
 
+def retention(heads, dim, vdim, decay, base=10000.0, rot_dims=None, ff=None, **kw):
+    return dict({"type": "retention", "mlp": ff and {"kind": "dense", "ff": ff},
+                 "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay),
+                           "rot": {"base": base, "dims": dim if rot_dims is None else rot_dims}}}, **kw)
+
+
+def attention(heads, kv_heads, dim, vdim, scale=None, coef=0.7, every=5, ff=None, **kw):
+    return dict({"type": "attention", "mlp": ff and {"kind": "dense", "ff": ff},
+                 "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim,
+                           "scale": dim ** -0.5 if scale is None else scale, "q_temp": {"coef": coef, "every": every}}}, **kw)
+
+
 def config(layers, width=100, vocab=333, eps=1e-5):
-    return {"architecture": "Pabovik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
+    parallel = layers[0]["type"] in ("retention", "attention")
+    return {"architecture": "Nozurax" if parallel else "Pabovik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
 
 
 class Pair:
@@ -46,7 +59,7 @@ class Pair:
                 bits[name] = syn.f32_to_bf16_bits(np.asarray(f(syn.bf16_bits_to_f32(bits[name])), dtype=np.float32))
         self.bits = bits
         self.W = {n: syn.bf16_bits_to_f32(a) for n, a in bits.items()}
-        self.model = pkg.PabovikForCausalLM.from_weights(cfg, bits, pkg.Device.Cuda(0), weight_dtype=self.dtype)
+        self.model = pkg.models.model_class(cfg).from_weights(cfg, bits, pkg.Device.Cuda(0), weight_dtype=self.dtype)
         self.state = self.model.prepare_cuda()
 
     def table(self, max_seq, batch=1, page_tokens=256, kv=None):
