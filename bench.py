@@ -281,9 +281,9 @@ def main():
                          "ingesting the prompts (decode timing at long contexts without the prefill time)")
     ap.add_argument("--layers", type=int, default=None, help="profiling aid: keep only the first LAYERS layers")
     ap.add_argument("--vocab", type=int, default=None, help="profiling aid: shrink the vocabulary")
-    ap.add_argument("--design", default=None, choices=["pabovik"],
+    ap.add_argument("--design", default=None, choices=["pabovik", "nozurax"],
                     help="instead of the workload: prefill and decode throughput and per-kernel times of this design at a few "
-                         "sizes, beside a Gemma 4 model of equal width, depth and feed-forward (bench_layered.py)")
+                         "sizes, beside models of equal width, depth and feed-forward: Gemma 4, for nozurax also Pabovik (bench_layered.py)")
     args = ap.parse_args()
     if args.design:
         import bench_layered

@@ -1,5 +1,6 @@
-"""Throughput of models of listed layers beside a Gemma 4 model of equal width, depth, feed-forward and vocabulary.
-Run through `python bench.py --design pabovik`; prints ONE JSON line.
+"""Throughput of models of listed layers beside models of equal width, depth, feed-forward and vocabulary: Gemma 4, and for
+Nozurax (whose recurrence is like lightning attention) also Pabovik. Run through `python bench.py --design pabovik|nozurax`;
+prints ONE JSON line.
 
 Per size and model: prefill tokens/s (one prompt of 4096 tokens in one call, host clock around the call, which ends with a
 synchronisation), decode tokens/s of the captured greedy step (CUDA events on the library's stream) for one sequence and for
@@ -28,8 +29,8 @@ def peaks():
     return 6.65e12, 1.59e15, "fallback"
 
 
-def sizes():
-    """name -> (Pabovik config, Gemma 4 config) of equal width, depth, feed-forward and vocabulary."""
+def sizes(design):
+    """name -> {model: config} of equal width, depth, feed-forward and vocabulary, the design's own first."""
     syn = importlib.import_module("oxide-beta_b200").synthetic
     out = {}
     for name, width, heads, ff, q_rank in (("w2560", 2560, 16, 10240, 1024), ("w4096", 4096, 32, 14336, 1536)):
@@ -41,9 +42,17 @@ def sizes():
                "mixer": {"heads": width // 128, "dim": 128, "vdim": 128,
                          "decay": [float(np.exp(-2.0 ** (-8.0 * (h + 1) / (width // 128)))) for h in range(width // 128)]}}
         layers = [wkv, lat, lit] * 4
-        cfg = {"architecture": "Pabovik", "vocab": 65536, "width": width, "norm": {"eps": 1e-6}, "layers": layers}
-        gem = syn._cfg(65536, width, len(layers), heads // 2, heads // 4, 256, ff, 1024)
-        out[name] = (cfg, gem)
+        models = {"pabovik": {"architecture": "Pabovik", "vocab": 65536, "width": width, "norm": {"eps": 1e-6}, "layers": layers},
+                  "gemma4": syn._cfg(65536, width, len(layers), heads // 2, heads // 4, 256, ff, 1024)}
+        if design == "nozurax":
+            att = {"type": "attention", "mlp": {"kind": "dense", "ff": ff},
+                   "mixer": {"heads": width // 128, "kv_heads": width // 512, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                             "q_temp": {"coef": 0.1, "every": 8192}}}
+            ret = {"type": "retention", "mlp": {"kind": "dense", "ff": ff},
+                   "mixer": dict(lit["mixer"], rot={"dims": 128, "base": 10000.0})}
+            models = {"nozurax": {"architecture": "Nozurax", "vocab": 65536, "width": width, "norm": {"eps": 1e-6},
+                                  "layers": [att, ret] * (len(layers) // 2)}, **models}
+        out[name] = models
     return out
 
 
@@ -55,6 +64,8 @@ def device_weights(names):
         t = torch.empty(shape, dtype=torch.float32, device="cuda")
         if kind in ("matrix",):
             t.normal_(0.0, shape[-1] ** -0.5, generator=gen)
+        elif kind in ("norm0", "bias", "sink"):
+            t.normal_(0.0, 0.2, generator=gen)
         elif kind == "w0":
             t.uniform_(-6.0, 0.5, generator=gen)
         elif kind == "mu":
@@ -77,7 +88,20 @@ def work(cfg, kind, rows, contexts, chunk):
         def gemm(n, k, heads_=1):
             return heads_ * (2 * n * k + 2 * rows * k + 4 * rows * n), heads_ * 2 * n * k * rows
 
-        if kind == "gateup":
+        if t in ("attention", "retention"):
+            # mixer, gate and up rows are one input projection, mixer and feed-forward columns one output projection
+            kvh = c.get("kv_heads")
+            if kind == "o":
+                got.append(gemm(H, heads * vdim + ff))
+            elif kind == "qkv":
+                got.append(gemm(2 * ff + (heads * dim + kvh * (dim + vdim) if kvh else 2 * heads * (dim + vdim)), H))
+            elif kvh and kind == "attn":
+                seqs = 1 if chunk else rows
+                got.append((2 * seqs * contexts * kvh * (dim + vdim), 2 * rows * heads * contexts * (dim + vdim)))
+            elif not kvh and kind == "recur":
+                got.append((8 * (1 if chunk else rows) * heads * dim * vdim + 4 * rows * heads * 2 * (dim + vdim),
+                            6 * rows * heads * dim * vdim))
+        elif kind == "gateup":
             got.append(gemm(2 * ff, H))
         elif kind == "down":
             got.append(gemm(H, ff))
@@ -186,16 +210,18 @@ def main(design):
     hbm, tf, kind = peaks()
     out = {"design": design, "data": "synthetic", "dtype": "bf16", "context": CONTEXT, "batch": BATCH,
            "peaks": {"hbm_gbs": hbm / 1e9, "bf16_tflops": tf / 1e12, "kind": kind}, "sizes": {}}
-    for name, (cfg, gem) in sizes().items():
+    for name, models in sizes(design).items():
         r = {}
-        state = pkg.PabovikCudaState.load(pkg.PabovikConfig(cfg), device_weights(syn.layered_weight_names(cfg, low_rank=64)))
-        r["pabovik"] = {"weight_gb": round(state.weight_bytes() / 1e9, 3),
-                        **measure(pkg, state, cfg["vocab"], lambda k, n, c, ch: work(cfg, k, n, c, ch))}
-        state.close()
-        state = pkg.Gemma4CudaState.load(pkg.Gemma4TextConfig(gem), device_weights(syn.weight_names(gem)))
-        r["gemma4"] = {"weight_gb": round(state.weight_bytes() / 1e9, 3),
-                       **measure(pkg, state, gem["vocab_size"], lambda k, n, c, ch: gemma_work(gem, k, n, c, ch))}
-        state.close()
+        for model, cfg in models.items():
+            if model == "gemma4":
+                state, counter = pkg.Gemma4CudaState.load(pkg.Gemma4TextConfig(cfg), device_weights(syn.weight_names(cfg))), gemma_work
+            else:
+                cls = pkg.models.model_class(cfg)
+                state = cls.STATE.load(cls.CONFIG(cfg), device_weights(syn.layered_weight_names(cfg, low_rank=64)))
+                counter = work
+            r[model] = {"weight_gb": round(state.weight_bytes() / 1e9, 3),
+                        **measure(pkg, state, state.config.vocab_size, lambda k, n, c, ch: counter(cfg, k, n, c, ch))}
+            state.close()
         out["sizes"][name] = r
     sys.stdout.flush()
     os.write(json_fd, (json.dumps(out) + "\n").encode())

@@ -52,8 +52,8 @@ __global__ void __launch_bounds__(kHmThreads) head_mma_kernel(const HeadMmaArgs 
     uint16_t* skv = sq + (size_t)ROWS * qld;                         // [NST][tile][ldp]
     __shared__ int s_run, s_first;
     __shared__ float s_ml[kHmWarps][16][2];
-    pdl_wait();
-    pdl_launch();
+    // Rows, positions and pages were there before the preceding kernel started, and so were the cached tokens of earlier steps:
+    // they are read ahead of the dependency wait. The queries and this pass's own cache rows are not.
     const int kvh = blockIdx.y, split = blockIdx.z;
     const int t = gridDim.x - 1 - blockIdx.x;        // the longest rows are at the end of a run: they start first
     int run, first, row0, n_flat;
@@ -69,11 +69,19 @@ __global__ void __launch_bounds__(kHmThreads) head_mma_kernel(const HeadMmaArgs 
         __syncthreads();
         run = s_run;
         first = s_first;
-        if (run < 0) return;
+        if (run < 0) {
+            pdl_wait();
+            pdl_launch();
+            return;
+        }
         row0 = a.rows.row0[run];
         n_flat = a.rows.n[run] * a.group;
     }
-    if (a.rows.tok[row0] == kInactiveToken) return;
+    if (a.rows.tok[row0] == kInactiveToken) {
+        pdl_wait();
+        pdl_launch();
+        return;
+    }
     const int seq = a.rows.seq_of(row0), n_here = min(ROWS, n_flat - first);
     const int visible = a.rows.pos[row0 + (first + n_here - 1) / a.group] + 1;
     const int tiles = (visible + kHmTile - 1) / kHmTile, per = (tiles + a.part.splits - 1) / a.part.splits;
@@ -83,6 +91,8 @@ __global__ void __launch_bounds__(kHmThreads) head_mma_kernel(const HeadMmaArgs 
         return (size_t)split * a.part.rows + (size_t)(row0 + f / a.group) * a.heads + kvh * a.group + f % a.group;
     };
     if (tile0 >= tile1) {
+        pdl_wait();
+        pdl_launch();
         if (tid < n_here) {
             float* ml = a.part.ml + 2 * part_row(tid);
             ml[0] = -INFINITY;
@@ -91,25 +101,37 @@ __global__ void __launch_bounds__(kHmThreads) head_mma_kernel(const HeadMmaArgs 
         return;
     }
     const uint16_t* pool = (const uint16_t*)a.cache.pool;
-    // a lane looks up the page of one of its warp's rows, one tile ahead of the copies
+    // a lane looks up the page of one of its warp's rows, one tile ahead of the copies; its place in the pages moves on tile by tile
+    const int32_t* pages = a.cache.page_table + (size_t)seq * a.cache.pages_per_seq;
+    const int my_row = warp * RPW + (lane & (RPW - 1));
+    int page_i = (tile0 * kHmTile + my_row) / a.cache.page_tokens, page_o = (tile0 * kHmTile + my_row) % a.cache.page_tokens;
     size_t row_off = 0;
     bool row_ok = false;
-    auto look_up = [&](int tile) {
-        const int p = tile * kHmTile + warp * RPW + lane;
-        row_ok = lane < RPW && tile < tile1 && p < visible;
-        row_off = row_ok ? a.cache.row(seq, p, kvh) : 0;
-    };
-    const int chunks = ld / 8;
-    auto load_tile = [&](int stage) {
-        const unsigned valid = __ballot_sync(0xffffffffu, row_ok);
-        const uint32_t dst = smem_u32(skv + ((size_t)stage * kHmTile + warp * RPW) * ldp) + lane * 16;
-#pragma unroll
-        for (int i = 0; i < RPW; ++i) {
-            const uint16_t* src = pool + __shfl_sync(0xffffffffu, row_off, i) + lane * 8;
-            const bool ok = (valid >> i) & 1;
-            for (int c = 0; lane + 32 * c < chunks; ++c) cp_async16(dst + i * ldp * 2 + c * 512, src + c * 256, ok);
+    auto look_up = [&](int tile) {                   // called for tile0, tile0 + 1, ...
+        row_ok = tile < tile1 && tile * kHmTile + my_row < visible;
+        row_off = row_ok ? (((size_t)pages[page_i] * a.cache.kv_heads + kvh) * a.cache.page_tokens + page_o) * ld : 0;
+        page_o += kHmTile;
+        while (page_o >= a.cache.page_tokens) {
+            page_o -= a.cache.page_tokens;
+            ++page_i;
         }
     };
+    constexpr int LPR = COLS >= 128 ? 32 : COLS / 4, RPI = 32 / LPR, CPL = (COLS / 4 + 31) / 32;     // lanes per row, rows at a time, pieces per lane
+    const int chunk0 = lane & (LPR - 1), chunks = ld / 8;
+    auto load_tile = [&](int stage) {
+        const unsigned valid = __ballot_sync(0xffffffffu, row_ok);
+        const uint32_t dst = smem_u32(skv + ((size_t)stage * kHmTile + warp * RPW) * ldp) + chunk0 * 16;
+#pragma unroll
+        for (int i = 0; i < RPW; i += RPI) {
+            const int r = i + lane / LPR;
+            const uint16_t* src = pool + __shfl_sync(0xffffffffu, row_off, r) + chunk0 * 8;
+#pragma unroll
+            for (int c = 0; c < CPL; ++c)
+                if (chunk0 + 32 * c < chunks) cp_async16(dst + r * ldp * 2 + c * 512, src + c * 256, (valid >> r) & 1);
+        }
+    };
+    const bool early = (tile0 + NST - 1) * kHmTile <= a.rows.pos[row0];      // the first tiles hold no token of this pass
+    if (!early) pdl_wait();
     look_up(tile0);
 #pragma unroll
     for (int i = 0; i < NST - 1; ++i) {
@@ -117,6 +139,8 @@ __global__ void __launch_bounds__(kHmThreads) head_mma_kernel(const HeadMmaArgs 
         cp_async_commit();                           // one group per tile, empty past the end
         look_up(tile0 + i + 1);
     }
+    if (early) pdl_wait();
+    pdl_launch();
     for (int i = tid; i < ROWS * (a.kd / 8); i += kHmThreads) {
         const int row = i / (a.kd / 8), ch = i % (a.kd / 8), f = first + row;
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
@@ -132,13 +156,18 @@ __global__ void __launch_bounds__(kHmThreads) head_mma_kernel(const HeadMmaArgs 
         lim[h] = i < n_here ? a.rows.pos[row0 + (first + i) / a.group] : -1;
     }
     __syncthreads();
+    // Steps past kd multiply zero queries with columns that are there, value columns past vd are computed and not stored:
+    // the loops have no branches, so the loads of a step overlap the products of the one before.
     const int ksteps = a.kd / 16, vpairs = a.vd / 16;
     const uint32_t q_base = smem_u32(sq) + ((wr * 16 + (lane & 15)) * qld + (lane >> 4) * 8) * 2;
     uint32_t qf[QREG ? KSTEPS : 1][4];
     if constexpr (QREG) {
 #pragma unroll
-        for (int k = 0; k < KSTEPS; ++k)
-            if (k < ksteps) ldmatrix_x4(qf[k], q_base + k * 32);
+        for (int k = 0; k < KSTEPS; ++k) {
+            ldmatrix_x4(qf[k], q_base + min(k, ksteps - 1) * 32);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) qf[k][e] = k < ksteps ? qf[k][e] : 0u;
+        }
     }
     float o[VT][4];
 #pragma unroll
@@ -164,18 +193,20 @@ __global__ void __launch_bounds__(kHmThreads) head_mma_kernel(const HeadMmaArgs 
         const uint32_t kb = kv + (((lane >> 4) * 8 + (lane & 7)) * ldp + ((lane >> 3) & 1) * 8) * 2;
 #pragma unroll
         for (int k = 0; k < KSTEPS; ++k) {
-            if (k >= ksteps) break;
+            const int col = min(k, ksteps - 1) * 16;
             uint32_t q[4];
             if constexpr (QREG) {
 #pragma unroll
                 for (int e = 0; e < 4; ++e) q[e] = qf[k][e];
             } else {
-                ldmatrix_x4(q, q_base + k * 32);
+                ldmatrix_x4(q, q_base + col * 2);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) q[e] = k < ksteps ? q[e] : 0u;
             }
 #pragma unroll
             for (int j = 0; j < ST; j += 2) {
                 uint32_t b[4];
-                ldmatrix_x4(b, kb + (j * 8 * ldp + k * 16) * 2);
+                ldmatrix_x4(b, kb + (j * 8 * ldp + col) * 2);
                 mma_bf16_16816(s[j], q, b[0], b[1]);
                 mma_bf16_16816(s[j + 1], q, b[2], b[3]);
             }
@@ -229,9 +260,8 @@ __global__ void __launch_bounds__(kHmThreads) head_mma_kernel(const HeadMmaArgs 
             }
 #pragma unroll
             for (int j = 0; j < VT / 2; ++j) {
-                if (j >= vpairs) break;
                 uint32_t b[4];
-                ldmatrix_x4_trans(b, v_base + (k * 16 * ldp + j * 16) * 2);
+                ldmatrix_x4_trans(b, v_base + (k * 16 * ldp + min(j, vpairs - 1) * 16) * 2);
                 mma_bf16_16816(o[2 * j], ph, b[0], b[1]);
                 mma_bf16_16816(o[2 * j + 1], ph, b[2], b[3]);
                 mma_bf16_16816(o[2 * j], pl, b[0], b[1]);

@@ -233,7 +233,7 @@ static int32_t finalize_parallel(oxg4_model* m, const std::string& pre, const ox
     x.decay = (const float*)d;
     std::vector<float2> freq(std::max(1, x.rot_dims / 2));
     for (int i = 0; i < x.rot_dims / 2; ++i) {
-        const double f = std::pow((double)s.rot_base, -2.0 * i / (double)x.rot_dims);
+        const double f = std::pow((double)s.rot_base, -2.0 * i / (double)x.rot_dims) / 6.283185307179586476925;   // turns
         freq[i].x = (float)f;
         freq[i].y = (float)(f - (double)freq[i].x);
     }
@@ -418,7 +418,7 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
         return n * std::max((size_t)layered_splits(m, p, B, false) * B, (size_t)layered_splits(m, p, kPrefillRows, true) * kPrefillRows);
     };
     size_t in_n = 1, o_n = 1, gu_n = 1, down_n = 1, q_n = 1, uk_n = 1, uv_n = 1, dec = 1, latq = 1, rh = 1, rh_rank = 1, xo = 1, xi = 1, xq = 1,
-           xu = 1, xl = 1, rot = 1, act = 1;
+           xu = 1, xl = 1, rot = 1, act = 1, block_n = 1;
     bool any_shift = false;
     const int max_tiles = (*std::max_element(c->max_seq.begin(), c->max_seq.end()) + kLmTile - 1) / kLmTile;
     c->lat_splits = std::max(2, std::min({max_tiles, 64, (4 * m->num_sms + B - 1) / B}));
@@ -469,6 +469,10 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
             const size_t n = (size_t)B * x.heads * x.dim * x.vdim;
             TRY(dalloc(c, &c->state[l], n));
             c->kv_bytes += (int64_t)(4 * n);
+            if (x.kind != MIX_WKV) {
+                block_n = std::max(block_n, (size_t)x.heads * x.dim * x.vdim);
+                latq = std::max(latq, (size_t)x.heads * x.dim);
+            }
             if (x.kind == MIX_WKV) {
                 TRY(dalloc(c, &c->shift[l], (size_t)B * H));
                 c->kv_bytes += (int64_t)(4 * (size_t)B * H);
@@ -496,6 +500,7 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
         TRY(dalloc(c, &c->xf, (size_t)R * H));
         TRY(dalloc(c, &c->wdec, (size_t)R * dec));
     }
+    TRY(dalloc(c, &c->block_state, 2 * (kPrefillRows / kRecBlock) * block_n));
     TRY(dalloc(c, &c->q_buf, q_n));
     TRY(bytes_alloc(&c->x_q, (size_t)R * xq * xes));
     TRY(dalloc(c, &c->lat_q, (size_t)R * latq));
@@ -511,14 +516,21 @@ static int32_t layered_cache_build(oxg4_cache* c, int pages_full) {
 }
 
 // ---- a pass over the layers -----------------------------------------------------------------------------------
+static_assert(kRecMaxBlocks * kRecBlock == kPrefillRows, "blocks of a pass");
 typedef void (*RecurFn)(const RecurArgs);
+// lanes along the key channels and channels per lane for heads of `dim`
+static void recur_shape(int dim, int* ks, int* kpt) {
+    *kpt = dim <= 64 ? 8 : 16;
+    *ks = dim <= 32 ? 4 : dim <= 128 ? 8 : dim <= 256 ? 16 : 32;
+}
+// step: decode step
 template <int KIND, typename WT>
-static RecurFn pick_recur(int dim, bool step, int* ks, int* kpt) {
-#define PR(KS, KPT)                                    \
-    if (dim <= KS * KPT) {                             \
-        *ks = KS;                                      \
-        *kpt = KPT;                                    \
-        return step ? recur_kernel<KIND, WT, KS, KPT, 1> : recur_kernel<KIND, WT, KS, KPT, rec_tile(KS * KPT)>; \
+static RecurFn pick_recur(int ks, int kpt, bool step) {
+#define PR(KS, KPT)                                                                          \
+    if (ks == KS && kpt == KPT) {                                                            \
+        if (step) return recur_kernel<KIND, WT, KS, KPT, 1>;                                 \
+        if constexpr (KIND == REC_WKV) return recur_kernel<KIND, WT, KS, KPT, rec_tile(KS * KPT)>; \
+        else return fixed_recur_kernel<KIND, KS, KPT>;                                       \
     }
     PR(4, 8) PR(8, 8) PR(8, 16) PR(16, 16) PR(32, 16)
 #undef PR
@@ -596,9 +608,10 @@ static int32_t head_attn_setup(const MixPlan& x) {
         HeadMmaFn fn = pick_head_mma(x, rows, &tr, &smem);
         if (fn) TRY(allow_big_smem(fn));
     }
-    TRY((allow_big_smem(head_prep_kernel<uint16_t, uint16_t>)));
-    TRY((allow_big_smem(head_prep_kernel<float, uint16_t>)));
-    return allow_big_smem((head_prep_kernel<float, float>));
+    for (auto fn : {head_prep_kernel<uint16_t, uint16_t, 1>, head_prep_kernel<uint16_t, uint16_t, 4>}) TRY(allow_big_smem(fn));
+    for (auto fn : {head_prep_kernel<float, uint16_t, 1>, head_prep_kernel<float, uint16_t, 4>}) TRY(allow_big_smem(fn));
+    for (auto fn : {head_prep_kernel<float, float, 1>, head_prep_kernel<float, float, 4>}) TRY(allow_big_smem(fn));
+    return OXG4_OK;
 }
 
 // Splits of `tiles` cache tiles when `units` row tiles share the GPU: the cheapest number of rounds times tiles per CTA, with
@@ -834,17 +847,33 @@ struct LayeredPass {
             a.rot_dims = x.rot_dims;
             a.k_scale = 1.0f / sqrtf((float)x.dim);
         }
-        int ks = 1, kpt = 1;
+        int ks, kpt;
+        recur_shape(x.dim, &ks, &kpt);
         RecurFn fn;
         const bool step = !rs.chunk;
-        if (wkv) fn = m->es == 2 ? pick_recur<REC_WKV, uint16_t>(x.dim, step, &ks, &kpt) : pick_recur<REC_WKV, float>(x.dim, step, &ks, &kpt);
-        else if (ret) fn = pick_recur<REC_RETENTION, float>(x.dim, step, &ks, &kpt);
-        else fn = pick_recur<REC_LIGHTNING, float>(x.dim, step, &ks, &kpt);
+        if (wkv) fn = m->es == 2 ? pick_recur<REC_WKV, uint16_t>(ks, kpt, step) : pick_recur<REC_WKV, float>(ks, kpt, step);
+        else fn = ret ? pick_recur<REC_RETENTION, float>(ks, kpt, step) : pick_recur<REC_LIGHTNING, float>(ks, kpt, step);
         const int vs = kRecThreads / ks * kRecCols, dp = ks * kpt, tile = step ? 1 : rec_tile(dp);
-        const size_t smem = sizeof(float) * ((step ? 1 : 2) * ((size_t)tile * dp * (wkv ? 3 : 2) + tile * vs + pad_to(tile, 4)) +
-                                             (wkv ? dp + x.low_rank : 0));
+        size_t smem = sizeof(float) * ((step ? 1 : 2) * ((size_t)tile * dp * (wkv ? 3 : 2) + tile * vs + pad_to(tile, 4)) + (wkv ? dp + x.low_rank : 0));
+        int parts = (int)rs.run_len.size();
+        bool join = false;
+        if (!step && !wkv) {               // blocks of the runs, joined where a run has several
+            smem = fixed_recur_smem(ks, kpt);
+            parts = 0;
+            for (int n : rs.run_len) {
+                parts += (n + kRecBlock - 1) / kRecBlock;
+                join |= n > kRecBlock;
+            }
+            a.runs = (int)rs.run_len.size();
+            a.block_state = c->block_state;
+            a.block_q = c->lat_q;
+        }
         if (ln.status == OXG4_OK && smem > 48 * 1024) ln.status = allow_big_smem(fn);
-        ln.go("recur", fn, dim3(x.heads, (x.vdim + vs - 1) / vs, (unsigned)rs.run_len.size()), dim3(kRecThreads), smem, a);
+        ln.go("recur", fn, dim3(x.heads, (x.vdim + vs - 1) / vs, (unsigned)parts), dim3(kRecThreads), smem, a);
+        if (join) {
+            if (ln.status == OXG4_OK && join_smem(x.dim) > 48 * 1024) ln.status = allow_big_smem(recur_join_kernel);
+            ln.go("recjoin", recur_join_kernel, dim3(x.heads, (x.vdim + kJoinCols - 1) / kJoinCols, (unsigned)parts), dim3(kJoinThreads), join_smem(x.dim), a);
+        }
         if (ret) output(x, one(c->attn_out, x.owp), x.vdim, x.vdim, nullptr, in, ACT_SILU);
         else output(x, one(c->attn_out, x.owp), x.vdim, wkv ? x.dim : x.ow, x.out_norm, in, wkv ? ACT_SILU : ACT_SIGMOID);
     }
@@ -949,8 +978,11 @@ struct LayeredPass {
         size_t mma_smem = 0;
         const HeadMmaFn mma = sizeof(WT) == 2 && sizeof(KT) == 2 ? pick_head_mma(x, longest * group, &tile_rows, &mma_smem) : nullptr;
         const size_t prep_smem = sizeof(float) * x.heads * x.dim;
+        const bool vec = x.dim % 4 == 0 && x.vdim % 4 == 0;
+        const dim3 prep_block(R <= m->num_sms ? 1024 : 256);
         if (mma) {
-            ln.go("qkv_post", head_prep_kernel<uint16_t, uint16_t>, dim3(R, 3), dim3(256), prep_smem, a, (uint16_t*)c->x_u, x.kd);
+            ln.go("qkv_post", vec ? head_prep_kernel<uint16_t, uint16_t, 4> : head_prep_kernel<uint16_t, uint16_t, 1>, dim3(R, 3), prep_block, prep_smem, a,
+                  (uint16_t*)c->x_u, x.kd);
             int units = 0;
             for (int n : rs.run_len) units += (n * group + tile_rows - 1) / tile_rows;
             const int most = rs.chunk ? kLatentChunkSplits : c->lat_splits;
@@ -966,7 +998,7 @@ struct LayeredPass {
             h.part = part;
             ln.go("attn", mma, dim3(units, x.kv_heads, part.splits), dim3(kHmThreads), mma_smem, h);
         } else {
-            ln.go("qkv_post", head_prep_kernel<float, KT>, dim3(R, 3), dim3(256), prep_smem, a, c->lat_q, x.dim);
+            ln.go("qkv_post", vec ? head_prep_kernel<float, KT, 4> : head_prep_kernel<float, KT, 1>, dim3(R, 3), prep_block, prep_smem, a, c->lat_q, x.dim);
             const RowAttnArgs ra{c->lat_q, x.heads, group, x.dim, x.kd, x.vdim, x.scale, a.rows, a.cache, part};
             ln.go("attn", pick_row_attn<KT, false>(x.vdim), dim3(x.heads, R, part.splits), dim3(256), row_attn_smem(ra.dk, ra.vw), ra);
         }

@@ -149,21 +149,29 @@ wkv_decay_kernel(int R, int N, int rank, SplitIn low, int col, const WT* w2, con
 //   REC_RETENTION  the same recurrence; q and k are rotated (channel i with i + rot_dims / 2) and k is scaled instead
 //   REC_WKV        o = (S + diag(u) k v^T)^T r;  S = diag(w) S + k v^T, w per token and key channel
 // The bonus term is v * sum_k r_k u_k k_k, one scalar per token and head.
-// Grid (heads, slices of vdim, runs). A thread owns KPT key channels of two value columns; the KS threads that share
+// recur_kernel: decode steps, and time mixing in prompts. Grid (heads, slices of vdim, runs). A thread owns KPT key channels of two value columns; the KS threads that share
 // a column are neighbouring lanes. Tokens are staged in shared memory in tiles, activations applied on
 // the way; the dot products of up to 8 tokens are reduced across the KS lanes together.
 // State in memory: [sequence][head][vdim][dim]. At position 0 the state starts at zero whatever the memory holds.
+//
+// Prompts with fixed decays (LIGHTNING, RETENTION) go through fixed_recur_kernel: a run is cut into blocks of kRecBlock tokens
+// that are walked side by side, every block but the first from a zero state, and recur_join_kernel adds what the state at a
+// block's start contributes: o_t += decay^(t + 1) S_start^T q_t for the block's t-th token, S_start = sum of the earlier
+// blocks' end states times the decay in between. End states lie in slots of their own, 2 * (first row / kRecBlock), plus one
+// for a block that is not full: full blocks begin kRecBlock rows apart, and a last, shorter block follows a full one.
 enum { REC_LIGHTNING = 0, REC_WKV = 1, REC_RETENTION = 2 };
 constexpr int kRecThreads = 128;
 constexpr int kRecCols = 2;              // value columns per thread
-constexpr int rec_tile(int dp) { return dp <= 128 ? 16 : dp <= 256 ? 8 : 4; }   // tokens staged at a time
+constexpr int kRecBlock = 64;            // tokens of a block
+constexpr int kRecMaxBlocks = 4;         // blocks of the longest run (a pass carries at most 256 rows)
+__host__ __device__ constexpr int rec_tile(int dp) { return dp <= 128 ? 16 : dp <= 256 ? 8 : 4; }   // tokens staged at a time
 
 struct RecurArgs {
     SplitIn in;                          // fused input projection
     int c_q, c_k, c_v;                   // first columns of q (r), k and v, head by head
     int heads, dim, vdim;
     const float* decay;                  // LIGHTNING, RETENTION: [heads]
-    const float2* freq;                  // RETENTION: [rot_dims / 2] angle per position, high and low part
+    const float2* freq;                  // RETENTION: [rot_dims / 2] turns per position, high and low part
     int rot_dims;
     float k_scale;
     const float* u;                      // WKV: [heads, dim]
@@ -172,6 +180,9 @@ struct RecurArgs {
     const void* w2;                      //   [heads * dim, rank]
     const float* w0;                     //   [heads * dim]
     float* state;
+    float* block_state;                  // fixed_recur_kernel: [slots][heads][vdim][dim]
+    float* block_q;                      //   [R, heads * dim] activated queries for recur_join_kernel
+    int runs;
     RunRows rows;
     float* out;                          // [R, ld_out]
     int ld_out;
@@ -208,13 +219,33 @@ DEVINL void column_reduce(float (&acc)[N], int ks, int& first) {
 // TILE: tokens staged at a time; 1 for decode steps (row r is sequence r's one token). Tiles of longer runs are
 // double-buffered: the next tile's values are fetched into registers while the current one is walked. A thread's key
 // channels come in groups of four, KS * 4 apart, so that the lanes of a column read neighbouring 16-byte pieces.
+// sine and cosine of the angle at `pos`: p * (hi + lo) turns to more than f32, whole turns taken off exactly
 DEVINL void rotation(int pos, float2 freq, float& sn, float& cs) {
-    // the angle to more than f32: p * (hi + lo), its rounding error e turned into a first-order correction
-    const float a = (float)pos * freq.x, e = fmaf((float)pos, freq.x, -a) + (float)pos * freq.y;
-    float s, c;
-    sincosf(a, &s, &c);
-    sn = fmaf(c, e, s);
-    cs = fmaf(-s, e, c);
+    const float p = (float)pos, a = p * freq.x, e = fmaf(p, freq.x, -a) + p * freq.y;
+    sincospif(2.0f * ((a - rintf(a)) + e), &sn, &cs);
+}
+
+struct RecBlock {
+    int row0, n, first;                  // rows, place of the first one in its run
+    bool split, last;                    // the run has more than one block; this is its last one
+    size_t slot;
+};
+DEVINL bool find_block(const RecurArgs& a, int t, RecBlock& b) {
+    __shared__ int s_run, s_first;
+    if (threadIdx.x < 32) {
+        int run, first;
+        find_row_tile(a.rows, a.runs, 1, kRecBlock, t, run, first);
+        if (threadIdx.x == 0) { s_run = run; s_first = first; }
+    }
+    __syncthreads();
+    if (s_run < 0) return false;
+    b.first = s_first;
+    b.row0 = a.rows.row0[s_run] + b.first;
+    b.n = min(kRecBlock, a.rows.n[s_run] - b.first);
+    b.split = a.rows.n[s_run] > kRecBlock;
+    b.last = b.first + b.n == a.rows.n[s_run];
+    b.slot = 2 * (size_t)(b.row0 / kRecBlock) + (b.n < kRecBlock ? 1 : 0);
+    return true;
 }
 
 template <int KIND, typename WT, int KS, int KPT, int TILE>
@@ -451,6 +482,339 @@ __global__ void __launch_bounds__(kRecThreads) recur_kernel(const RecurArgs a) {
             for (int i = 0; i < KPT; ++i)
                 if (channel(i) < a.dim) sj[channel(i)] = S[j][i];
         }
+    }
+}
+
+// two f32 multiply-adds or products per instruction
+DEVINL uint64_t fma_f32x2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+DEVINL uint64_t mul_f32x2(uint64_t a, uint64_t b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+DEVINL uint64_t pack_f32x2(float x, float y) {
+    uint64_t d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(x), "f"(y));
+    return d;
+}
+DEVINL float2 unpack_f32x2(uint64_t v) {
+    float2 d;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(v));
+    return d;
+}
+
+// tokens staged at a time: 37 KB of q, k and v at most, so that six CTAs fit on an SM
+__host__ __device__ constexpr int rec_stage(int dp) { return dp <= 128 ? 32 : dp <= 256 ? 16 : 8; }
+__host__ __device__ constexpr size_t fixed_recur_smem(int ks, int kpt) { return sizeof(float) * rec_stage(ks * kpt) * (2 * ks * kpt + kRecThreads / ks * kRecCols); }
+
+// One block of a run per CTA: grid (heads, slices of vdim, blocks), threads and key channels as in recur_kernel, two channels
+// per register pair. The loops are kept short on purpose: a launch of a few thousand instructions per warp spends its time on
+// fetching code that it runs once.
+template <int KIND, int KS, int KPT>
+__global__ void __launch_bounds__(kRecThreads, KPT <= 16 && KS <= 8 ? 5 : 3) fixed_recur_kernel(const RecurArgs a) {
+    constexpr int DP = KS * KPT, VG = kRecThreads / KS, VS = VG * kRecCols, ROWS = rec_stage(DP);
+    constexpr int NV = 2 * kRecCols;     // dot products of two tokens
+    static_assert(kRecCols == 2, "two value columns per thread");
+    constexpr int LD = 2 * DP + VS, L4 = LD / 4;             // a staged token: q | k | v
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* st = reinterpret_cast<float*>(smem_raw);          // [ROWS][LD]
+    const int tid = threadIdx.x, hd = blockIdx.x, v0 = blockIdx.y * VS, ks = tid % KS, vg = tid / KS;
+    const int hk = hd * a.dim, hv = hd * a.vdim;
+    auto channel = [&](int i) { return (i / 4) * (KS * 4) + ks * 4 + i % 4; };
+    RecBlock b;                                              // rows and positions were there before the preceding kernel
+    const bool any = find_block(a, blockIdx.z, b);
+    const int seq = any ? a.rows.seq_of(b.row0) : 0, pos = any ? a.rows.pos[b.row0] : 0;
+    pdl_wait();
+    pdl_launch();
+    if (!any) return;
+    const size_t mine = ((size_t)hd * a.vdim + v0 + vg) * a.dim, all = (size_t)a.heads * a.vdim * a.dim;
+    uint64_t S[kRecCols][KPT / 2];
+    const bool resume = b.first == 0 && pos > 0, vec = a.dim % 4 == 0;
+#pragma unroll
+    for (int j = 0; j < kRecCols; ++j) {
+        const bool have = resume && v0 + vg + j * VG < a.vdim;
+        const float* sj = a.state + seq * all + mine + (size_t)j * VG * a.dim;
+#pragma unroll
+        for (int i = 0; i < KPT; i += 4) {
+            const int c = channel(i);
+            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (have && c < a.dim) {
+                if (vec) x = *reinterpret_cast<const float4*>(sj + c);
+                else x = make_float4(sj[c], c + 1 < a.dim ? sj[c + 1] : 0.0f, c + 2 < a.dim ? sj[c + 2] : 0.0f, c + 3 < a.dim ? sj[c + 3] : 0.0f);
+            }
+            S[j][i / 2] = pack_f32x2(x.x, x.y);
+            S[j][i / 2 + 1] = pack_f32x2(x.z, x.w);
+        }
+    }
+    const float dh = a.decay[hd], kf = a.k_scale;
+    const bool vec_in = vec && (a.vdim & 3) == 0 && ((a.c_q | a.c_k | a.c_v | a.in.ld) & 3) == 0;
+    auto place = [&](int c, bool& ok) {                      // column of the input projection for column c of a staged token
+        const int d = c < DP ? c : c < 2 * DP ? c - DP : c - 2 * DP;
+        ok = c < 2 * DP ? d < a.dim : v0 + d < a.vdim;
+        return c < DP ? a.c_q + hk + d : c < 2 * DP ? a.c_k + hk + d : a.c_v + hv + v0 + d;
+    };
+    auto act = [&](float x, int c) { return KIND == REC_LIGHTNING ? silu(x) : c >= DP && c < 2 * DP ? x * kf : x; };
+#pragma unroll 1
+    for (int t0 = 0; t0 < b.n; t0 += ROWS) {
+        const int n = min(ROWS, b.n - t0), row = b.row0 + t0;
+        if (t0 > 0) __syncthreads();
+        if (vec_in) {
+            constexpr int U = 6;                             // loads in flight per thread
+#pragma unroll 1
+            for (int i0 = tid; i0 < ROWS * L4; i0 += U * kRecThreads) {
+                float4 v[U];
+#pragma unroll
+                for (int u = 0; u < U; ++u) v[u] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                const float* p = a.in.p + (size_t)row * a.in.ld;
+#pragma unroll 1
+                for (int s = 0; s < a.in.splits; ++s, p += a.in.stride) {
+                    float4 w[U];
+#pragma unroll
+                    for (int u = 0; u < U; ++u) {
+                        const int i = i0 + u * kRecThreads, t = i / L4;
+                        bool ok;
+                        const int c = place(i % L4 * 4, ok);
+                        w[u] = ok && t < n ? __ldcg(reinterpret_cast<const float4*>(p + (size_t)t * a.in.ld + c)) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                    }
+#pragma unroll
+                    for (int u = 0; u < U; ++u) { v[u].x += w[u].x; v[u].y += w[u].y; v[u].z += w[u].z; v[u].w += w[u].w; }
+                }
+#pragma unroll
+                for (int u = 0; u < U; ++u) {
+                    const int i = i0 + u * kRecThreads, c = i % L4 * 4;
+                    if (i < ROWS * L4) *reinterpret_cast<float4*>(st + 4 * i) = make_float4(act(v[u].x, c), act(v[u].y, c), act(v[u].z, c), act(v[u].w, c));
+                }
+            }
+        } else {
+#pragma unroll 1
+            for (int i = tid; i < ROWS * LD; i += kRecThreads) {
+                bool ok;
+                const int t = i / LD, c = i % LD, from = place(c, ok);
+                st[i] = ok && t < n ? act(a.in.at(row + t, from), c) : 0.0f;
+            }
+        }
+        if constexpr (KIND == REC_RETENTION) {
+            __syncthreads();
+            const int half = a.rot_dims / 2;
+#pragma unroll 1
+            for (int i = tid; i < n * half; i += kRecThreads) {
+                const int t = i / half, d = i % half;
+                float sn, cs;
+                rotation(pos + t0 + t, a.freq[d], sn, cs);
+                float *q = st + t * LD + d, *k = q + DP;
+                const float qu = q[0], qv = q[half], ku = k[0], kv = k[half];
+                q[0] = qu * cs - qv * sn;
+                q[half] = qv * cs + qu * sn;
+                k[0] = ku * cs - kv * sn;
+                k[half] = kv * cs + ku * sn;
+            }
+        }
+        __syncthreads();
+        if (blockIdx.y == 0 && b.first > 0) {
+            float* to = a.block_q + (size_t)row * a.heads * a.dim + hk;
+            if (vec) {
+#pragma unroll 4
+                for (int i = tid; i < n * (DP / 4); i += kRecThreads) {
+                    const int t = i / (DP / 4), d = i % (DP / 4) * 4;
+                    if (d < a.dim) *reinterpret_cast<float4*>(to + (size_t)t * a.heads * a.dim + d) = *reinterpret_cast<const float4*>(st + t * LD + d);
+                }
+            } else {
+#pragma unroll 1
+                for (int i = tid; i < n * DP; i += kRecThreads)
+                    if (i % DP < a.dim) to[(size_t)(i / DP) * a.heads * a.dim + i % DP] = st[i / DP * LD + i % DP];
+            }
+        }
+#pragma unroll 1
+        for (int t = 0; t < n; t += 2) {
+            uint64_t acc[2][kRecCols] = {};
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {                    // a second token that is not there (zeros) keeps the state
+                const float *q = st + (t + u) * LD + ks * 4, *k = q + DP, *v = st + (t + u) * LD + 2 * DP + vg;
+                const float f = t + u < n ? dh : 1.0f;
+                const uint64_t d2 = pack_f32x2(f, f);
+                uint64_t x[kRecCols];
+#pragma unroll
+                for (int j = 0; j < kRecCols; ++j) x[j] = pack_f32x2(v[j * VG], v[j * VG]);
+#pragma unroll
+                for (int i = 0; i < KPT; i += 4) {
+                    const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(q + i * KS), k4 = *reinterpret_cast<const ulonglong2*>(k + i * KS);
+#pragma unroll
+                    for (int j = 0; j < kRecCols; ++j) {
+                        uint64_t &s0 = S[j][i / 2], &s1 = S[j][i / 2 + 1];
+                        s0 = fma_f32x2(d2, s0, mul_f32x2(k4.x, x[j]));
+                        s1 = fma_f32x2(d2, s1, mul_f32x2(k4.y, x[j]));
+                        acc[u][j] = fma_f32x2(q4.x, s0, acc[u][j]);
+                        acc[u][j] = fma_f32x2(q4.y, s1, acc[u][j]);
+                    }
+                }
+            }
+            float o[NV];
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const float2 v = unpack_f32x2(acc[i / kRecCols][i % kRecCols]);
+                o[i] = v.x + v.y;
+            }
+            int first;
+            column_reduce<NV, KS>(o, ks, first);             // this lane's total is number `first`
+            const int u = first / kRecCols, c = vg + first % kRecCols * VG;
+            if (t + u < n && v0 + c < a.vdim && (KS <= NV || ks % (KS > NV ? KS / NV : 1) == 0))
+                a.out[(size_t)(row + t + u) * a.ld_out + hv + v0 + c] = o[0];
+        }
+    }
+    float* end = (b.split ? a.block_state + b.slot * all : a.state + seq * all) + mine;
+#pragma unroll
+    for (int j = 0; j < kRecCols; ++j) {
+        if (v0 + vg + j * VG >= a.vdim) continue;
+        float* sj = end + (size_t)j * VG * a.dim;
+#pragma unroll
+        for (int i = 0; i < KPT; i += 4) {
+            const int c = channel(i);
+            const float2 x = unpack_f32x2(S[j][i / 2]), y = unpack_f32x2(S[j][i / 2 + 1]);
+            if (c >= a.dim) continue;
+            if (vec) {
+                *reinterpret_cast<float4*>(sj + c) = make_float4(x.x, x.y, y.x, y.y);
+            } else {
+                sj[c] = x.x;
+                if (c + 1 < a.dim) sj[c + 1] = x.y;
+                if (c + 2 < a.dim) sj[c + 2] = y.x;
+                if (c + 3 < a.dim) sj[c + 3] = y.y;
+            }
+        }
+    }
+}
+
+// Adds the start states' share to the outputs of the blocks behind the first one of a run and stores the run's end state.
+// Grid (heads, slices of kJoinCols value columns, blocks); a thread owns 4 tokens x 4 value columns. dynamic shared memory:
+// join_smem(dim).
+constexpr int kJoinCols = 32, kJoinThreads = kRecBlock / 4 * (kJoinCols / 4);
+constexpr int kJoinQ = kRecBlock + 4, kJoinS = kJoinCols + 4;            // rows of the staged queries and states
+__host__ __device__ constexpr size_t join_smem(int dim) { return sizeof(float) * ((dim + 3) / 4 * 4) * (kJoinQ + kJoinS); }
+__global__ void __launch_bounds__(kJoinThreads) recur_join_kernel(const RecurArgs a) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    const int tid = threadIdx.x, hd = blockIdx.x, v0 = blockIdx.y * kJoinCols, nv = min(kJoinCols, a.vdim - v0);
+    const int dim = a.dim, dp = (dim + 3) / 4 * 4;
+    float* sq = reinterpret_cast<float*>(smem_raw);          // [dp][kJoinQ] queries, channel by channel
+    float* ss = sq + (size_t)dp * kJoinQ;                    // [dp][kJoinS] state at the block's start
+    __shared__ float pw[kRecBlock + 1];                      // powers of the decay
+    const float dh = a.decay[hd];
+    if (tid <= kRecBlock) pw[tid] = powf(dh, (float)tid);
+    RecBlock b;
+    const bool mine_to_do = find_block(a, blockIdx.z, b) && b.first > 0;
+    const int seq = mine_to_do ? a.rows.seq_of(b.row0) : 0;
+    pdl_wait();
+    pdl_launch();
+    if (!mine_to_do) return;
+    // the earlier blocks of the run are full and lie one behind the other
+    const size_t all = (size_t)a.heads * a.vdim * dim, here = ((size_t)hd * a.vdim + v0) * dim;
+    const float* e0 = a.block_state + 2 * (size_t)((b.row0 - b.first) / kRecBlock) * all + here;
+    const float* mine = a.block_state + b.slot * all + here;
+    float* st = a.state + seq * all + here;
+    const int earlier = b.first / kRecBlock;
+    const float* q_in = a.block_q + (size_t)b.row0 * a.heads * dim + hd * dim;
+    if (dim % 4 == 0) {
+        const float4 none = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        const int d4 = dim / 4;
+        constexpr int U = 8, W = 2;                          // loads in flight per thread: U, W * (kRecMaxBlocks + 1)
+#pragma unroll 1
+        for (int i0 = tid; i0 < kRecBlock * d4; i0 += U * kJoinThreads) {
+            float4 v[U];
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int i = i0 + u * kJoinThreads, t = i / d4, d = i % d4 * 4;
+                v[u] = t < b.n ? __ldcg(reinterpret_cast<const float4*>(q_in + (size_t)t * a.heads * dim + d)) : none;
+            }
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int i = i0 + u * kJoinThreads, t = i / d4;
+                float* to = sq + i % d4 * 4 * kJoinQ + t;
+                if (t < kRecBlock) { to[0] = v[u].x; to[kJoinQ] = v[u].y; to[2 * kJoinQ] = v[u].z; to[3 * kJoinQ] = v[u].w; }
+            }
+        }
+        __syncthreads();                                     // pw
+        const float p = pw[kRecBlock], pn = pw[b.n];
+#pragma unroll 1
+        for (int i0 = tid; i0 < kJoinCols * d4; i0 += W * kJoinThreads) {
+            float4 e[W][kRecMaxBlocks];                      // earlier blocks' end states, then this one's
+#pragma unroll
+            for (int u = 0; u < W; ++u) {
+                const int i = i0 + u * kJoinThreads, c = i / d4;
+                const size_t at = (size_t)4 * i;
+#pragma unroll
+                for (int j = 0; j < kRecMaxBlocks - 1; ++j)
+                    e[u][j] = c < nv && j < earlier ? __ldcg(reinterpret_cast<const float4*>(e0 + 2 * j * all + at)) : none;
+                e[u][kRecMaxBlocks - 1] = c < nv && b.last ? __ldcg(reinterpret_cast<const float4*>(mine + at)) : none;
+            }
+#pragma unroll
+            for (int u = 0; u < W; ++u) {
+                const int i = i0 + u * kJoinThreads, c = i / d4;
+                if (c >= kJoinCols) continue;
+                float4 s = none;
+#pragma unroll
+                for (int j = 0; j < kRecMaxBlocks - 1; ++j) {
+                    const float f = j < earlier ? p : 1.0f;
+                    s = make_float4(fmaf(s.x, f, e[u][j].x), fmaf(s.y, f, e[u][j].y), fmaf(s.z, f, e[u][j].z), fmaf(s.w, f, e[u][j].w));
+                }
+                float* to = ss + i % d4 * 4 * kJoinS + c;
+                to[0] = s.x; to[kJoinS] = s.y; to[2 * kJoinS] = s.z; to[3 * kJoinS] = s.w;
+                const float4 m = e[u][kRecMaxBlocks - 1];
+                if (c < nv && b.last)
+                    *reinterpret_cast<float4*>(st + (size_t)4 * i) = make_float4(fmaf(s.x, pn, m.x), fmaf(s.y, pn, m.y), fmaf(s.z, pn, m.z), fmaf(s.w, pn, m.w));
+            }
+        }
+    } else {
+        __syncthreads();
+#pragma unroll 1
+        for (int i = tid; i < kRecBlock * dp; i += kJoinThreads) {
+            const int t = i / dp, d = i % dp;
+            sq[d * kJoinQ + t] = t < b.n && d < dim ? __ldcg(q_in + (size_t)t * a.heads * dim + d) : 0.0f;
+        }
+#pragma unroll 1
+        for (int i = tid; i < kJoinCols * dp; i += kJoinThreads) {
+            const int c = i / dp, d = i % dp;
+            const size_t at = (size_t)c * dim + d;
+            float s = 0.0f;
+            if (c < nv && d < dim) {
+                for (int j = 0; j < earlier; ++j) s = fmaf(s, pw[kRecBlock], __ldcg(e0 + 2 * j * all + at));
+                if (b.last) st[at] = fmaf(s, pw[b.n], __ldcg(mine + at));
+            }
+            ss[d * kJoinS + c] = s;
+        }
+    }
+    __syncthreads();
+    const int t0 = tid / (kJoinCols / 4) * 4, c0 = tid % (kJoinCols / 4) * 4;
+    float acc[4][4] = {};
+#pragma unroll 4
+    for (int d = 0; d < dp; ++d) {
+        const float4 q = *reinterpret_cast<const float4*>(sq + d * kJoinQ + t0), x = *reinterpret_cast<const float4*>(ss + d * kJoinS + c0);
+        const float qe[4] = {q.x, q.y, q.z, q.w}, xe[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+        for (int t = 0; t < 4; ++t)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) acc[t][c] = fmaf(qe[t], xe[c], acc[t][c]);
+    }
+    float* out = a.out + (size_t)(b.row0 + t0) * a.ld_out + hd * a.vdim + v0 + c0;
+    if (((a.vdim | a.ld_out) & 3) == 0) {
+        float4 o[4];
+#pragma unroll
+        for (int t = 0; t < 4; ++t)
+            if (t0 + t < b.n && c0 < nv) o[t] = *reinterpret_cast<const float4*>(out + (size_t)t * a.ld_out);
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+            const float p = pw[t0 + t + 1];
+            if (t0 + t < b.n && c0 < nv)
+                *reinterpret_cast<float4*>(out + (size_t)t * a.ld_out) =
+                    make_float4(fmaf(p, acc[t][0], o[t].x), fmaf(p, acc[t][1], o[t].y), fmaf(p, acc[t][2], o[t].z), fmaf(p, acc[t][3], o[t].w));
+        }
+    } else {
+#pragma unroll
+        for (int t = 0; t < 4; ++t)
+#pragma unroll
+            for (int c = 0; c < 4; ++c)
+                if (t0 + t < b.n && c0 + c < nv) out[(size_t)t * a.ld_out + c] += pw[t0 + t + 1] * acc[t][c];
     }
 }
 
@@ -923,10 +1287,20 @@ struct HeadAttnArgs {
     RowCache cache;
 };
 
+template <int E> DEVINL void store_act_e(uint16_t* p, const float (&v)[E]) {
+    if constexpr (E == 4) store_x4(p, make_float4(v[0], v[1], v[2], v[3]));
+    else store_act(p, v[0]);
+}
+template <int E> DEVINL void store_act_e(float* p, const float (&v)[E]) {
+    if constexpr (E == 4) store_x4(p, make_float4(v[0], v[1], v[2], v[3]));
+    else store_act(p, v[0]);
+}
+
 // Queries [R, heads, ld_q] (BF16 rows padded with zeros for the tensor-core kernel, f32 rows of dim values for the other one)
-// and the cache append. grid (R, 3): queries, keys, values. dynamic shared memory heads * dim floats.
-template <typename QT, typename KT>
-__global__ void __launch_bounds__(256) head_prep_kernel(const HeadAttnArgs a, QT* q_out, int ld_q) {
+// and the cache append. E: values per access, 4 when the head sizes are multiples of 4. grid (R, 3): queries, keys, values;
+// up to 1024 threads. dynamic shared memory heads * dim floats.
+template <typename QT, typename KT, int E>
+__global__ void __launch_bounds__(1024) head_prep_kernel(const HeadAttnArgs a, QT* q_out, int ld_q) {
     __shared__ float red[32];
     extern __shared__ __align__(16) unsigned char smem_raw[];
     float* v = reinterpret_cast<float*>(smem_raw);
@@ -934,13 +1308,21 @@ __global__ void __launch_bounds__(256) head_prep_kernel(const HeadAttnArgs a, QT
     pdl_launch();
     const int r = blockIdx.x, part = blockIdx.y, tid = threadIdx.x;
     if (a.rows.tok[r] == kInactiveToken) return;
-    const int pos = a.rows.pos[r];
+    const int pos = a.rows.pos[r], seq = a.rows.seq_of(r);
     KT* pool = (KT*)a.cache.pool;
+    float t[E];
     if (part == 2) {
-        const int seq = a.rows.seq_of(r), vp = a.cache.ld - a.kd;
-        for (int i = tid; i < a.kv_heads * vp; i += blockDim.x) {
+        const int vp = a.cache.ld - a.kd;
+        for (int i = tid * E; i < a.kv_heads * vp; i += blockDim.x * E) {
             const int g = i / vp, d = i % vp, c = g * a.vdim + d;
-            store_act(pool + a.cache.row(seq, pos, g) + a.kd + d, d < a.vdim ? a.in.at(r, a.c_v + c) + a.v_b[c] : 0.0f);
+#pragma unroll
+            for (int e = 0; e < E; ++e) t[e] = 0.0f;
+            if (d < a.vdim) {
+                split_load<E>(a.in, r, a.c_v + c, t);
+#pragma unroll
+                for (int e = 0; e < E; ++e) t[e] += a.v_b[c + e];
+            }
+            store_act_e<E>(pool + a.cache.row(seq, pos, g) + a.kd + d, t);
         }
         return;
     }
@@ -948,25 +1330,25 @@ __global__ void __launch_bounds__(256) head_prep_kernel(const HeadAttnArgs a, QT
     const int n = (key ? a.kv_heads : a.heads) * a.dim, col = key ? a.c_k : a.c_q;
     const float *bias = key ? a.k_b : a.q_b, *w = key ? a.k_norm : a.q_norm;
     float ss[1] = {0.0f};
-    for (int i = tid; i < n; i += blockDim.x) {
-        const float t = a.in.at(r, col + i) + bias[i];
-        v[i] = t;
-        ss[0] += t * t;
+    for (int i = tid * E; i < n; i += blockDim.x * E) {
+        split_load<E>(a.in, r, col + i, t);
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+            t[e] += bias[i + e];
+            v[i + e] = t[e];
+            ss[0] += t[e] * t[e];
+        }
     }
     block_sum<1>(ss, red);
     float s = 1.0f / sqrtf(ss[0] / (float)n + a.eps);
-    if (key) {
-        const int seq = a.rows.seq_of(r);
-        for (int i = tid; i < a.kv_heads * a.kd; i += blockDim.x) {
-            const int g = i / a.kd, d = i % a.kd, c = g * a.dim + d;
-            store_act(pool + a.cache.row(seq, pos, g) + d, d < a.dim ? v[c] * s * w[c] : 0.0f);
-        }
-        return;
-    }
-    s *= 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.0f);
-    for (int i = tid; i < a.heads * ld_q; i += blockDim.x) {
-        const int h = i / ld_q, d = i % ld_q, c = h * a.dim + d;
-        store_act(q_out + ((size_t)r * a.heads + h) * ld_q + d, d < a.dim ? v[c] * s * w[c] : 0.0f);
+    if (!key) s *= 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.0f);
+    const int ld = key ? a.kd : ld_q, heads = key ? a.kv_heads : a.heads;
+    for (int i = tid * E; i < heads * ld; i += blockDim.x * E) {
+        const int h = i / ld, d = i % ld, c = h * a.dim + d;
+#pragma unroll
+        for (int e = 0; e < E; ++e) t[e] = d < a.dim ? v[c + e] * s * w[c + e] : 0.0f;
+        if (key) store_act_e<E>(pool + a.cache.row(seq, pos, h) + d, t);
+        else store_act_e<E>(q_out + ((size_t)r * a.heads + h) * ld_q + d, t);
     }
 }
 

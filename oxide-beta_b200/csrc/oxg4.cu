@@ -110,7 +110,7 @@ struct MixPlan {
     const float *out_norm = nullptr, *mu = nullptr, *w0 = nullptr, *u = nullptr, *decay = nullptr, *dq_norm = nullptr,
                 *dkv_norm = nullptr, *inv_freq = nullptr, *q_norm = nullptr, *k_norm = nullptr, *q_b = nullptr, *k_b = nullptr,
                 *v_b = nullptr, *sink = nullptr;
-    const float2* freq2 = nullptr;   // retention: angle per position, high and low part
+    const float2* freq2 = nullptr;   // retention: turns per position, high and low part
 };
 
 struct LayerPlan {            // Gemma4DecodeLayerPlan (gemma4_cuda/mod.rs:65-93)
@@ -780,7 +780,7 @@ struct oxg4_cache {
     void *mix_x = nullptr, *mix_y = nullptr, *x_q = nullptr, *x_u = nullptr, *x_l = nullptr;
     float *xf = nullptr, *in_buf = nullptr, *q_buf = nullptr, *uk_buf = nullptr, *uv_buf = nullptr, *wdec = nullptr, *lat_q = nullptr,
           *lat_o = nullptr, *lat_ml = nullptr;
-    float* lat_rot = nullptr;
+    float *lat_rot = nullptr, *block_state = nullptr;
     int lat_splits = 1;
 
     int32_t *dec_grp_row0 = nullptr, *dec_grp_n = nullptr;      // decode: one group per sequence

@@ -409,7 +409,7 @@ class Gemma4CudaState:
                                             repetition_penalty, _ptr(s), _ptr(out), C.byref(ms)))
         return out, s, ms.value
 
-    PROFILE_KINDS = ["qkv", "shift", "decay", "recur", "outnorm", "latent", "uq", "latsplit", "uk", "latq", "latmerge", "uv",
+    PROFILE_KINDS = ["qkv", "shift", "decay", "recur", "recjoin", "outnorm", "latent", "uq", "latsplit", "uk", "latq", "latmerge", "uv",
                      "latout", "qkv_post", "attn", "attn_merge", "o", "gateup", "down", "lmhead", "norm", "geglu", "sum",
                      "topk1", "topk2", "tp_pick", "allreduce", "allgather", "step_begin", "step_end"]
 
