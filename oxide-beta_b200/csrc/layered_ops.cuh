@@ -691,14 +691,14 @@ __global__ void __launch_bounds__(kRecThreads, KPT <= 16 && KS <= 8 ? 5 : 3) fix
 // Grid (heads, slices of kJoinCols value columns, blocks); a thread owns 4 tokens x 4 value columns. dynamic shared memory:
 // join_smem(dim).
 constexpr int kJoinCols = 32, kJoinThreads = kRecBlock / 4 * (kJoinCols / 4);
-constexpr int kJoinQ = kRecBlock + 4, kJoinS = kJoinCols + 4;            // rows of the staged queries and states
-__host__ __device__ constexpr size_t join_smem(int dim) { return sizeof(float) * ((dim + 3) / 4 * 4) * (kJoinQ + kJoinS); }
+__host__ __device__ constexpr int join_ld(int dim) { return (dim + 3) / 4 * 4 + 4; }     // neighbouring rows start 4 banks apart at dim 32, 64, ...
+__host__ __device__ constexpr size_t join_smem(int dim) { return sizeof(float) * join_ld(dim) * (kRecBlock + kJoinCols); }
 __global__ void __launch_bounds__(kJoinThreads) recur_join_kernel(const RecurArgs a) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int tid = threadIdx.x, hd = blockIdx.x, v0 = blockIdx.y * kJoinCols, nv = min(kJoinCols, a.vdim - v0);
-    const int dim = a.dim, dp = (dim + 3) / 4 * 4;
-    float* sq = reinterpret_cast<float*>(smem_raw);          // [dp][kJoinQ] queries, channel by channel
-    float* ss = sq + (size_t)dp * kJoinQ;                    // [dp][kJoinS] state at the block's start
+    const int dim = a.dim, ld = join_ld(dim), d4 = (ld - 4) / 4;
+    float* sq = reinterpret_cast<float*>(smem_raw);          // [kRecBlock][ld] queries
+    float* ss = sq + (size_t)kRecBlock * ld;                 // [kJoinCols][ld] state at the block's start
     __shared__ float pw[kRecBlock + 1];                      // powers of the decay
     const float dh = a.decay[hd];
     if (tid <= kRecBlock) pw[tid] = powf(dh, (float)tid);
@@ -708,6 +708,7 @@ __global__ void __launch_bounds__(kJoinThreads) recur_join_kernel(const RecurArg
     pdl_wait();
     pdl_launch();
     if (!mine_to_do) return;
+    __syncthreads();
     // the earlier blocks of the run are full and lie one behind the other
     const size_t all = (size_t)a.heads * a.vdim * dim, here = ((size_t)hd * a.vdim + v0) * dim;
     const float* e0 = a.block_state + 2 * (size_t)((b.row0 - b.first) / kRecBlock) * all + here;
@@ -715,10 +716,10 @@ __global__ void __launch_bounds__(kJoinThreads) recur_join_kernel(const RecurArg
     float* st = a.state + seq * all + here;
     const int earlier = b.first / kRecBlock;
     const float* q_in = a.block_q + (size_t)b.row0 * a.heads * dim + hd * dim;
+    const float p = pw[kRecBlock], pn = pw[b.n];
     if (dim % 4 == 0) {
         const float4 none = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        const int d4 = dim / 4;
-        constexpr int U = 8, W = 2;                          // loads in flight per thread: U, W * (kRecMaxBlocks + 1)
+        constexpr int U = 8, W = 2;                          // loads in flight per thread: U, W * kRecMaxBlocks
 #pragma unroll 1
         for (int i0 = tid; i0 < kRecBlock * d4; i0 += U * kJoinThreads) {
             float4 v[U];
@@ -730,12 +731,9 @@ __global__ void __launch_bounds__(kJoinThreads) recur_join_kernel(const RecurArg
 #pragma unroll
             for (int u = 0; u < U; ++u) {
                 const int i = i0 + u * kJoinThreads, t = i / d4;
-                float* to = sq + i % d4 * 4 * kJoinQ + t;
-                if (t < kRecBlock) { to[0] = v[u].x; to[kJoinQ] = v[u].y; to[2 * kJoinQ] = v[u].z; to[3 * kJoinQ] = v[u].w; }
+                if (t < kRecBlock) *reinterpret_cast<float4*>(sq + t * ld + i % d4 * 4) = v[u];
             }
         }
-        __syncthreads();                                     // pw
-        const float p = pw[kRecBlock], pn = pw[b.n];
 #pragma unroll 1
         for (int i0 = tid; i0 < kJoinCols * d4; i0 += W * kJoinThreads) {
             float4 e[W][kRecMaxBlocks];                      // earlier blocks' end states, then this one's
@@ -758,64 +756,61 @@ __global__ void __launch_bounds__(kJoinThreads) recur_join_kernel(const RecurArg
                     const float f = j < earlier ? p : 1.0f;
                     s = make_float4(fmaf(s.x, f, e[u][j].x), fmaf(s.y, f, e[u][j].y), fmaf(s.z, f, e[u][j].z), fmaf(s.w, f, e[u][j].w));
                 }
-                float* to = ss + i % d4 * 4 * kJoinS + c;
-                to[0] = s.x; to[kJoinS] = s.y; to[2 * kJoinS] = s.z; to[3 * kJoinS] = s.w;
+                *reinterpret_cast<float4*>(ss + c * ld + i % d4 * 4) = s;
                 const float4 m = e[u][kRecMaxBlocks - 1];
                 if (c < nv && b.last)
                     *reinterpret_cast<float4*>(st + (size_t)4 * i) = make_float4(fmaf(s.x, pn, m.x), fmaf(s.y, pn, m.y), fmaf(s.z, pn, m.z), fmaf(s.w, pn, m.w));
             }
         }
     } else {
-        __syncthreads();
 #pragma unroll 1
-        for (int i = tid; i < kRecBlock * dp; i += kJoinThreads) {
-            const int t = i / dp, d = i % dp;
-            sq[d * kJoinQ + t] = t < b.n && d < dim ? __ldcg(q_in + (size_t)t * a.heads * dim + d) : 0.0f;
+        for (int i = tid; i < kRecBlock * ld; i += kJoinThreads) {
+            const int t = i / ld, d = i % ld;
+            sq[i] = t < b.n && d < dim ? __ldcg(q_in + (size_t)t * a.heads * dim + d) : 0.0f;
         }
 #pragma unroll 1
-        for (int i = tid; i < kJoinCols * dp; i += kJoinThreads) {
-            const int c = i / dp, d = i % dp;
+        for (int i = tid; i < kJoinCols * ld; i += kJoinThreads) {
+            const int c = i / ld, d = i % ld;
             const size_t at = (size_t)c * dim + d;
             float s = 0.0f;
             if (c < nv && d < dim) {
-                for (int j = 0; j < earlier; ++j) s = fmaf(s, pw[kRecBlock], __ldcg(e0 + 2 * j * all + at));
-                if (b.last) st[at] = fmaf(s, pw[b.n], __ldcg(mine + at));
+                for (int j = 0; j < earlier; ++j) s = fmaf(s, p, __ldcg(e0 + 2 * j * all + at));
+                if (b.last) st[at] = fmaf(s, pn, __ldcg(mine + at));
             }
-            ss[d * kJoinS + c] = s;
+            ss[i] = s;
         }
     }
     __syncthreads();
-    const int t0 = tid / (kJoinCols / 4) * 4, c0 = tid % (kJoinCols / 4) * 4;
+    // tokens tg + 16 u, columns cg + 8 v: the rows that a warp reads together are neighbours
+    constexpr int TG = kRecBlock / 4, CG = kJoinCols / 4;
+    const int tg = tid / CG, cg = tid % CG;
     float acc[4][4] = {};
-#pragma unroll 4
-    for (int d = 0; d < dp; ++d) {
-        const float4 q = *reinterpret_cast<const float4*>(sq + d * kJoinQ + t0), x = *reinterpret_cast<const float4*>(ss + d * kJoinS + c0);
-        const float qe[4] = {q.x, q.y, q.z, q.w}, xe[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll 2
+    for (int d = 0; d < 4 * d4; d += 4) {
+        float4 q[4], x[4];
 #pragma unroll
-        for (int t = 0; t < 4; ++t)
-#pragma unroll
-            for (int c = 0; c < 4; ++c) acc[t][c] = fmaf(qe[t], xe[c], acc[t][c]);
-    }
-    float* out = a.out + (size_t)(b.row0 + t0) * a.ld_out + hd * a.vdim + v0 + c0;
-    if (((a.vdim | a.ld_out) & 3) == 0) {
-        float4 o[4];
-#pragma unroll
-        for (int t = 0; t < 4; ++t)
-            if (t0 + t < b.n && c0 < nv) o[t] = *reinterpret_cast<const float4*>(out + (size_t)t * a.ld_out);
-#pragma unroll
-        for (int t = 0; t < 4; ++t) {
-            const float p = pw[t0 + t + 1];
-            if (t0 + t < b.n && c0 < nv)
-                *reinterpret_cast<float4*>(out + (size_t)t * a.ld_out) =
-                    make_float4(fmaf(p, acc[t][0], o[t].x), fmaf(p, acc[t][1], o[t].y), fmaf(p, acc[t][2], o[t].z), fmaf(p, acc[t][3], o[t].w));
+        for (int u = 0; u < 4; ++u) {
+            q[u] = *reinterpret_cast<const float4*>(sq + (tg + TG * u) * ld + d);
+            x[u] = *reinterpret_cast<const float4*>(ss + (cg + CG * u) * ld + d);
         }
-    } else {
 #pragma unroll
-        for (int t = 0; t < 4; ++t)
+        for (int u = 0; u < 4; ++u)
 #pragma unroll
-            for (int c = 0; c < 4; ++c)
-                if (t0 + t < b.n && c0 + c < nv) out[(size_t)t * a.ld_out + c] += pw[t0 + t + 1] * acc[t][c];
+            for (int v = 0; v < 4; ++v)
+                acc[u][v] = fmaf(q[u].w, x[v].w, fmaf(q[u].z, x[v].z, fmaf(q[u].y, x[v].y, fmaf(q[u].x, x[v].x, acc[u][v]))));
     }
+    float* out = a.out + (size_t)b.row0 * a.ld_out + hd * a.vdim + v0;
+    float o[4][4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+#pragma unroll
+        for (int v = 0; v < 4; ++v)
+            o[u][v] = tg + TG * u < b.n && cg + CG * v < nv ? out[(size_t)(tg + TG * u) * a.ld_out + cg + CG * v] : 0.0f;
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+#pragma unroll
+        for (int v = 0; v < 4; ++v)
+            if (tg + TG * u < b.n && cg + CG * v < nv) out[(size_t)(tg + TG * u) * a.ld_out + cg + CG * v] = fmaf(pw[tg + TG * u + 1], acc[u][v], o[u][v]);
 }
 
 // ---- output norm and gate of a mixer ------------------------------------------------------------------------
