@@ -161,6 +161,25 @@ def test_table_reuse_after_reset(dtype):
         table.reset()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("lens", [(65, 1, 64, 70, 2), (128, 66, 62), (64, 65, 127), (256, 3), (3, 253), (130, 126, 200)])
+def test_runs_of_one_pass_of_all_lengths(lens, dtype):
+    """Runs that are shorter than, as long as and longer than a block of the recurrence, side by side in one pass, then more of each."""
+    pair = Pair(config([retention(2, 40, 36, (0.98, 0.9995)), retention(3, 10, 7, (0.9, 1.0, 0.5), rot_dims=6)]), dtype, seed=22)
+    tokens = [pair.prompt(2 * n + 1, seed=60 + i) for i, n in enumerate(lens)]
+    want = [pair.want(t) for t in tokens]
+    table = pair.table([2 * n + 1 for n in lens], batch=len(lens))
+    at = [0] * len(lens)
+    for take in (lens, [n + 1 for n in lens]):
+        flat = np.concatenate([t[a:a + n] for t, a, n in zip(tokens, at, take)])
+        got = pair.state.extend(flat, table, lens=list(take), want=range(flat.size))
+        i = 0
+        for b, n in enumerate(take):
+            assert error(got[i:i + n], want[b][at[b]:at[b] + n]) <= TOL[dtype], b
+            i += n
+            at[b] += n
+
+
 def far_key_edits(dim):
     """Weights under which token 63 is the only one whose key answers to the query that all tokens share: channel 1 of the
     embedding feeds the query, channel 0, which only token 63 has, the key."""
